@@ -129,3 +129,71 @@ class CacheConfig:
         for n in self.index_cache_shape:
             ix *= n
         return 2 * (kv + ix)
+
+
+@dataclass(frozen=True)
+class RingCacheConfig:
+    """Caches of a model whose layers see a bounded stretch of the sequence, one GPU.
+
+    Every layer has its own ring of key and value rows per lane: position ``p`` lives in slot ``p % ring(layer)``.  A layer that attends
+    inside chunks of ``chunk`` positions needs the rows of the current chunk only, so its ring has ``min(chunk, capacity)`` slots whatever
+    the context capacity; a layer that sees the whole sequence has one slot per position.  A layer with a short convolution over time also
+    keeps the last ``taps - 1`` projected rows of every lane.  Head rows are padded to a multiple of 8 elements (16-byte vectors).
+
+    ``geometry.layers[i].mixer`` gives a layer's ``kv_heads``, ``dim``, ``vdim``, ``chunk``, ``conv`` and ``qkv_width``.
+    """
+
+    geometry: object
+    context_capacity: int
+    lanes: int = 1
+    element_bytes: int = 2
+    page: int = 1
+
+    def __post_init__(self) -> None:
+        if self.context_capacity < 1 or not 1 <= self.lanes <= 8:
+            raise PlanValidationError("the context capacity must be positive and the lanes between 1 and 8")
+
+    def _mixer(self, layer: int):
+        return self.geometry.layers[layer].mixer
+
+    def ring(self, layer: int) -> int:
+        chunk = self._mixer(layer).chunk
+        return self.context_capacity if chunk is None else min(chunk, self.context_capacity)
+
+    def chunk(self, layer: int) -> int:
+        """Chunk length in positions (a chunk that nothing ends within the capacity is the capacity)."""
+        chunk = self._mixer(layer).chunk
+        return self.context_capacity if chunk is None else min(chunk, self.context_capacity)
+
+    def first_position(self, layer: int, position: int) -> int:
+        """The first position that ``position`` can see."""
+        return position // self.chunk(layer) * self.chunk(layer)
+
+    def ring_from(self, layer: int, start: int, rows: int) -> tuple[int, bool]:
+        """Which rows of a step ``start .. start + rows - 1`` the ring keeps: ``(first row, only afterwards)``.  The rows of the last
+        chunk are kept.  When that chunk began inside the step, its slots may still hold keys that earlier rows of the step see, so the
+        rows go in after the attention has read them."""
+        keep = self.first_position(layer, start + rows - 1)
+        return max(keep - start, 0), keep > start
+
+    def k_shape(self, layer: int) -> tuple[int, int, int, int]:
+        m = self._mixer(layer)
+        return (self.lanes, self.ring(layer), m.kv_heads, -(-m.dim // 8) * 8)
+
+    def v_shape(self, layer: int) -> tuple[int, int, int, int]:
+        m = self._mixer(layer)
+        return (self.lanes, self.ring(layer), m.kv_heads, -(-m.vdim // 8) * 8)
+
+    def conv_shape(self, layer: int) -> tuple[int, int, int]:
+        m = self._mixer(layer)
+        return (self.lanes, m.conv - 1, m.qkv_width)
+
+    def cache_bytes_per_gpu(self) -> int:
+        total = 0
+        for layer in range(len(self.geometry.layers)):
+            for shape in (self.k_shape(layer), self.v_shape(layer), self.conv_shape(layer)):
+                count = 1
+                for n in shape:
+                    count *= n
+                total += count * self.element_bytes
+        return total

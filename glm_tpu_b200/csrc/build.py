@@ -3,6 +3,9 @@
 ``python -m glm_tpu_b200.csrc.build`` (or ``build()``) cross-compiles without a GPU.  Objects are rebuilt
 only when a source or header is newer.  The library links nothing but the CUDA runtime, so it loads in
 any process (ctypes) and its path shows up in the process map.
+
+``build(component=...)`` compiles only what one model family launches (``COMPONENTS``) into a library of its own, unless the
+complete library is already there and current; it returns the path to load (``ops.native.select_library``).
 """
 
 from __future__ import annotations
@@ -18,6 +21,10 @@ OUT_DIR = CSRC.parent / "ops"
 LIB = OUT_DIR / "libglmb200.so"
 OBJ_DIR = CSRC / "build"
 NVCC = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
+# sources each model family needs when the complete library has not been built
+COMPONENTS = {
+    "namizen": ("parallel_block", "qkv_conv", "chunk_attention", "gemm_f32", "swiglu_rows", "gemv", "gemm_tcgen05", "misc", "peer_registry"),
+}
 FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden", "--expt-relaxed-constexpr",
@@ -31,9 +38,15 @@ def _stale(target: Path, deps: list[Path]) -> bool:
     return any(d.stat().st_mtime > stamp for d in deps)
 
 
-def build(verbose: bool = False, force: bool = False) -> Path:
+def build(verbose: bool = False, force: bool = False, component: str | None = None) -> Path:
     sources = sorted(CSRC.glob("*.cu"))
     headers = sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
+    target = LIB
+    if component in COMPONENTS:  # a family without an entry needs the complete library
+        if not force and not _stale(LIB, [*sources, *headers]):
+            return LIB
+        sources = [CSRC / (name + ".cu") for name in COMPONENTS[component]]
+        target = OUT_DIR / f"libglmb200_{component}.so"
     OBJ_DIR.mkdir(exist_ok=True)
     OUT_DIR.mkdir(exist_ok=True)
 
@@ -53,12 +66,12 @@ def build(verbose: bool = False, force: bool = False) -> Path:
 
     with ThreadPoolExecutor(max_workers=min(8, len(sources) or 1)) as pool:
         objects = list(pool.map(compile_one, sources))
-    if force or _stale(LIB, objects):
-        cmd = [NVCC, "-shared", "-o", str(LIB), *map(str, objects), "-lcudart"]
+    if force or _stale(target, objects):
+        cmd = [NVCC, "-shared", "-o", str(target), *map(str, objects), "-lcudart"]
         done = subprocess.run(cmd, capture_output=True, text=True)
         if done.returncode != 0:
             raise RuntimeError(f"link failed:\n{done.stdout}\n{done.stderr}")
-    return LIB
+    return target
 
 
 if __name__ == "__main__":

@@ -1,0 +1,595 @@
+// Causal attention inside chunks of the sequence, grouped query heads, a sink per query head:
+//
+//   query i sees key j  <=>  j <= i and j / chunk == i / chunk          (chunks counted from position 0 of the sequence)
+//   out_i = sum_j exp(s_ij) v_j / (exp(sink_h) + sum_j exp(s_ij)),       s_ij = scale * q_i . k_j
+//
+// Keys live in the lane's ring (slot = position mod ring, ring >= min(chunk, capacity): a ring holds the whole current chunk) and, for the
+// rows of a prefill step, in linear buffers whose row 0 is position `start`.  Scores, exponentials and sums are fp32; the weights enter
+// the product with the values as two bf16 pieces (value and remainder), so they keep 16 bits of mantissa.
+//
+//   chunk_attn_prefill_kernel  bf16, many rows of one sequence: 64 query rows of one head per CTA, mma.sync, cp.async double buffer
+//   chunk_attn_decode_kernel   bf16, one row per lane: up to 16 query heads of one key head per cluster; the keys are dealt to the warps of
+//                              the cluster's CTAs, the partial softmax states meet in distributed shared memory
+//   chunk_attn_any_kernel      any head size and element type, one CTA per (row, head): the 32-bit path and head sizes beyond 256
+//
+// The running maximum starts at the sink and the sum gets the sink's term once; the sink has no value.
+#include <cooperative_groups.h>
+
+#include "attention_core.cuh"
+#include "common.cuh"
+#include "vec8.cuh"
+
+namespace cg = cooperative_groups;
+
+struct ChunkAttnArgs {
+    const void* q;                            // [rows, H, dimp]
+    const void *k_new, *v_new;                // [rows, G, dimp], [rows, G, vdimp]; NULL: every key is in the ring (decode)
+    const void *k_ring, *v_ring;              // [lanes, ring, G, dimp], [lanes, ring, G, vdimp]
+    const float* sink;                        // [H], or NULL: no sink
+    const int *row_pos, *row_lane, *row_active;  // row_active may be NULL
+    void* out; int64_t out_stride;            // [rows, H * vdim (+ more)]
+    int rows, H, G, dim, dimp, vdim, vdimp;
+    int chunk, ring, capacity, lanes;
+    float scale;
+    uint32_t* status;
+};
+
+#define CA_LOG2E 1.4426950408889634f
+
+__device__ __forceinline__ int ca_lane(const ChunkAttnArgs& a, int row) {
+    const int lane = a.row_lane[row];
+    if (lane >= 0 && lane < a.lanes) return lane;
+    if (threadIdx.x == 0) raise_status(a.status, GLMB_STATUS_BAD_INDEX);
+    return min(max(lane, 0), a.lanes - 1);
+}
+__device__ __forceinline__ int ca_pos(const ChunkAttnArgs& a, int row) {
+    const int pos = a.row_pos[row];
+    if (pos >= 0 && pos < a.capacity) return pos;
+    if (threadIdx.x == 0) raise_status(a.status, GLMB_STATUS_BAD_INDEX);
+    return min(max(pos, 0), a.capacity - 1);
+}
+// bf16 value and bf16 remainder of two weights, packed as mma operands
+__device__ __forceinline__ void ca_split(float x, float y, uint32_t& hi, uint32_t& lo) {
+    hi = pack_bf16(x, y);
+    lo = pack_bf16(x - bf16_lo(hi), y - bf16_hi(hi));
+}
+__device__ __forceinline__ void ca_store2(bf16* p, float x, float y, bool both, bool aligned) {
+    if (both && aligned) {
+        *reinterpret_cast<uint32_t*>(p) = pack_bf16(x, y);
+    } else {
+        p[0] = __float2bfloat16_rn(x);
+        if (both) p[1] = __float2bfloat16_rn(y);
+    }
+}
+
+// ---------------------------------------------------------------------------------------------------
+#define CP_ROWS 64
+#define CP_KEYS 64
+#define CP_THREADS 128
+
+static inline size_t chunk_prefill_smem(int dk, int dv) {  // dk, dv: head sizes rounded up to 16
+    return (size_t)(CP_ROWS * (dk + 8) + 2 * CP_KEYS * (dk + 8) + 2 * CP_KEYS * (dv + 8)) * 2;
+}
+
+// DV: columns of the output accumulator (the value size rounded up to it).
+template <int DV>
+__global__ void __launch_bounds__(CP_THREADS) chunk_attn_prefill_kernel(ChunkAttnArgs a) {
+    GLMB_PDL_PROLOGUE();
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    const int dk = (a.dim + 15) & ~15, dv = (a.vdim + 15) & ~15;
+    const int KP = dk + 8, VP = dv + 8;  // padded rows (elements): 16-byte aligned, banks staggered for ldmatrix
+    bf16* q_s = reinterpret_cast<bf16*>(smem_raw);
+    bf16* k_s = q_s + CP_ROWS * KP;
+    bf16* v_s = k_s + 2 * CP_KEYS * KP;
+    const int head = blockIdx.y, group = head / (a.H / a.G);
+    const int r0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * CP_ROWS;  // the rows with most keys (towards a chunk's end) first
+    const int nrows = min(CP_ROWS, a.rows - r0);
+    const int start = ca_pos(a, 0), lane_id = ca_lane(a, 0);
+    const int first = start + r0, last = min(start + r0 + nrows, a.capacity) - 1;
+    const int key0 = first / a.chunk * a.chunk;
+    const int tiles = max((last - key0) / CP_KEYS + 1, 1);
+    const bf16* k_new = reinterpret_cast<const bf16*>(a.k_new) + (int64_t)group * a.dimp;
+    const bf16* v_new = reinterpret_cast<const bf16*>(a.v_new) + (int64_t)group * a.vdimp;
+    const bf16* k_ring = reinterpret_cast<const bf16*>(a.k_ring) + ((int64_t)lane_id * a.ring * a.G + group) * a.dimp;
+    const bf16* v_ring = reinterpret_cast<const bf16*>(a.v_ring) + ((int64_t)lane_id * a.ring * a.G + group) * a.vdimp;
+    const int tid = threadIdx.x;
+
+    auto load_rows = [&](bf16* dst, int stride, int pieces, const bf16* fresh, const bf16* ring, int padded, int key_base) {
+        const int have = padded / 8;
+        for (int i = tid; i < CP_KEYS * pieces; i += CP_THREADS) {
+            const int r = i / pieces, c = i % pieces, key = key_base + r;
+            bf16* d = dst + r * stride + c * 8;
+            if (key > last || c >= have) { *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0); continue; }
+            const bf16* src = key >= start ? fresh + (int64_t)(key - start) * a.G * padded : ring + (int64_t)(key % a.ring) * a.G * padded;
+            cp_async16(d, src + c * 8);
+        }
+    };
+    auto load_tile = [&](int t) {
+        load_rows(k_s + (t & 1) * CP_KEYS * KP, KP, dk / 8, k_new, k_ring, a.dimp, key0 + t * CP_KEYS);
+        load_rows(v_s + (t & 1) * CP_KEYS * VP, VP, dv / 8, v_new, v_ring, a.vdimp, key0 + t * CP_KEYS);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    {
+        const bf16* q = reinterpret_cast<const bf16*>(a.q) + ((int64_t)r0 * a.H + head) * a.dimp;
+        const int pieces = dk / 8, have = a.dimp / 8;
+        for (int i = tid; i < CP_ROWS * pieces; i += CP_THREADS) {
+            const int r = i / pieces, c = i % pieces;
+            bf16* d = q_s + r * KP + c * 8;
+            if (r < nrows && c < have) cp_async16(d, q + (int64_t)r * a.H * a.dimp + c * 8);
+            else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
+        }
+    }
+    load_tile(0);
+
+    const int warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+    const int mr = lane & 7, mi = lane >> 3;
+    const float scale2 = a.scale * CA_LOG2E;
+    const float sink2 = a.sink ? a.sink[head] * CA_LOG2E : -INFINITY;
+    float m[2] = {sink2, sink2}, l[2] = {0.f, 0.f};  // the sink's own term joins the sum at the end
+    int pos[2], lo[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        pos[i] = first + warp * 16 + g + 8 * i;
+        lo[i] = pos[i] / a.chunk * a.chunk;
+    }
+    const int warp_last = first + warp * 16 + 15, warp_lo = (first + warp * 16) / a.chunk * a.chunk;
+    float o[DV / 8][4];
+#pragma unroll
+    for (int j = 0; j < DV / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+
+    for (int t = 0; t < tiles; ++t) {
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
+        if (t + 1 < tiles) load_tile(t + 1);
+        const int key_base = key0 + t * CP_KEYS;
+        if (key_base > warp_last || key_base + CP_KEYS <= warp_lo) continue;  // nothing in this tile for the warp's rows
+        const bf16* kt = k_s + (t & 1) * CP_KEYS * KP;
+        const bf16* vt = v_s + (t & 1) * CP_KEYS * VP;
+        float s[8][4];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
+        const bf16* qa = q_s + (warp * 16 + mr + 8 * (mi & 1)) * KP + 8 * (mi >> 1);
+        const bf16* kb = kt + (mr + 8 * (mi >> 1)) * KP + 8 * (mi & 1);
+        for (int k0 = 0; k0 < dk; k0 += 16) {
+            uint32_t qf[4];
+            ldmatrix_x4(qf, qa + k0);
+#pragma unroll
+            for (int j = 0; j < 8; j += 2) {
+                uint32_t kf[4];
+                ldmatrix_x4(kf, kb + j * 8 * KP + k0);
+                mma_bf16_16816(s[j], qf, kf[0], kf[1]);
+                mma_bf16_16816(s[j + 1], qf, kf[2], kf[3]);
+            }
+        }
+        const bool edge = key_base < (warp_last / a.chunk * a.chunk) || key_base + CP_KEYS - 1 > first + warp * 16;
+        float mx[2] = {m[0], m[1]};
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int key = key_base + j * 8 + 2 * t4 + (e & 1), i = e >> 1;
+                float x = s[j][e] * scale2;
+                if (edge && (key > pos[i] || key < lo[i])) x = -INFINITY;
+                s[j][e] = x;
+                mx[i] = fmaxf(mx[i], x);
+            }
+        float fix[2], base[2];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));
+            mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
+            base[i] = mx[i] == -INFINITY ? 0.f : mx[i];
+            fix[i] = exp2f(m[i] - base[i]);
+            m[i] = mx[i];
+        }
+        float sum[2] = {0.f, 0.f};
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                s[j][e] = exp2f(s[j][e] - base[e >> 1]);
+                sum[e >> 1] += s[j][e];
+            }
+        l[0] = l[0] * fix[0] + sum[0];  // this thread's keys; the four threads of a row meet at the end
+        l[1] = l[1] * fix[1] + sum[1];
+#pragma unroll
+        for (int j = 0; j < DV / 8; ++j) { o[j][0] *= fix[0]; o[j][1] *= fix[0]; o[j][2] *= fix[1]; o[j][3] *= fix[1]; }
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk) {
+            uint32_t hi[4], lw[4];
+            ca_split(s[2 * kk][0], s[2 * kk][1], hi[0], lw[0]);
+            ca_split(s[2 * kk][2], s[2 * kk][3], hi[1], lw[1]);
+            ca_split(s[2 * kk + 1][0], s[2 * kk + 1][1], hi[2], lw[2]);
+            ca_split(s[2 * kk + 1][2], s[2 * kk + 1][3], hi[3], lw[3]);
+            const bf16* vb = vt + (kk * 16 + mr + 8 * (mi & 1)) * VP + 8 * (mi >> 1);
+#pragma unroll
+            for (int j = 0; j < DV / 8; j += 2)
+                if (j * 8 < dv) {
+                    uint32_t vf[4];
+                    ldmatrix_x4_trans(vf, vb + j * 8);
+                    mma_bf16_16816(o[j], hi, vf[0], vf[1]);
+                    mma_bf16_16816(o[j + 1], hi, vf[2], vf[3]);
+                    mma_bf16_16816(o[j], lw, vf[0], vf[1]);
+                    mma_bf16_16816(o[j + 1], lw, vf[2], vf[3]);
+                }
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        l[i] += __shfl_xor_sync(0xffffffffu, l[i], 1);
+        l[i] += __shfl_xor_sync(0xffffffffu, l[i], 2);
+        if (a.sink) l[i] += exp2f(sink2 - m[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        const int r = warp * 16 + g + 8 * i;
+        if (r >= nrows) continue;
+        bf16* dst = reinterpret_cast<bf16*>(a.out) + (int64_t)(r0 + r) * a.out_stride + (int64_t)head * a.vdim;
+        const bool aligned = !(reinterpret_cast<uintptr_t>(dst) & 3);
+        const float inv = 1.f / l[i];
+#pragma unroll
+        for (int j = 0; j < DV / 8; ++j) {
+            const int c = j * 8 + 2 * t4;
+            if (c < a.vdim) ca_store2(dst + c, o[j][2 * i] * inv, o[j][2 * i + 1] * inv, c + 1 < a.vdim, aligned);
+        }
+    }
+}
+
+// ---------------------------------------------------------------------------------------------------
+#define CD_WARPS 4
+#define CD_THREADS (CD_WARPS * 32)
+#define CD_HEADS 16
+#define CD_KEYS 16  // keys a warp takes at a time
+
+static inline size_t chunk_decode_smem(int dk, int dv, int stages) {
+    const size_t stage = (size_t)CD_WARPS * stages * CD_KEYS * (dk + 8 + dv + 8) * 2, merge = (size_t)CD_WARPS * CD_HEADS * dv * 4;
+    return (size_t)CD_HEADS * (dk + 8) * 2 + (stage > merge ? stage : merge);
+}
+
+// grid (splits, key heads x blocks of 16 query heads, rows), cluster (splits, 1, 1).
+template <int DV>
+__global__ void __launch_bounds__(CD_THREADS) chunk_attn_decode_kernel(ChunkAttnArgs a, int stages) {
+    GLMB_PDL_PROLOGUE();
+    cg::cluster_group cluster = cg::this_cluster();
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    __shared__ float ml_s[CD_WARPS][CD_HEADS][2];  // (maximum, sum) per warp
+    __shared__ float cta_ml[CD_HEADS][2];
+    const int dk = (a.dim + 15) & ~15, dv = (a.vdim + 15) & ~15, KP = dk + 8, VP = dv + 8;
+    const int per = a.H / a.G, head_blocks = (per + CD_HEADS - 1) / CD_HEADS;
+    const int group = blockIdx.y / head_blocks, h0 = group * per + (blockIdx.y % head_blocks) * CD_HEADS;
+    const int heads = min(CD_HEADS, group * per + per - h0);
+    const int row = blockIdx.z, split = blockIdx.x, splits = gridDim.x;
+    const bool active = !a.row_active || a.row_active[row] != 0;
+    const int pos = ca_pos(a, row), lane_id = ca_lane(a, row);
+    const int key0 = pos / a.chunk * a.chunk;
+    const int keys = active ? pos - key0 + 1 : 0;
+    bf16* q_s = reinterpret_cast<bf16*>(smem_raw);
+    unsigned char* rest = smem_raw + (size_t)CD_HEADS * KP * 2;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3, mr = lane & 7, mi = lane >> 3;
+    bf16* kv_s = reinterpret_cast<bf16*>(rest) + (size_t)warp * stages * CD_KEYS * (KP + VP);
+    const bf16* k_ring = reinterpret_cast<const bf16*>(a.k_ring) + ((int64_t)lane_id * a.ring * a.G + group) * a.dimp;
+    const bf16* v_ring = reinterpret_cast<const bf16*>(a.v_ring) + ((int64_t)lane_id * a.ring * a.G + group) * a.vdimp;
+
+    const int blocks = (keys + CD_KEYS - 1) / CD_KEYS, stride = splits * CD_WARPS, b0 = split * CD_WARPS + warp;
+    auto load_block = [&](int b, int stage) {  // 16 keys and values of this warp
+        if (b < blocks) {
+            bf16* kd = kv_s + (size_t)stage * CD_KEYS * (KP + VP);
+            bf16* vd = kd + CD_KEYS * KP;
+            const int kp = dk / 8, vp = dv / 8, key_base = key0 + b * CD_KEYS;
+            for (int i = lane; i < CD_KEYS * (kp + vp); i += 32) {
+                const int r = i / (kp + vp), c = i % (kp + vp), key = key_base + r;
+                const bool is_k = c < kp;
+                const int col = is_k ? c : c - kp, have = (is_k ? a.dimp : a.vdimp) / 8;
+                bf16* d = is_k ? kd + r * KP + col * 8 : vd + r * VP + col * 8;
+                if (key > pos || col >= have) { *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0); continue; }
+                const int64_t slot = (int64_t)(key % a.ring) * a.G;
+                cp_async16(d, is_k ? k_ring + slot * a.dimp + col * 8 : v_ring + slot * a.vdimp + col * 8);
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    {
+        const bf16* q = reinterpret_cast<const bf16*>(a.q) + ((int64_t)row * a.H + h0) * a.dimp;
+        const int pieces = dk / 8, have = a.dimp / 8;
+        for (int i = threadIdx.x; i < CD_HEADS * pieces; i += CD_THREADS) {
+            const int r = i / pieces, c = i % pieces;
+            uint4 v = make_uint4(0, 0, 0, 0);
+            if (r < heads && c < have) v = *reinterpret_cast<const uint4*>(q + (int64_t)r * a.dimp + c * 8);
+            *reinterpret_cast<uint4*>(q_s + r * KP + c * 8) = v;
+        }
+    }
+    for (int s = 0; s < stages - 1; ++s) load_block(b0 + s * stride, s);
+    __syncthreads();
+
+    const float scale2 = a.scale * CA_LOG2E;
+    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+    float o[DV / 8][4];
+#pragma unroll
+    for (int j = 0; j < DV / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+    const bf16* qa = q_s + (mr + 8 * (mi & 1)) * KP + 8 * (mi >> 1);
+    int stage = 0;
+    for (int b = b0; b < blocks; b += stride) {
+        load_block(b + (stages - 1) * stride, (stage + stages - 1) % stages);
+        if (stages == 2) asm volatile("cp.async.wait_group 1;" ::: "memory");
+        else if (stages == 3) asm volatile("cp.async.wait_group 2;" ::: "memory");
+        else asm volatile("cp.async.wait_group 3;" ::: "memory");
+        __syncwarp();
+        const bf16* kt = kv_s + (size_t)stage * CD_KEYS * (KP + VP);
+        const bf16* vt = kt + CD_KEYS * KP;
+        float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+        const bf16* kb = kt + (mr + 8 * (mi >> 1)) * KP + 8 * (mi & 1);
+        for (int k0 = 0; k0 < dk; k0 += 16) {
+            uint32_t qf[4], kf[4];
+            ldmatrix_x4(qf, qa + k0);
+            ldmatrix_x4(kf, kb + k0);
+            mma_bf16_16816(s[0], qf, kf[0], kf[1]);
+            mma_bf16_16816(s[1], qf, kf[2], kf[3]);
+        }
+        float mx[2] = {m[0], m[1]};
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int key = key0 + b * CD_KEYS + j * 8 + 2 * t4 + (e & 1);
+                const float x = key > pos ? -INFINITY : s[j][e] * scale2;
+                s[j][e] = x;
+                mx[e >> 1] = fmaxf(mx[e >> 1], x);
+            }
+        float fix[2];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));
+            mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
+            fix[i] = exp2f(m[i] - mx[i]);  // a block holds at least one visible key: the maximum is finite
+            m[i] = mx[i];
+        }
+        float sum[2] = {0.f, 0.f};
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                s[j][e] = exp2f(s[j][e] - m[e >> 1]);
+                sum[e >> 1] += s[j][e];
+            }
+        l[0] = l[0] * fix[0] + sum[0];
+        l[1] = l[1] * fix[1] + sum[1];
+        uint32_t hi[4], lw[4];
+        ca_split(s[0][0], s[0][1], hi[0], lw[0]);
+        ca_split(s[0][2], s[0][3], hi[1], lw[1]);
+        ca_split(s[1][0], s[1][1], hi[2], lw[2]);
+        ca_split(s[1][2], s[1][3], hi[3], lw[3]);
+        const bf16* vb = vt + (mr + 8 * (mi & 1)) * VP + 8 * (mi >> 1);
+#pragma unroll
+        for (int j = 0; j < DV / 8; j += 2)
+            if (j * 8 < dv) {
+                o[j][0] *= fix[0]; o[j][1] *= fix[0]; o[j][2] *= fix[1]; o[j][3] *= fix[1];
+                o[j + 1][0] *= fix[0]; o[j + 1][1] *= fix[0]; o[j + 1][2] *= fix[1]; o[j + 1][3] *= fix[1];
+                uint32_t vf[4];
+                ldmatrix_x4_trans(vf, vb + j * 8);
+                mma_bf16_16816(o[j], hi, vf[0], vf[1]);
+                mma_bf16_16816(o[j + 1], hi, vf[2], vf[3]);
+                mma_bf16_16816(o[j], lw, vf[0], vf[1]);
+                mma_bf16_16816(o[j + 1], lw, vf[2], vf[3]);
+            }
+        __syncwarp();  // everyone is done with this stage before it is filled again
+        stage = (stage + 1) % stages;
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        l[i] += __shfl_xor_sync(0xffffffffu, l[i], 1);
+        l[i] += __shfl_xor_sync(0xffffffffu, l[i], 2);
+        if (t4 == 0) { ml_s[warp][g + 8 * i][0] = m[i]; ml_s[warp][g + 8 * i][1] = l[i]; }
+    }
+    __syncthreads();  // every warp has left its key and value stages: the merge area takes their place
+    float* o_s = reinterpret_cast<float*>(rest);  // [warp][head][dv]
+#pragma unroll
+    for (int j = 0; j < DV / 8; ++j)
+        if (j * 8 < dv) {
+            float* d = o_s + ((size_t)warp * CD_HEADS + g) * dv + j * 8 + 2 * t4;
+            *reinterpret_cast<float2*>(d) = make_float2(o[j][0], o[j][1]);
+            *reinterpret_cast<float2*>(d + 8 * dv) = make_float2(o[j][2], o[j][3]);
+        }
+    __syncthreads();
+    // ---- warps of the CTA into warp 0's area ------------------------------------------------------------
+    if (threadIdx.x < CD_HEADS) {
+        float top = -INFINITY, sum = 0.f;
+        for (int w = 0; w < CD_WARPS; ++w) top = fmaxf(top, ml_s[w][threadIdx.x][0]);
+        for (int w = 0; w < CD_WARPS; ++w)
+            if (ml_s[w][threadIdx.x][0] != -INFINITY) sum += ml_s[w][threadIdx.x][1] * exp2f(ml_s[w][threadIdx.x][0] - top);
+        cta_ml[threadIdx.x][0] = top;
+        cta_ml[threadIdx.x][1] = sum;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < CD_HEADS * dv; i += CD_THREADS) {
+        const int h = i / dv;
+        const float top = cta_ml[h][0];
+        float v = 0.f;
+        for (int w = 0; w < CD_WARPS; ++w)
+            if (ml_s[w][h][0] != -INFINITY) v += o_s[(size_t)w * CD_HEADS * dv + i] * exp2f(ml_s[w][h][0] - top);
+        o_s[i] = v;
+    }
+    cluster.sync();
+    // ---- CTAs of the cluster: each finishes its share of the outputs, the sink joins here -----------------
+    const int total = heads * a.vdim;
+    bf16* out = reinterpret_cast<bf16*>(a.out) + (int64_t)row * a.out_stride + (int64_t)h0 * a.vdim;
+    for (int i = split * CD_THREADS + threadIdx.x; i < total; i += splits * CD_THREADS) {
+        const int h = i / a.vdim, c = i % a.vdim;
+        const float sink2 = a.sink ? a.sink[h0 + h] * CA_LOG2E : -INFINITY;
+        float top = sink2;
+        for (int p = 0; p < splits; ++p) top = fmaxf(top, cluster.map_shared_rank(&cta_ml[0][0], p)[h * 2]);
+        float sum = a.sink ? exp2f(sink2 - top) : 0.f, v = 0.f;
+        for (int p = 0; p < splits; ++p) {
+            const float* pml = cluster.map_shared_rank(&cta_ml[0][0], p);
+            if (pml[h * 2] == -INFINITY) continue;
+            const float w = exp2f(pml[h * 2] - top);
+            sum += pml[h * 2 + 1] * w;
+            v += cluster.map_shared_rank(o_s, p)[h * dv + c] * w;
+        }
+        out[i] = __float2bfloat16_rn(sum > 0.f ? v / sum : 0.f);
+    }
+    cluster.sync();  // nobody leaves while a peer may still read its shared memory
+}
+
+// ---------------------------------------------------------------------------------------------------
+#define CX_THREADS 128
+#define CX_KEYS 128
+#define CX_COLS 8  // value columns per thread: value sizes up to 1024
+
+template <typename T>
+__global__ void __launch_bounds__(CX_THREADS) chunk_attn_any_kernel(ChunkAttnArgs a) {
+    GLMB_PDL_PROLOGUE();
+    extern __shared__ float q_f[];  // [dim]
+    __shared__ float p_s[CX_KEYS];
+    __shared__ float red[CX_THREADS / 32];
+    const int row = blockIdx.x, head = blockIdx.y, group = head / (a.H / a.G);
+    const bool decode = a.k_new == nullptr;
+    const bool active = !a.row_active || a.row_active[row] != 0;
+    const int start = decode ? a.capacity : ca_pos(a, 0);
+    const int pos = ca_pos(a, row), lane_id = ca_lane(a, decode ? row : 0);
+    const int key0 = pos / a.chunk * a.chunk, keys = active ? pos - key0 + 1 : 0;
+    const T* q = reinterpret_cast<const T*>(a.q) + ((int64_t)row * a.H + head) * a.dimp;
+    for (int d = threadIdx.x; d < a.dim; d += CX_THREADS) q_f[d] = to_f32(q[d]);
+    __syncthreads();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    auto at = [&](const void* fresh, const void* ring, int padded, int key) {
+        return key >= start ? reinterpret_cast<const T*>(fresh) + ((int64_t)(key - start) * a.G + group) * padded
+                            : reinterpret_cast<const T*>(ring) + (((int64_t)lane_id * a.ring + key % a.ring) * a.G + group) * padded;
+    };
+    float m = a.sink ? a.sink[head] : -INFINITY, l = a.sink ? 1.f : 0.f;
+    float acc[CX_COLS];
+#pragma unroll
+    for (int i = 0; i < CX_COLS; ++i) acc[i] = 0.f;
+    for (int t = 0; t < keys; t += CX_KEYS) {
+        const int n = min(CX_KEYS, keys - t);
+        for (int j = warp; j < n; j += CX_THREADS / 32) {
+            const T* k = at(a.k_new, a.k_ring, a.dimp, key0 + t + j);
+            float s = 0.f;
+            for (int d = lane; d < a.dim; d += 32) s = fmaf(q_f[d], to_f32(k[d]), s);
+            s = warp_sum(s);
+            if (lane == 0) p_s[j] = s * a.scale;
+        }
+        __syncthreads();
+        const float x = (int)threadIdx.x < n ? p_s[threadIdx.x] : -INFINITY;
+        float top = warp_max(x);
+        if (lane == 0) red[warp] = top;
+        __syncthreads();
+        top = m;
+#pragma unroll
+        for (int w = 0; w < CX_THREADS / 32; ++w) top = fmaxf(top, red[w]);
+        const float fix = expf(m - top), p = (int)threadIdx.x < n ? expf(x - top) : 0.f;
+        __syncthreads();
+        p_s[threadIdx.x] = p;
+        const float part = warp_sum(p);
+        if (lane == 0) red[warp] = part;
+        __syncthreads();
+        float sum = 0.f;
+#pragma unroll
+        for (int w = 0; w < CX_THREADS / 32; ++w) sum += red[w];
+        l = l * fix + sum;
+        m = top;
+#pragma unroll
+        for (int i = 0; i < CX_COLS; ++i) acc[i] *= fix;
+        for (int j = 0; j < n; ++j) {
+            const T* v = at(a.v_new, a.v_ring, a.vdimp, key0 + t + j);
+            const float w = p_s[j];
+#pragma unroll
+            for (int i = 0; i < CX_COLS; ++i) {
+                const int c = threadIdx.x + i * CX_THREADS;
+                if (c < a.vdim) acc[i] = fmaf(w, to_f32(v[c]), acc[i]);
+            }
+        }
+        __syncthreads();
+    }
+    T* out = reinterpret_cast<T*>(a.out) + (int64_t)row * a.out_stride + (int64_t)head * a.vdim;
+#pragma unroll
+    for (int i = 0; i < CX_COLS; ++i) {
+        const int c = threadIdx.x + i * CX_THREADS;
+        if (c < a.vdim) from_f32(l > 0.f ? acc[i] / l : 0.f, out[c]);
+    }
+}
+
+// ===================================================================================================
+static bool chunk_args_ok(const ChunkAttnArgs& a) {
+    return a.rows >= 1 && a.H >= 1 && a.G >= 1 && a.H % a.G == 0 && a.dim >= 1 && a.vdim >= 1 && !(a.dimp & 7) && !(a.vdimp & 7) && a.dimp >= a.dim &&
+           a.vdimp >= a.vdim && a.chunk >= 1 && a.ring >= 1 && a.capacity >= 1 && a.lanes >= 1 && (a.ring >= a.chunk || a.ring >= a.capacity);
+}
+
+template <typename K>
+static cudaError_t chunk_smem_limit(K kernel, DeviceOnce& once) {
+    const int dev = once.pending();
+    if (dev == DeviceOnce::SET) return cudaSuccess;
+    const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    if (e == cudaSuccess) once.mark(dev);
+    return e;
+}
+
+template <int DV>
+static int launch_chunk_prefill(const ChunkAttnArgs& a, cudaStream_t st) {
+    static DeviceOnce once;
+    const cudaError_t e = chunk_smem_limit(chunk_attn_prefill_kernel<DV>, once);
+    if (e != cudaSuccess) return (int)e;
+    const size_t smem = chunk_prefill_smem((a.dim + 15) & ~15, (a.vdim + 15) & ~15);
+    GLMB_LAUNCH(chunk_attn_prefill_kernel<DV>, dim3(ceil_div(a.rows, CP_ROWS), a.H), CP_THREADS, smem, st, a);
+    return (int)cudaGetLastError();
+}
+
+template <int DV>
+static int launch_chunk_decode(const ChunkAttnArgs& a, int splits, cudaStream_t st) {
+    static DeviceOnce once;
+    const cudaError_t e = chunk_smem_limit(chunk_attn_decode_kernel<DV>, once);
+    if (e != cudaSuccess) return (int)e;
+    const int dk = (a.dim + 15) & ~15, dv = (a.vdim + 15) & ~15;
+    int stages = 4;
+    while (stages > 2 && chunk_decode_smem(dk, dv, stages) > 112 * 1024) --stages;
+    const int per = a.H / a.G;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(splits, a.G * ceil_div(per, CD_HEADS), a.rows);
+    cfg.blockDim = dim3(CD_THREADS);
+    cfg.dynamicSmemBytes = chunk_decode_smem(dk, dv, stages);
+    cfg.stream = st;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = g_glmb_pdl_enabled ? 1 : 0;
+    attr[1].id = cudaLaunchAttributeClusterDimension;
+    attr[1].val.clusterDim.x = splits;
+    attr[1].val.clusterDim.y = attr[1].val.clusterDim.z = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = 2;
+    const cudaError_t le = cudaLaunchKernelEx(&cfg, chunk_attn_decode_kernel<DV>, a, stages);
+    return le != cudaSuccess ? (int)le : (int)cudaGetLastError();
+}
+
+GLMB_API size_t glmb_chunk_attn_args_sizeof(void) { return sizeof(ChunkAttnArgs); }
+
+// bf16, rows of one sequence at consecutive positions; head sizes up to 256.
+GLMB_API int glmb_chunk_attn_prefill(const ChunkAttnArgs* args, void* stream) {
+    const ChunkAttnArgs a = *args;
+    if (!chunk_args_ok(a) || !a.k_new || !a.v_new || a.dim > 256 || a.vdim > 256) return 1;
+    if (a.vdim <= 64) return launch_chunk_prefill<64>(a, (cudaStream_t)stream);
+    if (a.vdim <= 128) return launch_chunk_prefill<128>(a, (cudaStream_t)stream);
+    return launch_chunk_prefill<256>(a, (cudaStream_t)stream);
+}
+
+// bf16, one row per sequence, every key in the ring; head sizes up to 256.
+GLMB_API int glmb_chunk_attn_decode(const ChunkAttnArgs* args, void* stream) {
+    const ChunkAttnArgs a = *args;
+    if (!chunk_args_ok(a) || a.k_new || a.v_new || a.dim > 256 || a.vdim > 256) return 1;
+    // CTAs per cluster: enough that a full ring leaves each warp a few blocks of keys, at most the portable cluster size
+    int splits = 1;
+    while (splits < 8 && a.ring > splits * CD_WARPS * CD_KEYS) splits *= 2;
+    if (a.vdim <= 64) return launch_chunk_decode<64>(a, splits, (cudaStream_t)stream);
+    if (a.vdim <= 128) return launch_chunk_decode<128>(a, splits, (cudaStream_t)stream);
+    return launch_chunk_decode<256>(a, splits, (cudaStream_t)stream);
+}
+
+// Any head size (values up to 1024 columns), bf16 or fp32.
+GLMB_API int glmb_chunk_attn_any(const ChunkAttnArgs* args, int is_f32, void* stream) {
+    const ChunkAttnArgs a = *args;
+    if (!chunk_args_ok(a) || !a.k_new != !a.v_new || a.vdim > CX_THREADS * CX_COLS || a.dim > 8192) return 1;
+    const dim3 grid(a.rows, a.H);
+    const size_t smem = (size_t)a.dim * sizeof(float);
+    if (is_f32) GLMB_LAUNCH(chunk_attn_any_kernel<float>, grid, CX_THREADS, smem, (cudaStream_t)stream, a);
+    else GLMB_LAUNCH(chunk_attn_any_kernel<bf16>, grid, CX_THREADS, smem, (cudaStream_t)stream, a);
+    return (int)cudaGetLastError();
+}

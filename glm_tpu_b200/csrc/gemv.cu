@@ -39,7 +39,8 @@ __device__ __forceinline__ void sk_prefetch_rows(const void* first_row, int rows
 
 // ---------------------------------------------------------------------------------------------------
 // out[r][n] = sum_k x[r][k] * w[n][k]          (bf16 weights)
-enum { SK_OUT_F32 = 0, SK_OUT_BF16 = 1, SK_OUT_ALLREDUCE_BF16 = 2, SK_OUT_ARGMAX = 3 };
+// ARGMAX compares bf16-rounded logits, ARGMAX_F32 the fp32 sums themselves.
+enum { SK_OUT_F32 = 0, SK_OUT_BF16 = 1, SK_OUT_ALLREDUCE_BF16 = 2, SK_OUT_ARGMAX = 3, SK_OUT_ARGMAX_F32 = 4 };
 
 // ks (1, 2, 4 or 8) warps of a CTA split K for the same pair of output rows and add their partial sums through
 // shared memory: small-N projections then still fill the machine.  A CTA produces 16 / ks output rows.
@@ -114,7 +115,7 @@ skinny_bf16_kernel(const bf16* __restrict__ x, int64_t xs, int rows, const bf16*
         }
         return;
     }
-    if (mode == SK_OUT_ARGMAX) {
+    if (mode == SK_OUT_ARGMAX || mode == SK_OUT_ARGMAX_F32) {
         // out: unsigned long long best[rows]; `channel` carries the id of output column 0 (vocabulary offset).
         __shared__ unsigned long long best_s[SK_WARPS][R];
         if (lane == 0) {
@@ -124,7 +125,7 @@ skinny_bf16_kernel(const bf16* __restrict__ x, int64_t xs, int rows, const bf16*
 #pragma unroll
                 for (int j = 0; j < 2; ++j)
                     if (kpart == 0 && n0 + j < N) {
-                        const float v = bf16_round(acc[j][r]);
+                        const float v = mode == SK_OUT_ARGMAX ? bf16_round(acc[j][r]) : acc[j][r];
                         if (!isfinite(v)) raise_status(comm.status, GLMB_STATUS_NONFINITE);
                         const unsigned long long k2 = candidate_key(v, channel + n0 + j);
                         key = k2 > key ? k2 : key;

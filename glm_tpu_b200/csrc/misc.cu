@@ -67,19 +67,23 @@ router_topk256_kernel(const float* __restrict__ logits, const float* __restrict_
 
 // ---------------------------------------------------------------------------------------------------
 // cand [world][rows][2] (fp32 value, int32 global id) lives in the staging buffer when world > 1.
+__device__ __forceinline__ float logit_f32(bf16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ float logit_f32(float v) { return v; }
+
+template <typename T>
 __global__ void __launch_bounds__(1024)
-argmax_rows_kernel(const bf16* __restrict__ logits, int64_t stride, int V, int vocab_base, float* __restrict__ cand,
+argmax_rows_kernel(const T* __restrict__ logits, int64_t stride, int V, int vocab_base, float* __restrict__ cand,
                    int64_t cand_offset, PeerComm comm, int sig, uint32_t* status) {
     GLMB_PDL_PROLOGUE();
     __shared__ float s_val[32];
     __shared__ int s_idx[32];
     const int r = blockIdx.x, rows = gridDim.x;
-    const bf16* lg = logits + (int64_t)r * stride;
+    const T* lg = logits + (int64_t)r * stride;
     float best = -INFINITY;
     int best_i = 0x7fffffff;
     bool bad = false;
     for (int i = threadIdx.x; i < V; i += blockDim.x) {
-        const float v = __bfloat162float(lg[i]);
+        const float v = logit_f32(lg[i]);
         if (!isfinite(v)) bad = true;
         if (v > best || (v == best && i < best_i)) { best = v; best_i = i; }
     }
@@ -221,8 +225,17 @@ GLMB_API int glmb_argmax_rows(const void* logits, int64_t stride, int rows, int 
                               const PeerComm* comm, int sig, uint32_t* status, void* stream) {
     PeerComm c;
     if (comm) c = *comm; else { memset(&c, 0, sizeof(c)); c.world = 1; }
-    GLMB_LAUNCH(argmax_rows_kernel, rows, 1024, 0, (cudaStream_t)stream, (const bf16*)logits, stride, V, vocab_base, cand, cand_offset, c, sig,
+    GLMB_LAUNCH(argmax_rows_kernel<bf16>, rows, 1024, 0, (cudaStream_t)stream, (const bf16*)logits, stride, V, vocab_base, cand, cand_offset, c, sig,
                                                                 status);
+    return (int)cudaGetLastError();
+}
+
+// The same over fp32 logits.
+GLMB_API int glmb_argmax_rows_f32(const float* logits, int64_t stride, int rows, int V, int vocab_base, float* cand, int64_t cand_offset,
+                                  const PeerComm* comm, int sig, uint32_t* status, void* stream) {
+    PeerComm c;
+    if (comm) c = *comm; else { memset(&c, 0, sizeof(c)); c.world = 1; }
+    GLMB_LAUNCH(argmax_rows_kernel<float>, rows, 1024, 0, (cudaStream_t)stream, logits, stride, V, vocab_base, cand, cand_offset, c, sig, status);
     return (int)cudaGetLastError();
 }
 

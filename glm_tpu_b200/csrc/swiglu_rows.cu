@@ -4,6 +4,7 @@
 //
 // Reference counterpart: `glm_tpu/layers/mlp.py:21-51`.
 #include "common.cuh"
+#include "vec8.cuh"
 
 __global__ void __launch_bounds__(256)
 swiglu_rows_kernel(const uint4* __restrict__ gate, const uint4* __restrict__ up, uint4* __restrict__ act, int64_t n8) {
@@ -29,5 +30,42 @@ GLMB_API int glmb_swiglu_rows(const void* gate, const void* up, void* act, int64
     const int64_t blocks = (n8 + 255) / 256;
     const int grid = blocks < 148 * 8 ? (int)blocks : 148 * 8;
     GLMB_LAUNCH(swiglu_rows_kernel, grid, 256, 0, (cudaStream_t)stream, (const uint4*)gate, (const uint4*)up, (uint4*)act, n8);
+    return (int)cudaGetLastError();
+}
+
+// Gated activation of strided rows: act[r][i] = f(gate[r][i]) * up[r][i] for i < n (a multiple of 8), f by `kind` (vec8.cuh), arithmetic
+// in fp32 and one rounding.  gate and up may be the two halves of one projection's output, act the tail of a wider row.
+template <typename T>
+__global__ void __launch_bounds__(256)
+glu_rows_kernel(const T* __restrict__ gate, const T* __restrict__ up, int64_t in_stride, T* __restrict__ act, int64_t out_stride, int rows, int n,
+                int kind) {
+    GLMB_PDL_PROLOGUE();
+    const int per_row = n / 8;
+    const int64_t total = (int64_t)rows * per_row;
+    for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
+        const int64_t r = i / per_row;
+        const int c = (int)(i % per_row) * 8;
+        float g[8], u[8];
+        load8(gate + r * in_stride + c, g);
+        load8(up + r * in_stride + c, u);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) g[e] = glu_activation(kind, g[e]) * u[e];
+        store8(act + r * out_stride + c, g);
+    }
+}
+
+// n and both strides multiples of 8 elements, all pointers 16-byte aligned.
+GLMB_API int glmb_glu_rows(const void* gate, const void* up, int64_t in_stride, void* act, int64_t out_stride, int rows, int n, int kind, int is_f32,
+                           void* stream) {
+    if (rows < 1 || n < 8 || (n & 7) || (in_stride & 7) || (out_stride & 7) || (kind != GLU_SILU && kind != GLU_GELU_TANH)) return 1;
+    if ((reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(up) | reinterpret_cast<uintptr_t>(act)) & 15) return 1;
+    const int64_t blocks = ((int64_t)rows * (n / 8) + 255) / 256;
+    const int grid = blocks < 148 * 8 ? (int)blocks : 148 * 8;
+    if (is_f32)
+        GLMB_LAUNCH(glu_rows_kernel<float>, grid, 256, 0, (cudaStream_t)stream, (const float*)gate, (const float*)up, in_stride, (float*)act, out_stride,
+                    rows, n, kind);
+    else
+        GLMB_LAUNCH(glu_rows_kernel<bf16>, grid, 256, 0, (cudaStream_t)stream, (const bf16*)gate, (const bf16*)up, in_stride, (bf16*)act, out_stride,
+                    rows, n, kind);
     return (int)cudaGetLastError();
 }

@@ -2,6 +2,7 @@
 
     info                         supported scope and limits
     ask [QUESTION | --questions FILE] [--context 8k|32k|128k|256k] [--concurrent] [--keep-loaded] ...
+    trace                        replay given token ids step by step and write the logits
     prepare-request              messages or token ids -> prepared request (nothing is launched)
     collect-env | doctor         environment report checked against a profile
     checkpoint inventory|mark-source|pack|verify
@@ -28,6 +29,8 @@ def _info(args) -> int:
     print(json.dumps({
         "engine": "glm_tpu_b200",
         "model": "GlmMoeDsaForCausalLM (GLM-5.3), FP8 e4m3 routed experts with 128x128 block scales, bf16 elsewhere",
+        "other_models": {"Namizen": "small parallel-block decoder with chunked attention; bf16 (32-bit for checks), one GPU, any directory "
+                                    "with its config.json and safetensors"},
         "hardware": "one box of 1, 2, 4 or 8 NVIDIA B200 (sm_100a) with NVLink peer access",
         "modes": ["one-shot answer", "sequential queue (<= 10)", "four concurrent chats (32k)", "resident session",
                   "loopback chat UI", "OpenAI-compatible /v1 (chat completions, models, tools, SSE)"],
@@ -41,6 +44,12 @@ def _info(args) -> int:
 
 def _ask(args) -> int:
     from glm_tpu_b200.entrypoints.cli.ask import main
+
+    return main(args)
+
+
+def _trace(args) -> int:
+    from glm_tpu_b200.entrypoints.cli.trace import main
 
     return main(args)
 
@@ -106,11 +115,18 @@ def build_parser() -> argparse.ArgumentParser:
     ask.add_argument("--max-new-tokens", type=int)
     ask.add_argument("--wall-seconds", type=int, default=86400)
     ask.add_argument("--prepare-only", action="store_true")
-    ask.add_argument("--model", help="random:<tiny|small|glm53>[:layers] or a packed checkpoint (default: the site's)")
+    ask.add_argument("--model", help="random:<tiny|small|glm53|namizen-tiny>[:layers], a packed checkpoint, or a Namizen directory (default: the site's)")
     ask.add_argument("--backend", choices=("gpu", "oracle"), default="gpu")
     ask.add_argument("--gpus", type=int)
     ask.add_argument("--site", type=Path)
     ask.set_defaults(fn=_ask)
+
+    trace = sub.add_parser("trace", help="replay given token ids (JSON steps on standard input) and write the logits")
+    trace.add_argument("--model", required=True, help="a directory with config.json and weights (or random:<preset>)")
+    trace.add_argument("--dtype", choices=("bfloat16", "float32"), default="bfloat16")
+    trace.add_argument("--out", type=Path, required=True, help="directory the logits of every step are written to")
+    trace.add_argument("--max-tokens", type=int, required=True, help="the most tokens that live requests hold at any time")
+    trace.set_defaults(fn=_trace)
 
     prep = sub.add_parser("prepare-request", help="prepare a request without launching the model")
     source = prep.add_mutually_exclusive_group(required=True)

@@ -32,8 +32,7 @@ from glm_tpu_b200.models.glm_moe_dsa.weights import DeviceWeights, LayerWeights
 from glm_tpu_b200.ops import native
 from glm_tpu_b200.oracle.contract import rope_table
 from glm_tpu_b200.parallel.peer import PeerGroup
-
-RING = 64
+from glm_tpu_b200.runner.lane_state import RING, LaneRegisters
 
 
 def _f32(x: float) -> float:
@@ -41,38 +40,20 @@ def _f32(x: float) -> float:
 
 
 @dataclass
-class DecoderState:
+class DecoderState(LaneRegisters):
     """Device-resident caches and lane registers (reference ``models/glm_moe_dsa/state.py:23-69``)."""
 
-    kv_cache: torch.Tensor  # [lanes, layers, local_cap, W] bf16
-    index_cache: torch.Tensor  # [lanes, full_layers, local_cap, D] bf16
-    tokens: torch.Tensor  # [lanes] int32: the token each lane feeds next
-    positions: torch.Tensor  # [lanes] int32: its position (= tokens already cached)
-    active: torch.Tensor  # [lanes] int32
-    lane_ids: torch.Tensor  # [lanes] int32 arange
-    out_tokens: torch.Tensor  # [RING, lanes] int32
-    step_counter: torch.Tensor  # [1] int32
+    kv_cache: torch.Tensor | None = None  # [lanes, layers, local_cap, W] bf16
+    index_cache: torch.Tensor | None = None  # [lanes, full_layers, local_cap, D] bf16
 
     @classmethod
     def allocate(cls, cache: CacheConfig, device) -> "DecoderState":
         dev = torch.device(device)
-        z = lambda *s: torch.zeros(s, dtype=torch.int32, device=dev)  # noqa: E731
         return cls(
+            **cls.registers(cache.lanes, dev),
             kv_cache=torch.zeros(cache.kv_cache_shape, dtype=torch.bfloat16, device=dev),
             index_cache=torch.zeros(cache.index_cache_shape, dtype=torch.bfloat16, device=dev),
-            tokens=z(cache.lanes),
-            positions=z(cache.lanes),
-            active=z(cache.lanes),
-            lane_ids=torch.arange(cache.lanes, dtype=torch.int32, device=dev),
-            out_tokens=torch.full((RING, cache.lanes), -1, dtype=torch.int32, device=dev),
-            step_counter=z(1),
         )
-
-    def reset_lane(self, lane: int) -> None:
-        """Fresh cache for a new request on ``lane`` (stale rows are never read: reads are bounded by the position)."""
-        self.positions[lane] = 0
-        self.tokens[lane] = 0
-        self.active[lane] = 0
 
 
 class Workspace:

@@ -1,7 +1,8 @@
 """ctypes binding of ``libglmb200.so`` (the hand-written sm_100a kernels).
 
 The library is built in-tree by ``glm_tpu_b200.csrc.build`` and loaded with ``ctypes`` (it links only the
-CUDA runtime).  Every wrapper takes torch CUDA tensors, passes raw device pointers plus the current torch
+CUDA runtime).  ``select_library`` names another build of the same kernels: the component library that holds just what one model
+family launches.  Every wrapper takes torch CUDA tensors, passes raw device pointers plus the current torch
 stream, and raises on a non-zero return code.  There is no fallback: if the library is missing or a launch
 fails on a GPU machine the call raises.
 """
@@ -17,7 +18,8 @@ LIB_PATH = Path(__file__).resolve().parent / "libglmb200.so"
 MAX_WORLD = 8
 MAX_ROWS = 8
 
-SK_OUT_F32, SK_OUT_BF16, SK_OUT_ALLREDUCE_BF16, SK_OUT_ARGMAX = 0, 1, 2, 3
+SK_OUT_F32, SK_OUT_BF16, SK_OUT_ALLREDUCE_BF16, SK_OUT_ARGMAX, SK_OUT_ARGMAX_F32 = 0, 1, 2, 3, 4
+GLU_SILU, GLU_GELU_TANH = 0, 1
 STATUS_WAIT_TIMEOUT, STATUS_BAD_INDEX, STATUS_NONFINITE, STATUS_BAD_SHAPE = 1, 2, 4, 8
 
 # signals (producer -> consumer exchanges) and all-reduce channels used by the model
@@ -65,11 +67,49 @@ class QPostArgs(C.Structure):
     ]
 
 
+class QkvConvArgs(C.Structure):
+    _fields_ = [
+        ("proj", C.c_void_p), ("proj_stride", C.c_int64),
+        ("conv_w", C.c_void_p), ("taps", C.c_int),
+        ("state", C.c_void_p),
+        ("row_pos", C.c_void_p), ("row_lane", C.c_void_p), ("row_active", C.c_void_p),
+        ("rot", C.c_void_p), ("rot_dims", C.c_int),
+        ("q", C.c_void_p), ("k_new", C.c_void_p), ("v_new", C.c_void_p),
+        ("k_ring", C.c_void_p), ("v_ring", C.c_void_p), ("ring", C.c_int),
+        ("v_first", C.c_void_p), ("v_mode", C.c_int), ("mix", C.c_float),
+        ("H", C.c_int), ("G", C.c_int), ("dim", C.c_int), ("dimp", C.c_int), ("vdim", C.c_int), ("vdimp", C.c_int), ("rows", C.c_int),
+        ("decode", C.c_int), ("ring_from", C.c_int), ("capacity", C.c_int), ("lanes", C.c_int), ("rows_per_block", C.c_int),
+        ("status", C.c_void_p),
+    ]
+
+
+class ChunkAttnArgs(C.Structure):
+    _fields_ = [
+        ("q", C.c_void_p), ("k_new", C.c_void_p), ("v_new", C.c_void_p), ("k_ring", C.c_void_p), ("v_ring", C.c_void_p), ("sink", C.c_void_p),
+        ("row_pos", C.c_void_p), ("row_lane", C.c_void_p), ("row_active", C.c_void_p),
+        ("out", C.c_void_p), ("out_stride", C.c_int64),
+        ("rows", C.c_int), ("H", C.c_int), ("G", C.c_int), ("dim", C.c_int), ("dimp", C.c_int), ("vdim", C.c_int), ("vdimp", C.c_int),
+        ("chunk", C.c_int), ("ring", C.c_int), ("capacity", C.c_int), ("lanes", C.c_int),
+        ("scale", C.c_float),
+        ("status", C.c_void_p),
+    ]
+
+
 _lib = None
 
 
 def available() -> bool:
     return LIB_PATH.exists()
+
+
+def select_library(path) -> None:
+    """Load the kernels from ``path`` (a library built by ``csrc.build``).  One library per process: naming another one after the
+    first has been loaded is an error."""
+    global LIB_PATH
+    path = Path(path).resolve()
+    if _lib is not None and path != LIB_PATH.resolve():
+        raise RuntimeError(f"{LIB_PATH.name} is already loaded in this process")
+    LIB_PATH = path
 
 
 def lib() -> C.CDLL:
@@ -82,7 +122,12 @@ def lib() -> C.CDLL:
         _lib.glmb_peer_comm_sizeof.restype = C.c_size_t
         _lib.glmb_peer_data.restype = C.c_void_p
         _lib.glmb_peer_status_ptr.restype = C.c_void_p
-        _lib.glmb_indexer_rows_scratch_bytes.restype = C.c_int64
+        if hasattr(_lib, "glmb_indexer_rows_scratch_bytes"):  # a component library holds one family's kernels only
+            _lib.glmb_indexer_rows_scratch_bytes.restype = C.c_int64
+        for entry, struct in (("glmb_qkv_conv_args_sizeof", QkvConvArgs), ("glmb_chunk_attn_args_sizeof", ChunkAttnArgs)):
+            getattr(_lib, entry).restype = C.c_size_t
+            if getattr(_lib, entry)() != C.sizeof(struct):
+                raise RuntimeError(f"{struct.__name__} layout differs between Python and the CUDA library")
         if _lib.glmb_peer_comm_sizeof() != C.sizeof(PeerComm):
             raise RuntimeError("PeerComm layout differs between Python and the CUDA library")
         import os
@@ -305,6 +350,13 @@ def swiglu_rows(gate, up, act=None):
     return act
 
 
+def glu_rows(gate, up, act, kind):
+    """``act[r, :n] = f(gate[r]) * up[r]`` for strided rows (``kind``: ``GLU_SILU`` or ``GLU_GELU_TANH``); bf16 or fp32, fp32 arithmetic."""
+    rows, n = gate.shape
+    _check(lib().glmb_glu_rows(_p(gate), _p(up), C.c_int64(gate.stride(0)), _p(act), C.c_int64(act.stride(0)), rows, n, int(kind),
+                               int(gate.dtype == torch.float32), _stream()), "glu_rows")
+
+
 def route_sort128(topk_ids, ebase: int, el: int, tiles, n_tiles, perm) -> None:
     """Stable sort of this GPU's routes by expert, cut into 128-route tiles, in one launch (see csrc/route_sort.cu).
 
@@ -359,6 +411,50 @@ def embed_rows(tokens, table, residual, status):
 def add_rmsnorm(update, residual, weight, out, eps):
     rows, H = residual.shape
     _check(lib().glmb_add_rmsnorm(_p(update), _p(residual), _p(weight), _p(out), rows, H, f32(eps), _stream()), "add_rmsnorm")
+
+
+def parallel_norm(residual, width, w1, out1, eps, *, w2=None, out2=None, update=None, tokens=None, table=None, vocab=0, status=None):
+    """Both RMS-normalized inputs of a parallel layer from one fp32 residual: ``residual += update`` (fp32), or ``residual =
+    table[tokens]``, first; then ``out = residual / sqrt(mean(residual**2) + eps) * w``.  Rows are padded to a multiple of 8 columns."""
+    rows, padded = out1.shape
+    _check(lib().glmb_parallel_norm(_p(tokens), _p(table), int(vocab), _p(update), _p(residual), rows, int(width), padded, _p(w1), _p(w2), _p(out1),
+                                    _p(out2), f32(eps), int(out1.dtype == torch.float32), _p(status), _stream()), "parallel_norm")
+
+
+def dual_proj(x1, w, out, x2=None, wg=None, wu=None, act=None, kind=GLU_SILU):
+    """Decode (1..8 rows, bf16): ``out = x1 @ w.T`` and, from another input, ``act = f(x2 @ wg.T) * (x2 @ wu.T)`` in one launch."""
+    rows, K = x1.shape
+    _check(lib().glmb_dual_proj(_p(x1), _p(x2), C.c_int64(x1.stride(0)), rows, K, _p(w), w.shape[0], _p(out), C.c_int64(out.stride(0)), _p(wg), _p(wu),
+                                wg.shape[0] if wg is not None else 0, _p(act), C.c_int64(act.stride(0) if act is not None else 0), int(kind),
+                                _stream()), "dual_proj")
+
+
+# ----------------------------------------------------------------------------- short convolution, ring cache, chunked attention
+def qkv_conv_max_taps(widest_head: int) -> int:
+    return int(lib().glmb_qkv_conv_max_taps(int(widest_head)))
+
+
+def qkv_conv(args: QkvConvArgs, is_f32: bool) -> None:
+    """Short causal convolution, rotation, value mixing and cache write of an attention layer's fused q | k | v projection."""
+    _check(lib().glmb_qkv_conv(C.byref(args), int(is_f32), _stream()), "qkv_conv")
+
+
+def ring_store(args: QkvConvArgs, first: int, is_f32: bool) -> None:
+    """Rows ``first ..`` of a step's linear key / value buffers into the lane's ring (``args`` of the ``qkv_conv`` that made them)."""
+    _check(lib().glmb_ring_store(C.c_void_p(args.k_new), C.c_void_p(args.v_new), C.c_void_p(args.row_pos), C.c_void_p(args.row_lane),
+                                 C.c_void_p(args.k_ring), C.c_void_p(args.v_ring), args.ring, args.G * args.dimp, args.G * args.vdimp, int(first),
+                                 args.rows, args.lanes, args.capacity, int(is_f32), _stream()), "ring_store")
+
+
+def chunk_attention(args: ChunkAttnArgs, is_f32: bool, *, plain: bool = False) -> None:
+    """Chunked causal attention with sinks.  bf16 heads up to 256 wide run on the tensor cores (``k_new`` set: prefill, otherwise decode);
+    other head sizes, the 32-bit path and ``plain=True`` take the kernel that needs no particular size."""
+    if plain or is_f32 or max(args.dim, args.vdim) > 256:
+        _check(lib().glmb_chunk_attn_any(C.byref(args), int(is_f32), _stream()), "chunk_attn_any")
+    elif args.k_new:
+        _check(lib().glmb_chunk_attn_prefill(C.byref(args), _stream()), "chunk_attn_prefill")
+    else:
+        _check(lib().glmb_chunk_attn_decode(C.byref(args), _stream()), "chunk_attn_decode")
 
 
 def set_qkv_fast(enabled: int) -> None:
@@ -548,8 +644,9 @@ def router_topk(logits, bias, top_k, ids, weights):
 
 def argmax_rows(logits, rows, V, vocab_base, cand, cand_offset=0, comm=None, sig=SIG_SAMPLE, status=None):
     _note_signal("argmax_rows", comm, sig)
+    entry = lib().glmb_argmax_rows_f32 if logits.dtype == torch.float32 else lib().glmb_argmax_rows
     _check(
-        lib().glmb_argmax_rows(_p(logits), C.c_int64(logits.stride(0)), rows, V, vocab_base, _p(cand), C.c_int64(cand_offset),
+        entry(_p(logits), C.c_int64(logits.stride(0)), rows, V, vocab_base, _p(cand), C.c_int64(cand_offset),
                                _comm(comm), sig, _p(status), _stream()),
         "argmax_rows",
     )
@@ -618,6 +715,13 @@ def gemm_bf16_tc_allreduce(a, b, comm, part_offset, out_offset, *, sig=SIG_GEMM,
 
 def wait_signal(comm, sig):
     _check(lib().glmb_wait_signal(_comm(comm), sig, _stream()), "wait_signal")
+
+
+def gemm_f32(a, b, out):
+    """``out[rows, N] = a @ b.T`` in plain fp32 (no reduced-precision tensor mode)."""
+    rows, K = a.shape
+    _check(lib().glmb_gemm_f32(_p(a), C.c_int64(a.stride(0)), _p(b), C.c_int64(b.stride(0)), _p(out), C.c_int64(out.stride(0)), rows, b.shape[0], K,
+                               _stream()), "gemm_f32")
 
 
 def set_mega_cooperative(enabled: int) -> None:

@@ -1,6 +1,6 @@
-"""Per-GPU model runner: resident weights, caches, the prefill program and the CUDA-graph decode program.
+"""The GLM-MoE-DSA runner of one GPU: resident weights, caches, the prefill program and the CUDA-graph decode program.
 
-The runner is what the engine drives.  It owns
+The runner is what the engine drives (``LaneRunner`` is the part it shares with the other model families).  It owns
 
 * the resident weights (``DeviceWeights``) and the peer-buffer registry,
 * the device state for ``lanes`` concurrent chats (striped KV/index caches, token/position registers),
@@ -17,59 +17,20 @@ from __future__ import annotations
 
 import os
 import time
-from dataclasses import dataclass, field
 
 import torch
 
 from glm_tpu_b200.config.cache import CacheConfig
 from glm_tpu_b200.config.parallel import ParallelLayout, default_expert_split
-from glm_tpu_b200.models.glm_moe_dsa.model import RING, DecoderState, GlmMoeDsaModel, Workspace
+from glm_tpu_b200.models.glm_moe_dsa.model import DecoderState, GlmMoeDsaModel, Workspace
 from glm_tpu_b200.models.glm_moe_dsa.weights import DeviceWeights
 from glm_tpu_b200.ops import native
 from glm_tpu_b200.parallel.peer import PeerGroup
-from glm_tpu_b200.runner.admission import check_collective_plan, project_live, project_memory, require_admitted
+from glm_tpu_b200.runner.admission import project_live, project_memory, require_admitted
+from glm_tpu_b200.runner.lane_runner import LaneRunner, ProgramRecord, RunnerReport
 
 
-@dataclass
-class ProgramRecord:
-    name: str
-    kind: str  # 'cuda_graph' or 'eager'
-    rows: int
-    launches: int
-    capture_seconds: float = 0.0
-
-
-@dataclass
-class RunnerReport:
-    phases: dict = field(default_factory=dict)
-    programs: list = field(default_factory=list)
-    memory: dict = field(default_factory=dict)
-
-
-class _LaunchCounter:
-    """Counts kernel launches issued through the native library while a program is being recorded."""
-
-    def __init__(self):
-        self.count = 0
-
-    def __enter__(self):
-        from glm_tpu_b200.ops import native
-
-        self._native = native
-        self._orig = native._check
-
-        def counting(code, what):
-            self.count += 1
-            self._orig(code, what)
-
-        native._check = counting
-        return self
-
-    def __exit__(self, *exc):
-        self._native._check = self._orig
-
-
-class GpuModelRunner:
+class GpuModelRunner(LaneRunner):
     def __init__(self, weights: DeviceWeights, *, context_capacity: int, lanes: int = 1, stripe: int = 64, comm: str | None = None,
                  group=None, prefill_chunk: int = 512, use_graphs: bool | None = None, wait_limit: int | None = None,
                  staging_bytes: int | None = None, kv_layout: str = "auto", replica_budget_bytes: int = 32 << 30,
@@ -149,15 +110,8 @@ class GpuModelRunner:
                 elif decode_path != "auto":
                     raise ValueError(f"the fused decode phases do not take this configuration (code {mega.supported_code})")
             self.decode_path = ("mega" if self.mega.mode == "persistent" else "phases") if self.mega is not None else "kernels"
-            self.prefill_ws = None
-            self._prefill_out = torch.zeros(1, dtype=torch.int32, device=self.device)
-            self._graph = None
-            self._graph_stream = torch.cuda.Stream(device=self.device)
+        self._ready()
         self.report.phases["allocate"] = time.perf_counter() - t0
-        self.decode_launches = 0
-        self.steps_issued = 0
-        self._feed_host = None
-        self.fed_bytes_per_step = 0
 
     # ------------------------------------------------------------------ admission
     def _project(self, weight_bytes: int, staging_bytes: int, *, already_resident: int, mem_info=None) -> dict:
@@ -175,127 +129,31 @@ class GpuModelRunner:
 
     # ------------------------------------------------------------------ decode program
     def _decode_body(self) -> None:
-        st, ws, m = self.state, self.decode_ws, self.model
         if self.mega is not None:
             self.mega.step()
             return
-        logits = m.run_rows(ws, st, st.tokens, st.positions, st.lane_ids, st.active, self.lanes, decode=True,
-                            max_ctx=self.cache.context_capacity, head="argmax")
-        m.sample(ws, st, logits, self.lanes, st.active, advance=3)
+        super()._decode_body()
 
-    def build_decode_program(self) -> ProgramRecord:
-        """Warm up eagerly (lanes inactive: no cache write, no advance), then capture the step in a CUDA graph."""
-        t0 = time.perf_counter()
-        with torch.cuda.device(self.device):
-            saved = self.state.active.clone()
-            self.state.active.zero_()
-            with _LaunchCounter() as counter, native.record_exchanges() as plan:
-                self._decode_body()
-            self.decode_launches = counter.count
-            # the cross-GPU exchanges of the step, in launch order, against the rules the in-kernel protocol rests on (alternating
-            # all-reduce channels, a signal at most once between two all-reduces, payloads within the slots): refused before capture
-            check_collective_plan(plan, world=self.peer.world)
-            self.report.phases["collective_plan"] = {"exchanges": len(plan), "allreduces": sum(1 for op in plan if op["kind"] == "allreduce")}
+    def _captures_graphs(self) -> bool:
+        return self.use_graphs and (self.model.comm_mode == "fused" or self.world == 1)
+
+    def _capture_decode(self) -> torch.cuda.CUDAGraph:
+        try:
+            return super()._capture_decode()
+        except RuntimeError:
+            if self.mega is None:
+                raise
+            # a driver that will not record a cooperative launch: the same grid as an ordinary launch (it fits the GPU
+            # and nothing else runs beside it, so every CTA is resident all the same)
             torch.cuda.synchronize(self.device)
-            kind = "eager"
-            if self.use_graphs and self.model.comm_mode == "fused" or (self.use_graphs and self.world == 1):  # noqa: E129
-                try:
-                    graph = torch.cuda.CUDAGraph()
-                    with torch.cuda.graph(graph, stream=self._graph_stream):
-                        self._decode_body()
-                except RuntimeError:
-                    if self.mega is None:
-                        raise
-                    # a driver that will not record a cooperative launch: the same grid as an ordinary launch (it fits the GPU
-                    # and nothing else runs beside it, so every CTA is resident all the same)
-                    torch.cuda.synchronize(self.device)
-                    native.set_mega_cooperative(0)
-                    self.report.phases["mega_cooperative_capture"] = "refused: ordinary launch"
-                    graph = torch.cuda.CUDAGraph()
-                    with torch.cuda.graph(graph, stream=self._graph_stream):
-                        self._decode_body()
-                self._graph = graph
-                kind = "cuda_graph"
-            self.state.active.copy_(saved)
-            self.state.step_counter.zero_()
-            self.steps_issued = 0
-            torch.cuda.synchronize(self.device)
-            self.peer.check_status()
-        rec = ProgramRecord("decode:" + self.decode_path, kind, self.lanes, self.decode_launches, time.perf_counter() - t0)
-        self.report.programs.append(rec)
-        return rec
-
-    def decode_step(self) -> None:
-        """Enqueue one decode step for every active lane (asynchronous)."""
-        if self._graph is None and not self.report.programs:
-            self.build_decode_program()
-        if self._graph is not None:
-            self._graph.replay()
-        else:
-            self._decode_body()
-        self.steps_issued += 1
-
-    def feed_tokens(self, tokens: dict) -> None:
-        """Copy the committed tokens of the given lanes (``lane -> token``) from pinned host memory into the device's token
-        registers (asynchronous, on the current stream: the next decode step reads them).  4 bytes per lane; a lane that is not
-        named keeps being fed what it was fed last, which a frozen lane never uses."""
-        if self._feed_host is None:
-            self._feed_host = torch.zeros(self.lanes, dtype=torch.int32).pin_memory()
-        for lane, token in tokens.items():
-            self._feed_host[lane] = int(token)
-        with torch.cuda.device(self.device):
-            self.state.tokens.copy_(self._feed_host, non_blocking=True)
-        self.fed_bytes_per_step = 4 * self.lanes
-
-    def read_last_tokens(self) -> list[int]:
-        """Tokens of the most recent decode step, one per lane (-1 for a frozen lane).  Synchronizes."""
-        return self.read_step_tokens(self.steps_issued - 1)
-
-    def read_status(self) -> int:
-        """The device status word (0 = clean); reading clears it."""
-        return self.peer.read_status()
-
-    def read_step_tokens(self, step_index: int) -> list[int]:
-        """Tokens produced by decode step ``step_index`` (synchronizes; one small D2H copy)."""
-        row = self.state.out_tokens[step_index % RING].cpu()
-        return [int(v) for v in row]
+            native.set_mega_cooperative(0)
+            self.report.phases["mega_cooperative_capture"] = "refused: ordinary launch"
+            return super()._capture_decode()
 
     # ------------------------------------------------------------------ prefill program
-    def _ensure_prefill_ws(self) -> Workspace:
-        if self.prefill_ws is None:
-            with torch.cuda.device(self.device):
-                self.prefill_ws = Workspace(self.model, self.prefill_chunk, "prefill", attn_rows=min(self.prefill_chunk, 64),
-                                            score_stride=self.cache.context_capacity, peer_visible=False)
-        return self.prefill_ws
-
-    def prefill(self, lane: int, token_ids) -> int:
-        """Run a prompt through ``lane`` with a fresh cache; returns the first generated token.
-
-        After the call the lane is active, its position is ``len(token_ids)`` and its next input is that token.
-        """
-        n = len(token_ids)
-        if not 0 < n < self.cache.context_capacity:
-            raise ValueError("prompt does not fit the context capacity")
-        ws = self._ensure_prefill_ws()
-        st, m = self.state, self.model
-        with torch.cuda.device(self.device):
-            ids = torch.as_tensor(list(token_ids), dtype=torch.int32).pin_memory().to(self.device, non_blocking=True)
-            lane_t = torch.full((self.prefill_chunk,), lane, dtype=torch.int32, device=self.device)
-            st.reset_lane(lane)
-            logits = None
-            for start in range(0, n, self.prefill_chunk):
-                rows = min(self.prefill_chunk, n - start)
-                pos = torch.arange(start, start + rows, dtype=torch.int32, device=self.device)
-                last = start + rows == n
-                logits = m.run_rows(ws, st, ids[start : start + rows], pos, lane_t, None, rows, decode=False, max_ctx=start + rows,
-                                    head_rows=slice(rows - 1, rows) if last else slice(0, 1), lane_of_rows=lane)
-            m.sample(ws, st, logits, 1, None, advance=1, tokens_out=st.tokens[lane : lane + 1], positions=st.positions[lane : lane + 1],
-                     out=self._prefill_out)
-            st.positions[lane] = n
-            st.active[lane] = 1
-            token = int(self._prefill_out.cpu()[0])
-            self.peer.check_status()
-        return token
+    def _prefill_workspace(self) -> Workspace:
+        return Workspace(self.model, self.prefill_chunk, "prefill", attn_rows=min(self.prefill_chunk, 64),
+                         score_stride=self.cache.context_capacity, peer_visible=False)
 
     def memory_stats(self) -> dict:
         """Device memory as the allocator and the driver see it, plus what this runner knows it holds (per-request records)."""
@@ -331,20 +189,15 @@ class GpuModelRunner:
             st.active[lane] = 1
             torch.cuda.synchronize(self.device)
 
-    def deactivate(self, lane: int) -> None:
-        self.state.active[lane] = 0
-
-    def close(self) -> None:
-        self._graph = None
-        if self.peer.world > 1:
-            torch.cuda.synchronize(self.device)
-            self.peer.check_canaries()  # a kernel (of any rank) that overran a staging region wrote into its guard band
-        self.peer.close()
-
-
 def build_runner(geometry, *, world: int = 1, rank: int = 0, device=None, checkpoint=None, seed: int = 0, expert_split: str | None = None,
-                 **kwargs) -> GpuModelRunner:
-    """Convenience constructor: shard ``checkpoint`` (a runtime-layout mapping) or random-init on the device."""
+                 **kwargs) -> LaneRunner:
+    """Convenience constructor: shard ``checkpoint`` (a runtime-layout mapping) or random-init on the device.  The geometry says which
+    model family it is."""
+    from glm_tpu_b200.models import registry
+
+    family = registry.family_of(geometry)
+    if family.name != registry.GLM.name:
+        return family.build_runner(geometry, world=world, rank=rank, device=device, checkpoint=checkpoint, seed=seed, **kwargs)
     from glm_tpu_b200.models.glm_moe_dsa.weights import random_device_weights, shard_checkpoint
 
     device = torch.device(device if device is not None else f"cuda:{torch.cuda.current_device()}")

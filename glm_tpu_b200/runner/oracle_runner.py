@@ -1,7 +1,7 @@
 """A CPU runner built on the contract oracle: the engine's reference backend.
 
 It has the interface of ``GpuModelRunner`` (``prefill`` / ``decode_step`` / ``read_last_tokens`` / ``read_status`` /
-``deactivate``) but recomputes the whole sequence through ``oracle.contract.forward`` at every step.  It is the timed
+``deactivate``) but recomputes the whole sequence through the model family's oracle at every step.  It is the timed
 CPU baseline for small models, the backend of the CPU end-to-end tests of the worker, the controller and the servers,
 and an independent check of the incremental GPU runner (same tokens on the same checkpoint, up to near-ties).
 """
@@ -10,13 +10,13 @@ from __future__ import annotations
 
 from types import SimpleNamespace
 
-from glm_tpu_b200.oracle import contract
+from glm_tpu_b200.models import registry
 
 
 class OracleRunner:
     def __init__(self, geometry, checkpoint, *, context_capacity: int, lanes: int = 1):
         self.g = geometry
-        self.weights = contract.OracleWeights.from_checkpoint(geometry, checkpoint)
+        self._next_token = registry.family_of(geometry).next_token(geometry, checkpoint, context_capacity)
         self.cache = SimpleNamespace(context_capacity=context_capacity)
         self.lanes = lanes
         self.world, self.rank = 1, 0
@@ -27,8 +27,7 @@ class OracleRunner:
         self.steps_issued = 0
 
     def _next(self, lane: int) -> int:
-        trace = contract.forward(self.weights, self.sequences[lane], capacity=self.cache.context_capacity)
-        return int(trace.tokens[-1])
+        return self._next_token(self.sequences[lane])
 
     def prefill(self, lane: int, token_ids) -> int:
         if not 0 < len(token_ids) < self.cache.context_capacity:

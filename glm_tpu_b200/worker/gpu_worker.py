@@ -30,6 +30,8 @@ from glm_tpu_b200.engine import resident_protocol as proto
 from glm_tpu_b200.engine.llm_engine import LLMEngine
 from glm_tpu_b200.engine.outputs import final_channel
 from glm_tpu_b200.engine.request_session import LocalVote, fleet_vote
+from glm_tpu_b200.models import registry
+from glm_tpu_b200.models.registry import resolve_model  # noqa: F401 - the front ends resolve models through the worker
 from glm_tpu_b200.utils.io_utils import persist_json
 
 
@@ -39,7 +41,7 @@ def parse_args(argv=None):
     ap.add_argument("--request", help="prepared request or batch (JSON file); optional with --keep-loaded")
     ap.add_argument("--request-sha256", help="expected request_sha256 of --request")
     ap.add_argument("--keep-loaded", action="store_true")
-    ap.add_argument("--model", default="random:tiny", help="random:<tiny|small|glm53>[:layers] or a packed checkpoint directory")
+    ap.add_argument("--model", default="random:tiny", help="random:<tiny|small|glm53|namizen-tiny>[:layers], a packed checkpoint directory, or a directory with config.json and safetensors")
     ap.add_argument("--backend", default="gpu", choices=["gpu", "oracle"], help="'oracle' runs the CPU contract reference")
     ap.add_argument("--context", type=int, default=0, help="context capacity (0: the request's)")
     ap.add_argument("--lanes", type=int, default=1)
@@ -121,29 +123,15 @@ def preflight(args) -> dict:
     return payload
 
 
-def resolve_model(spec: str):
-    """``(geometry, source)``: source is ('random', seed-less) or ('checkpoint', Path)."""
-    from glm_tpu_b200.config import model as mc
-
-    if spec.startswith("random:"):
-        parts = spec.split(":")
-        base = {"tiny": mc.tiny_geometry, "small": mc.small_geometry, "glm53": mc.glm53_geometry}[parts[1]]()
-        if len(parts) > 2:
-            base = base.truncated(int(parts[2]))
-        return base, ("random", None)
-    path = Path(spec)
-    from glm_tpu_b200.model_loader.sharded_state import loader
-
-    return loader.read_geometry(path), ("checkpoint", path)
-
-
 def profile_for(geometry, capacity: int, tokenizer=None) -> request_schema.RequestProfile:
     from glm_tpu_b200.config import model as mc
 
-    if geometry.vocab_size == mc.glm53_geometry().vocab_size:
+    family = registry.family_of(geometry)
+    if family is registry.GLM and geometry.vocab_size == mc.glm53_geometry().vocab_size:
         return request_schema.GLM53_PROFILE
     caps = tuple(sorted({capacity}))
-    return request_schema.RequestProfile.for_geometry(geometry, caps, concurrent_capacity=capacity)
+    identity = {} if family is registry.GLM else {"model_id": family.architecture, "model_revision": geometry.geometry_hash}
+    return request_schema.RequestProfile.for_geometry(geometry, caps, concurrent_capacity=capacity, **identity)
 
 
 # ------------------------------------------------------------------------------------------------ worker
@@ -230,38 +218,32 @@ class Worker:
         geometry, (kind, path) = resolve_model(self.args.model)
         capacity = self.args.context or (self.payload or {}).get("context_capacity") or request_schema.CAPACITY
         lanes = max(self.args.lanes, len(self.payload["requests"]) if self.payload and request_schema.is_concurrent(self.payload) else 1)
+        family = registry.family_of(geometry)
+        if self.world > 1 and not family.multi_gpu:
+            raise SystemExit(f"{family.architecture} runs on one GPU, the fleet has {self.world} ranks")
         if self.args.backend == "oracle":
-            from glm_tpu_b200.models.glm_moe_dsa.weights import random_checkpoint
             from glm_tpu_b200.runner.oracle_runner import OracleRunner
 
-            if kind != "random":
-                from glm_tpu_b200.model_loader.sharded_state import loader
-
-                checkpoint = loader.load_full_checkpoint(path)
-            else:
-                checkpoint = random_checkpoint(geometry, seed=self.args.seed)
+            checkpoint = family.load_full_checkpoint(path) if kind == "checkpoint" else family.random_checkpoint(geometry, seed=self.args.seed)
             runner = OracleRunner(geometry, checkpoint, context_capacity=capacity, lanes=lanes)
         else:
             import torch
 
             from glm_tpu_b200.csrc.build import build
+            from glm_tpu_b200.ops import native
             from glm_tpu_b200.runner.gpu_runner import build_runner
 
             if self.rank == 0:
-                build()
+                native.select_library(build(component=family.library_component))
             self.vote.all(True, "library_built")
             device = torch.device("cuda", self.local_rank)
             checkpoint = None
             if kind == "checkpoint":
-                from glm_tpu_b200.model_loader.sharded_state import loader
-
                 # the site's pins travel with the load: another packed checkpoint than the pinned one is refused here
-                checkpoint = loader.load_rank_checkpoint(path, self.rank, self.world, pins=self.launch["pins"], device=device)
+                checkpoint = family.load_checkpoint(path, self.rank, self.world, pins=self.launch["pins"], device=device)
                 self.record["checkpoint_pins"] = {k: v for k, v in (self.launch["pins"] or {}).items() if v}
-            elif geometry.num_layers <= 8 and geometry.hidden_size <= 1024:
-                from glm_tpu_b200.models.glm_moe_dsa.weights import random_checkpoint
-
-                checkpoint = random_checkpoint(geometry, seed=self.args.seed)  # fixtures: the same bits as the oracle
+            elif family.small_enough_for_host(geometry):
+                checkpoint = family.random_checkpoint(geometry, seed=self.args.seed)  # fixtures: the same bits as the oracle
             stripe = 64 if capacity % (64 * self.world) == 0 else max(1, capacity // (8 * self.world))
             runner = build_runner(geometry, world=self.world, rank=self.rank, device=device, checkpoint=checkpoint, seed=self.args.seed,
                                   context_capacity=capacity, lanes=lanes, comm=self.args.comm, kv_layout=self.args.kv_layout,
@@ -272,16 +254,21 @@ class Worker:
         self.profile = profile_for(geometry, capacity)
         self.engine = LLMEngine(runner, vote=self.vote, profile=self.profile, digest_consensus=self.digest_consensus)
         self.record["geometry_hash"] = geometry.geometry_hash
-        from glm_tpu_b200.config.parallel import ParallelLayout
-
-        model = getattr(runner, "model", None)  # which tensor is split how: must agree on every rank
-        layout_hash = (model.layout if model is not None else ParallelLayout(geometry, self.world, self.rank)).layout_hash
+        layout_hash = self.layout_hash(geometry, getattr(runner, "model", None), family)
         self.record["layout_hash"] = layout_hash
         self.vote.all(self.digest_consensus(layout_hash), "layout_agreed")
         self.record["context_capacity"] = capacity
         self.record["kv_layout"] = getattr(runner, "kv_layout", None)
         self.record["memory_admission"] = getattr(getattr(runner, "report", None), "memory", None)
         return runner
+
+    def layout_hash(self, geometry, model, family) -> str:
+        """Which tensor is split how: must agree on every rank.  A one-GPU family splits nothing: its geometry is the layout."""
+        if not family.multi_gpu:
+            return geometry.geometry_hash
+        from glm_tpu_b200.config.parallel import ParallelLayout
+
+        return (model.layout if model is not None else ParallelLayout(geometry, self.world, self.rank)).layout_hash
 
     def build_programs(self, runner):
         rec = runner.build_decode_program()
