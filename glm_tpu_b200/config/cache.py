@@ -138,7 +138,8 @@ class RingCacheConfig:
     Every layer has its own ring of key and value rows per lane: position ``p`` lives in slot ``p % ring(layer)``.  A layer that attends
     inside chunks of ``chunk`` positions needs the rows of the current chunk only, so its ring has ``min(chunk, capacity)`` slots whatever
     the context capacity; a layer that sees the whole sequence has one slot per position.  A layer with a short convolution over time also
-    keeps the last ``taps - 1`` projected rows of every lane.  Head rows are padded to a multiple of 8 elements (16-byte vectors).
+    keeps the last ``taps - 1`` projected rows of every lane.  Head rows are padded to a multiple of 16 elements (whole tensor-core
+    steps, 16-byte vectors).
 
     ``geometry.layers[i].mixer`` gives a layer's ``kv_heads``, ``dim``, ``vdim``, ``chunk``, ``conv`` and ``qkv_width``.
     """
@@ -169,20 +170,24 @@ class RingCacheConfig:
         """The first position that ``position`` can see."""
         return position // self.chunk(layer) * self.chunk(layer)
 
-    def ring_from(self, layer: int, start: int, rows: int) -> tuple[int, bool]:
-        """Which rows of a step ``start .. start + rows - 1`` the ring keeps: ``(first row, only afterwards)``.  The rows of the last
-        chunk are kept.  When that chunk began inside the step, its slots may still hold keys that earlier rows of the step see, so the
-        rows go in after the attention has read them."""
-        keep = self.first_position(layer, start + rows - 1)
-        return max(keep - start, 0), keep > start
+    def crossing(self, layer: int, start: int, rows: int) -> tuple[int, int] | None:
+        """``None`` if the rows ``start .. start + rows - 1`` of a step lie in one chunk: they enter the ring right away and the ring then
+        holds every key they see, in order.  Otherwise ``(before, after)``: the ring's first ``before`` rows (the beginning of the first
+        row's chunk) are still needed by the step, and its last ``after`` rows (the last row's chunk) take their places afterwards."""
+        first, last = self.first_position(layer, start), self.first_position(layer, start + rows - 1)
+        return None if first == last else (start - first, start + rows - last)
+
+    def linear_rows(self, layer: int, rows: int) -> int:
+        """Rows of the linear key / value buffer a step of up to ``rows`` rows may need (0: its chunk is never crossed)."""
+        return 0 if self.chunk(layer) >= self.context_capacity else self.chunk(layer) - 1 + rows
 
     def k_shape(self, layer: int) -> tuple[int, int, int, int]:
         m = self._mixer(layer)
-        return (self.lanes, self.ring(layer), m.kv_heads, -(-m.dim // 8) * 8)
+        return (self.lanes, self.ring(layer), m.kv_heads, -(-m.dim // 16) * 16)
 
     def v_shape(self, layer: int) -> tuple[int, int, int, int]:
         m = self._mixer(layer)
-        return (self.lanes, self.ring(layer), m.kv_heads, -(-m.vdim // 8) * 8)
+        return (self.lanes, self.ring(layer), m.kv_heads, -(-m.vdim // 16) * 16)
 
     def conv_shape(self, layer: int) -> tuple[int, int, int]:
         m = self._mixer(layer)

@@ -23,7 +23,7 @@ OBJ_DIR = CSRC / "build"
 NVCC = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
 # sources each model family needs when the complete library has not been built
 COMPONENTS = {
-    "namizen": ("parallel_block", "qkv_conv", "chunk_attention", "gemm_f32", "swiglu_rows", "gemv", "gemm_tcgen05", "misc", "peer_registry"),
+    "namizen": ("parallel_block", "qkv_conv", "chunk_attention", "chunk_attention_tcgen05", "gemm_f32", "swiglu_rows", "gemv", "gemm_tcgen05", "misc", "peer_registry"),
 }
 FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",

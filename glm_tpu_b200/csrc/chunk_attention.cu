@@ -3,38 +3,29 @@
 //   query i sees key j  <=>  j <= i and j / chunk == i / chunk          (chunks counted from position 0 of the sequence)
 //   out_i = sum_j exp(s_ij) v_j / (exp(sink_h) + sum_j exp(s_ij)),       s_ij = scale * q_i . k_j
 //
-// Keys live in the lane's ring (slot = position mod ring, ring >= min(chunk, capacity): a ring holds the whole current chunk) and, for the
-// rows of a prefill step, in linear buffers whose row 0 is position `start`.  Scores, exponentials and sums are fp32; the weights enter
-// the product with the values as two bf16 pieces (value and remainder), so they keep 16 bits of mantissa.
+// Prefill: the rows are consecutive positions of one sequence and every key they can see lies in linear buffers whose row 0 is position
+// `base` (the lane's ring itself, or a copy of its current chunk followed by the step's rows).  Decode: one row per lane, the keys are in
+// the lane's ring (slot = position mod ring; a ring holds a whole chunk, so the current chunk starts at slot 0).  Scores, exponentials and
+// sums are fp32; the weights enter the product with the values as two bf16 pieces (value and remainder): 16 bits of mantissa.
 //
-//   chunk_attn_prefill_kernel  bf16, many rows of one sequence: 64 query rows of one head per CTA, mma.sync, cp.async double buffer
-//   chunk_attn_decode_kernel   bf16, one row per lane: up to 16 query heads of one key head per cluster; the keys are dealt to the warps of
-//                              the cluster's CTAs, the partial softmax states meet in distributed shared memory
-//   chunk_attn_any_kernel      any head size and element type, one CTA per (row, head): the 32-bit path and head sizes beyond 256
+//   chunk_attn_tc_kernel       prefill, bf16, head sizes up to 128: tcgen05, see chunk_attention_tcgen05.cu
+//   chunk_attn_prefill_kernel  prefill, bf16, head sizes up to 256: 64 query rows of one head per CTA, mma.sync, cp.async double buffer
+//   chunk_attn_decode_kernel   decode, bf16, head sizes up to 256: up to 16 query heads of one key head per cluster; key tiles come in by
+//                              TMA and are dealt to the cluster's CTAs, the partial softmax states meet in distributed shared memory
+//   chunk_attn_any_kernel      any head size and element type, one CTA per (row, head): the 32-bit path and larger heads
 //
 // The running maximum starts at the sink and the sum gets the sink's term once; the sink has no value.
 #include <cooperative_groups.h>
 
 #include "attention_core.cuh"
+#include "chunk_attention.cuh"
 #include "common.cuh"
+#include "tcgen05.cuh"
 #include "vec8.cuh"
 
 namespace cg = cooperative_groups;
 
-struct ChunkAttnArgs {
-    const void* q;                            // [rows, H, dimp]
-    const void *k_new, *v_new;                // [rows, G, dimp], [rows, G, vdimp]; NULL: every key is in the ring (decode)
-    const void *k_ring, *v_ring;              // [lanes, ring, G, dimp], [lanes, ring, G, vdimp]
-    const float* sink;                        // [H], or NULL: no sink
-    const int *row_pos, *row_lane, *row_active;  // row_active may be NULL
-    void* out; int64_t out_stride;            // [rows, H * vdim (+ more)]
-    int rows, H, G, dim, dimp, vdim, vdimp;
-    int chunk, ring, capacity, lanes;
-    float scale;
-    uint32_t* status;
-};
-
-#define CA_LOG2E 1.4426950408889634f
+#define CA_LOG2E 1.4426950408889634f  // log2(e)
 
 __device__ __forceinline__ int ca_lane(const ChunkAttnArgs& a, int row) {
     const int lane = a.row_lane[row];
@@ -76,7 +67,7 @@ template <int DV>
 __global__ void __launch_bounds__(CP_THREADS) chunk_attn_prefill_kernel(ChunkAttnArgs a) {
     GLMB_PDL_PROLOGUE();
     extern __shared__ __align__(16) unsigned char smem_raw[];
-    const int dk = (a.dim + 15) & ~15, dv = (a.vdim + 15) & ~15;
+    const int dk = a.dimp, dv = a.vdimp;
     const int KP = dk + 8, VP = dv + 8;  // padded rows (elements): 16-byte aligned, banks staggered for ldmatrix
     bf16* q_s = reinterpret_cast<bf16*>(smem_raw);
     bf16* k_s = q_s + CP_ROWS * KP;
@@ -84,38 +75,33 @@ __global__ void __launch_bounds__(CP_THREADS) chunk_attn_prefill_kernel(ChunkAtt
     const int head = blockIdx.y, group = head / (a.H / a.G);
     const int r0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * CP_ROWS;  // the rows with most keys (towards a chunk's end) first
     const int nrows = min(CP_ROWS, a.rows - r0);
-    const int start = ca_pos(a, 0), lane_id = ca_lane(a, 0);
-    const int first = start + r0, last = min(start + r0 + nrows, a.capacity) - 1;
+    const int first = a.start + r0, last = first + nrows - 1;
     const int key0 = first / a.chunk * a.chunk;
     const int tiles = max((last - key0) / CP_KEYS + 1, 1);
-    const bf16* k_new = reinterpret_cast<const bf16*>(a.k_new) + (int64_t)group * a.dimp;
-    const bf16* v_new = reinterpret_cast<const bf16*>(a.v_new) + (int64_t)group * a.vdimp;
-    const bf16* k_ring = reinterpret_cast<const bf16*>(a.k_ring) + ((int64_t)lane_id * a.ring * a.G + group) * a.dimp;
-    const bf16* v_ring = reinterpret_cast<const bf16*>(a.v_ring) + ((int64_t)lane_id * a.ring * a.G + group) * a.vdimp;
+    const bf16* k_head = reinterpret_cast<const bf16*>(a.k) + (int64_t)group * a.dimp;
+    const bf16* v_head = reinterpret_cast<const bf16*>(a.v) + (int64_t)group * a.vdimp;
     const int tid = threadIdx.x;
 
-    auto load_rows = [&](bf16* dst, int stride, int pieces, const bf16* fresh, const bf16* ring, int padded, int key_base) {
-        const int have = padded / 8;
+    auto load_rows = [&](bf16* dst, int stride, int pieces, const bf16* src, int padded, int key_base) {
         for (int i = tid; i < CP_KEYS * pieces; i += CP_THREADS) {
             const int r = i / pieces, c = i % pieces, key = key_base + r;
             bf16* d = dst + r * stride + c * 8;
-            if (key > last || c >= have) { *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0); continue; }
-            const bf16* src = key >= start ? fresh + (int64_t)(key - start) * a.G * padded : ring + (int64_t)(key % a.ring) * a.G * padded;
-            cp_async16(d, src + c * 8);
+            if (key > last) *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
+            else cp_async16(d, src + (int64_t)(key - a.base) * a.G * padded + c * 8);
         }
     };
     auto load_tile = [&](int t) {
-        load_rows(k_s + (t & 1) * CP_KEYS * KP, KP, dk / 8, k_new, k_ring, a.dimp, key0 + t * CP_KEYS);
-        load_rows(v_s + (t & 1) * CP_KEYS * VP, VP, dv / 8, v_new, v_ring, a.vdimp, key0 + t * CP_KEYS);
+        load_rows(k_s + (t & 1) * CP_KEYS * KP, KP, dk / 8, k_head, a.dimp, key0 + t * CP_KEYS);
+        load_rows(v_s + (t & 1) * CP_KEYS * VP, VP, dv / 8, v_head, a.vdimp, key0 + t * CP_KEYS);
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     {
         const bf16* q = reinterpret_cast<const bf16*>(a.q) + ((int64_t)r0 * a.H + head) * a.dimp;
-        const int pieces = dk / 8, have = a.dimp / 8;
+        const int pieces = dk / 8;
         for (int i = tid; i < CP_ROWS * pieces; i += CP_THREADS) {
             const int r = i / pieces, c = i % pieces;
             bf16* d = q_s + r * KP + c * 8;
-            if (r < nrows && c < have) cp_async16(d, q + (int64_t)r * a.H * a.dimp + c * 8);
+            if (r < nrows) cp_async16(d, q + (int64_t)r * a.H * a.dimp + c * 8);
             else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
         }
     }
@@ -239,66 +225,68 @@ __global__ void __launch_bounds__(CP_THREADS) chunk_attn_prefill_kernel(ChunkAtt
 #define CD_WARPS 4
 #define CD_THREADS (CD_WARPS * 32)
 #define CD_HEADS 16
-#define CD_KEYS 16  // keys a warp takes at a time
+#define CD_KEYS 64  // keys of a tile, 16 per warp
+#define CD_BOX (CD_KEYS * 128)  // bytes of a tile's 64-column box: 128-byte rows, 128-byte swizzle
 
+static inline int cd_boxes(int padded) { return (padded + 63) / 64; }
 static inline size_t chunk_decode_smem(int dk, int dv, int stages) {
-    const size_t stage = (size_t)CD_WARPS * stages * CD_KEYS * (dk + 8 + dv + 8) * 2, merge = (size_t)CD_WARPS * CD_HEADS * dv * 4;
-    return (size_t)CD_HEADS * (dk + 8) * 2 + (stage > merge ? stage : merge);
+    const size_t tiles = (size_t)stages * (cd_boxes(dk) + cd_boxes(dv)) * CD_BOX, merge = (size_t)CD_WARPS * CD_HEADS * dv * 4;
+    return 1024 + (tiles > merge ? tiles : merge) + (size_t)CD_HEADS * (dk + 8) * 2;
+}
+// 16-byte piece `c` of row `r` of a swizzled tile made of 64-column boxes
+__device__ __forceinline__ const unsigned char* cd_piece(const unsigned char* tile, int r, int c) {
+    return tile + (c >> 3) * CD_BOX + r * 128 + (((c & 7) ^ (r & 7)) << 4);
 }
 
 // grid (splits, key heads x blocks of 16 query heads, rows), cluster (splits, 1, 1).
 template <int DV>
-__global__ void __launch_bounds__(CD_THREADS) chunk_attn_decode_kernel(ChunkAttnArgs a, int stages) {
-    GLMB_PDL_PROLOGUE();
+__global__ void __launch_bounds__(CD_THREADS)
+chunk_attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, ChunkAttnArgs a, int stages) {
     cg::cluster_group cluster = cg::this_cluster();
-    extern __shared__ __align__(16) unsigned char smem_raw[];
+    extern __shared__ unsigned char smem_raw[];
     __shared__ float ml_s[CD_WARPS][CD_HEADS][2];  // (maximum, sum) per warp
     __shared__ float cta_ml[CD_HEADS][2];
-    const int dk = (a.dim + 15) & ~15, dv = (a.vdim + 15) & ~15, KP = dk + 8, VP = dv + 8;
+    __shared__ __align__(8) uint64_t full_bar[4];
+    const int dk = a.dimp, dv = a.vdimp, KP = dk + 8;
+    const int kboxes = (dk + 63) / 64, vboxes = (dv + 63) / 64;
+    unsigned char* tiles_s = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
+    const size_t stage_bytes = (size_t)(kboxes + vboxes) * CD_BOX;
+    const size_t tile_area = stages * stage_bytes, merge_area = (size_t)CD_WARPS * CD_HEADS * dv * 4;
+    bf16* q_s = reinterpret_cast<bf16*>(tiles_s + (tile_area > merge_area ? tile_area : merge_area));
+    if (threadIdx.x == 0) {
+        for (int s = 0; s < stages; ++s) mbar_init(full_bar + s, 1);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    __syncthreads();
+    GLMB_PDL_PROLOGUE();
     const int per = a.H / a.G, head_blocks = (per + CD_HEADS - 1) / CD_HEADS;
     const int group = blockIdx.y / head_blocks, h0 = group * per + (blockIdx.y % head_blocks) * CD_HEADS;
     const int heads = min(CD_HEADS, group * per + per - h0);
     const int row = blockIdx.z, split = blockIdx.x, splits = gridDim.x;
     const bool active = !a.row_active || a.row_active[row] != 0;
     const int pos = ca_pos(a, row), lane_id = ca_lane(a, row);
-    const int key0 = pos / a.chunk * a.chunk;
-    const int keys = active ? pos - key0 + 1 : 0;
-    bf16* q_s = reinterpret_cast<bf16*>(smem_raw);
-    unsigned char* rest = smem_raw + (size_t)CD_HEADS * KP * 2;
+    const int keys = active ? pos % a.chunk + 1 : 0;  // slots 0 .. keys - 1 of the lane's ring
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3, mr = lane & 7, mi = lane >> 3;
-    bf16* kv_s = reinterpret_cast<bf16*>(rest) + (size_t)warp * stages * CD_KEYS * (KP + VP);
-    const bf16* k_ring = reinterpret_cast<const bf16*>(a.k_ring) + ((int64_t)lane_id * a.ring * a.G + group) * a.dimp;
-    const bf16* v_ring = reinterpret_cast<const bf16*>(a.v_ring) + ((int64_t)lane_id * a.ring * a.G + group) * a.vdimp;
+    const int tiles = (keys + CD_KEYS - 1) / CD_KEYS, mine = tiles > split ? (tiles - split - 1) / splits + 1 : 0;  // tiles split, split + splits, ..
 
-    const int blocks = (keys + CD_KEYS - 1) / CD_KEYS, stride = splits * CD_WARPS, b0 = split * CD_WARPS + warp;
-    auto load_block = [&](int b, int stage) {  // 16 keys and values of this warp
-        if (b < blocks) {
-            bf16* kd = kv_s + (size_t)stage * CD_KEYS * (KP + VP);
-            bf16* vd = kd + CD_KEYS * KP;
-            const int kp = dk / 8, vp = dv / 8, key_base = key0 + b * CD_KEYS;
-            for (int i = lane; i < CD_KEYS * (kp + vp); i += 32) {
-                const int r = i / (kp + vp), c = i % (kp + vp), key = key_base + r;
-                const bool is_k = c < kp;
-                const int col = is_k ? c : c - kp, have = (is_k ? a.dimp : a.vdimp) / 8;
-                bf16* d = is_k ? kd + r * KP + col * 8 : vd + r * VP + col * 8;
-                if (key > pos || col >= have) { *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0); continue; }
-                const int64_t slot = (int64_t)(key % a.ring) * a.G;
-                cp_async16(d, is_k ? k_ring + slot * a.dimp + col * 8 : v_ring + slot * a.vdimp + col * 8);
-            }
-        }
-        asm volatile("cp.async.commit_group;" ::: "memory");
+    auto load_tile = [&](int i) {  // the i-th tile of this CTA, by one thread
+        unsigned char* dst = tiles_s + (size_t)(i % stages) * stage_bytes;
+        uint64_t* bar = full_bar + i % stages;
+        const int y = lane_id * a.ring + (split + i * splits) * CD_KEYS;
+        mbar_expect_tx(bar, (uint32_t)stage_bytes);
+        for (int b = 0; b < kboxes; ++b) tma_load_2d(dst + b * CD_BOX, &map_k, bar, group * dk + b * 64, y);
+        for (int b = 0; b < vboxes; ++b) tma_load_2d(dst + (kboxes + b) * CD_BOX, &map_v, bar, group * dv + b * 64, y);
     };
+    if (threadIdx.x == 0)
+        for (int i = 0; i < min(stages, mine); ++i) load_tile(i);
     {
-        const bf16* q = reinterpret_cast<const bf16*>(a.q) + ((int64_t)row * a.H + h0) * a.dimp;
-        const int pieces = dk / 8, have = a.dimp / 8;
+        const bf16* q = reinterpret_cast<const bf16*>(a.q) + ((int64_t)row * a.H + h0) * dk;
+        const int pieces = dk / 8;
         for (int i = threadIdx.x; i < CD_HEADS * pieces; i += CD_THREADS) {
             const int r = i / pieces, c = i % pieces;
-            uint4 v = make_uint4(0, 0, 0, 0);
-            if (r < heads && c < have) v = *reinterpret_cast<const uint4*>(q + (int64_t)r * a.dimp + c * 8);
-            *reinterpret_cast<uint4*>(q_s + r * KP + c * 8) = v;
+            *reinterpret_cast<uint4*>(q_s + r * KP + c * 8) = r < heads ? *reinterpret_cast<const uint4*>(q + (int64_t)r * dk + c * 8) : make_uint4(0, 0, 0, 0);
         }
     }
-    for (int s = 0; s < stages - 1; ++s) load_block(b0 + s * stride, s);
     __syncthreads();
 
     const float scale2 = a.scale * CA_LOG2E;
@@ -307,82 +295,87 @@ __global__ void __launch_bounds__(CD_THREADS) chunk_attn_decode_kernel(ChunkAttn
 #pragma unroll
     for (int j = 0; j < DV / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
     const bf16* qa = q_s + (mr + 8 * (mi & 1)) * KP + 8 * (mi >> 1);
-    int stage = 0;
-    for (int b = b0; b < blocks; b += stride) {
-        load_block(b + (stages - 1) * stride, (stage + stages - 1) % stages);
-        if (stages == 2) asm volatile("cp.async.wait_group 1;" ::: "memory");
-        else if (stages == 3) asm volatile("cp.async.wait_group 2;" ::: "memory");
-        else asm volatile("cp.async.wait_group 3;" ::: "memory");
-        __syncwarp();
-        const bf16* kt = kv_s + (size_t)stage * CD_KEYS * (KP + VP);
-        const bf16* vt = kt + CD_KEYS * KP;
-        float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-        const bf16* kb = kt + (mr + 8 * (mi >> 1)) * KP + 8 * (mi & 1);
-        for (int k0 = 0; k0 < dk; k0 += 16) {
-            uint32_t qf[4], kf[4];
-            ldmatrix_x4(qf, qa + k0);
-            ldmatrix_x4(kf, kb + k0);
-            mma_bf16_16816(s[0], qf, kf[0], kf[1]);
-            mma_bf16_16816(s[1], qf, kf[2], kf[3]);
+    for (int i = 0; i < mine; ++i) {
+        const int stage = i % stages, slot0 = (split + i * splits) * CD_KEYS;
+        if (!mbar_wait(full_bar + stage, (i / stages) & 1)) {
+            if (lane == 0) raise_status(a.status, GLMB_STATUS_WAIT_TIMEOUT);
+            break;
         }
-        float mx[2] = {m[0], m[1]};
-#pragma unroll
-        for (int j = 0; j < 2; ++j)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int key = key0 + b * CD_KEYS + j * 8 + 2 * t4 + (e & 1);
-                const float x = key > pos ? -INFINITY : s[j][e] * scale2;
-                s[j][e] = x;
-                mx[e >> 1] = fmaxf(mx[e >> 1], x);
-            }
-        float fix[2];
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-            mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));
-            mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
-            fix[i] = exp2f(m[i] - mx[i]);  // a block holds at least one visible key: the maximum is finite
-            m[i] = mx[i];
+        unsigned char* kt = tiles_s + (size_t)stage * stage_bytes;
+        unsigned char* vt = kt + kboxes * CD_BOX;
+        const int w0 = warp * 16, left = keys - slot0 - w0;  // this warp's keys of the tile, how many of them exist
+        if (left > 0 && left < 16) {  // values past the last key meet zero weights: they must not be infinite or NaN
+            for (int x = lane; x < (16 - left) * vboxes * 8; x += 32)
+                *reinterpret_cast<uint4*>(const_cast<unsigned char*>(cd_piece(vt, w0 + left + x / (vboxes * 8), x % (vboxes * 8)))) = make_uint4(0, 0, 0, 0);
+            __syncwarp();
         }
-        float sum[2] = {0.f, 0.f};
-#pragma unroll
-        for (int j = 0; j < 2; ++j)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                s[j][e] = exp2f(s[j][e] - m[e >> 1]);
-                sum[e >> 1] += s[j][e];
+        if (left > 0) {
+            float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+            for (int k0 = 0; k0 < dk; k0 += 16) {
+                uint32_t qf[4], kf[4];
+                ldmatrix_x4(qf, qa + k0);
+                ldmatrix_x4(kf, cd_piece(kt, w0 + mr + 8 * (mi >> 1), k0 / 8 + (mi & 1)));
+                mma_bf16_16816(s[0], qf, kf[0], kf[1]);
+                mma_bf16_16816(s[1], qf, kf[2], kf[3]);
             }
-        l[0] = l[0] * fix[0] + sum[0];
-        l[1] = l[1] * fix[1] + sum[1];
-        uint32_t hi[4], lw[4];
-        ca_split(s[0][0], s[0][1], hi[0], lw[0]);
-        ca_split(s[0][2], s[0][3], hi[1], lw[1]);
-        ca_split(s[1][0], s[1][1], hi[2], lw[2]);
-        ca_split(s[1][2], s[1][3], hi[3], lw[3]);
-        const bf16* vb = vt + (mr + 8 * (mi & 1)) * VP + 8 * (mi >> 1);
+            float mx[2] = {m[0], m[1]};
 #pragma unroll
-        for (int j = 0; j < DV / 8; j += 2)
-            if (j * 8 < dv) {
-                o[j][0] *= fix[0]; o[j][1] *= fix[0]; o[j][2] *= fix[1]; o[j][3] *= fix[1];
-                o[j + 1][0] *= fix[0]; o[j + 1][1] *= fix[0]; o[j + 1][2] *= fix[1]; o[j + 1][3] *= fix[1];
-                uint32_t vf[4];
-                ldmatrix_x4_trans(vf, vb + j * 8);
-                mma_bf16_16816(o[j], hi, vf[0], vf[1]);
-                mma_bf16_16816(o[j + 1], hi, vf[2], vf[3]);
-                mma_bf16_16816(o[j], lw, vf[0], vf[1]);
-                mma_bf16_16816(o[j + 1], lw, vf[2], vf[3]);
+            for (int j = 0; j < 2; ++j)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const float x = j * 8 + 2 * t4 + (e & 1) >= left ? -INFINITY : s[j][e] * scale2;
+                    s[j][e] = x;
+                    mx[e >> 1] = fmaxf(mx[e >> 1], x);
+                }
+            float fix[2];
+#pragma unroll
+            for (int i2 = 0; i2 < 2; ++i2) {
+                mx[i2] = fmaxf(mx[i2], __shfl_xor_sync(0xffffffffu, mx[i2], 1));
+                mx[i2] = fmaxf(mx[i2], __shfl_xor_sync(0xffffffffu, mx[i2], 2));
+                fix[i2] = exp2f(m[i2] - mx[i2]);  // at least one key exists: the maximum is finite
+                m[i2] = mx[i2];
             }
-        __syncwarp();  // everyone is done with this stage before it is filled again
-        stage = (stage + 1) % stages;
+            float sum[2] = {0.f, 0.f};
+#pragma unroll
+            for (int j = 0; j < 2; ++j)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    s[j][e] = exp2f(s[j][e] - m[e >> 1]);
+                    sum[e >> 1] += s[j][e];
+                }
+            l[0] = l[0] * fix[0] + sum[0];
+            l[1] = l[1] * fix[1] + sum[1];
+            uint32_t hi[4], lw[4];
+            ca_split(s[0][0], s[0][1], hi[0], lw[0]);
+            ca_split(s[0][2], s[0][3], hi[1], lw[1]);
+            ca_split(s[1][0], s[1][1], hi[2], lw[2]);
+            ca_split(s[1][2], s[1][3], hi[3], lw[3]);
+#pragma unroll
+            for (int j = 0; j < DV / 8; j += 2)
+                if (j * 8 < dv) {
+                    o[j][0] *= fix[0]; o[j][1] *= fix[0]; o[j][2] *= fix[1]; o[j][3] *= fix[1];
+                    o[j + 1][0] *= fix[0]; o[j + 1][1] *= fix[0]; o[j + 1][2] *= fix[1]; o[j + 1][3] *= fix[1];
+                    uint32_t vf[4];
+                    ldmatrix_x4_trans(vf, cd_piece(vt, w0 + mr + 8 * (mi & 1), j + (mi >> 1)));
+                    mma_bf16_16816(o[j], hi, vf[0], vf[1]);
+                    mma_bf16_16816(o[j + 1], hi, vf[2], vf[3]);
+                    mma_bf16_16816(o[j], lw, vf[0], vf[1]);
+                    mma_bf16_16816(o[j + 1], lw, vf[2], vf[3]);
+                }
+        }
+        if (i + stages < mine) {  // every warp has read the stage: fill it again
+            __syncthreads();
+            if (threadIdx.x == 0) load_tile(i + stages);
+        }
     }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
         l[i] += __shfl_xor_sync(0xffffffffu, l[i], 1);
         l[i] += __shfl_xor_sync(0xffffffffu, l[i], 2);
         if (t4 == 0) { ml_s[warp][g + 8 * i][0] = m[i]; ml_s[warp][g + 8 * i][1] = l[i]; }
     }
-    __syncthreads();  // every warp has left its key and value stages: the merge area takes their place
-    float* o_s = reinterpret_cast<float*>(rest);  // [warp][head][dv]
+    __syncthreads();  // every warp has left the tiles: the merge area takes their place
+    float* o_s = reinterpret_cast<float*>(tiles_s);  // [warp][head][dv]
 #pragma unroll
     for (int j = 0; j < DV / 8; ++j)
         if (j * 8 < dv) {
@@ -443,19 +436,15 @@ __global__ void __launch_bounds__(CX_THREADS) chunk_attn_any_kernel(ChunkAttnArg
     __shared__ float p_s[CX_KEYS];
     __shared__ float red[CX_THREADS / 32];
     const int row = blockIdx.x, head = blockIdx.y, group = head / (a.H / a.G);
-    const bool decode = a.k_new == nullptr;
-    const bool active = !a.row_active || a.row_active[row] != 0;
-    const int start = decode ? a.capacity : ca_pos(a, 0);
-    const int pos = ca_pos(a, row), lane_id = ca_lane(a, decode ? row : 0);
+    const bool active = !a.decode || !a.row_active || a.row_active[row] != 0;
+    const int pos = a.decode ? ca_pos(a, row) : a.start + row;
     const int key0 = pos / a.chunk * a.chunk, keys = active ? pos - key0 + 1 : 0;
+    const int64_t row0 = a.decode ? (int64_t)ca_lane(a, row) * a.ring : key0 - a.base;  // where the first visible key lies
     const T* q = reinterpret_cast<const T*>(a.q) + ((int64_t)row * a.H + head) * a.dimp;
     for (int d = threadIdx.x; d < a.dim; d += CX_THREADS) q_f[d] = to_f32(q[d]);
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    auto at = [&](const void* fresh, const void* ring, int padded, int key) {
-        return key >= start ? reinterpret_cast<const T*>(fresh) + ((int64_t)(key - start) * a.G + group) * padded
-                            : reinterpret_cast<const T*>(ring) + (((int64_t)lane_id * a.ring + key % a.ring) * a.G + group) * padded;
-    };
+    auto at = [&](const void* table, int padded, int key) { return reinterpret_cast<const T*>(table) + ((row0 + key) * a.G + group) * padded; };
     float m = a.sink ? a.sink[head] : -INFINITY, l = a.sink ? 1.f : 0.f;
     float acc[CX_COLS];
 #pragma unroll
@@ -463,7 +452,7 @@ __global__ void __launch_bounds__(CX_THREADS) chunk_attn_any_kernel(ChunkAttnArg
     for (int t = 0; t < keys; t += CX_KEYS) {
         const int n = min(CX_KEYS, keys - t);
         for (int j = warp; j < n; j += CX_THREADS / 32) {
-            const T* k = at(a.k_new, a.k_ring, a.dimp, key0 + t + j);
+            const T* k = at(a.k, a.dimp, t + j);
             float s = 0.f;
             for (int d = lane; d < a.dim; d += 32) s = fmaf(q_f[d], to_f32(k[d]), s);
             s = warp_sum(s);
@@ -491,7 +480,7 @@ __global__ void __launch_bounds__(CX_THREADS) chunk_attn_any_kernel(ChunkAttnArg
 #pragma unroll
         for (int i = 0; i < CX_COLS; ++i) acc[i] *= fix;
         for (int j = 0; j < n; ++j) {
-            const T* v = at(a.v_new, a.v_ring, a.vdimp, key0 + t + j);
+            const T* v = at(a.v, a.vdimp, t + j);
             const float w = p_s[j];
 #pragma unroll
             for (int i = 0; i < CX_COLS; ++i) {
@@ -511,8 +500,12 @@ __global__ void __launch_bounds__(CX_THREADS) chunk_attn_any_kernel(ChunkAttnArg
 
 // ===================================================================================================
 static bool chunk_args_ok(const ChunkAttnArgs& a) {
-    return a.rows >= 1 && a.H >= 1 && a.G >= 1 && a.H % a.G == 0 && a.dim >= 1 && a.vdim >= 1 && !(a.dimp & 7) && !(a.vdimp & 7) && a.dimp >= a.dim &&
-           a.vdimp >= a.vdim && a.chunk >= 1 && a.ring >= 1 && a.capacity >= 1 && a.lanes >= 1 && (a.ring >= a.chunk || a.ring >= a.capacity);
+    if (a.rows < 1 || a.H < 1 || a.G < 1 || a.H % a.G || a.dim < 1 || a.vdim < 1 || (a.dimp & 15) || (a.vdimp & 15) || a.dimp < a.dim || a.vdimp < a.vdim ||
+        a.chunk < 1 || !a.q || !a.k || !a.v || !a.out)
+        return false;
+    if (a.decode) return a.ring >= 1 && a.capacity >= 1 && a.lanes >= 1 && (a.ring == a.chunk || a.ring == a.capacity) && a.row_pos && a.row_lane;
+    // every key a row can see lies in the buffers
+    return a.start >= 0 && a.base >= 0 && a.start / a.chunk * a.chunk >= a.base && a.start + a.rows - a.base <= a.keys;
 }
 
 template <typename K>
@@ -529,24 +522,37 @@ static int launch_chunk_prefill(const ChunkAttnArgs& a, cudaStream_t st) {
     static DeviceOnce once;
     const cudaError_t e = chunk_smem_limit(chunk_attn_prefill_kernel<DV>, once);
     if (e != cudaSuccess) return (int)e;
-    const size_t smem = chunk_prefill_smem((a.dim + 15) & ~15, (a.vdim + 15) & ~15);
+    const size_t smem = chunk_prefill_smem(a.dimp, a.vdimp);
     GLMB_LAUNCH(chunk_attn_prefill_kernel<DV>, dim3(ceil_div(a.rows, CP_ROWS), a.H), CP_THREADS, smem, st, a);
     return (int)cudaGetLastError();
 }
 
 template <int DV>
-static int launch_chunk_decode(const ChunkAttnArgs& a, int splits, cudaStream_t st) {
+static int launch_chunk_decode(const ChunkAttnArgs& a, cudaStream_t st) {
     static DeviceOnce once;
-    const cudaError_t e = chunk_smem_limit(chunk_attn_decode_kernel<DV>, once);
+    cudaError_t e = chunk_smem_limit(chunk_attn_decode_kernel<DV>, once);
     if (e != cudaSuccess) return (int)e;
-    const int dk = (a.dim + 15) & ~15, dv = (a.vdim + 15) & ~15;
+    static DeviceOnce wide;  // clusters of 16 are beyond the portable size
+    const int wide_dev = wide.pending();
+    if (wide_dev != DeviceOnce::SET) {
+        e = cudaFuncSetAttribute(chunk_attn_decode_kernel<DV>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+        if (e != cudaSuccess) return (int)e;
+        wide.mark(wide_dev);
+    }
+    CUtensorMap map_k, map_v;
+    const uint64_t ring_rows = (uint64_t)a.lanes * a.ring;
+    if (make_map(&map_k, a.k, ring_rows, (uint64_t)a.G * a.dimp, (uint64_t)a.G * a.dimp, CD_KEYS)) return 3;
+    if (make_map(&map_v, a.v, ring_rows, (uint64_t)a.G * a.vdimp, (uint64_t)a.G * a.vdimp, CD_KEYS)) return 3;
     int stages = 4;
-    while (stages > 2 && chunk_decode_smem(dk, dv, stages) > 112 * 1024) --stages;
-    const int per = a.H / a.G;
+    while (stages > 2 && chunk_decode_smem(a.dimp, a.vdimp, stages) > 112 * 1024) --stages;
+    // CTAs per cluster: enough that the grid reaches every SM, at least one tile each
+    const int heads = a.G * ceil_div(a.H / a.G, CD_HEADS), tiles = ceil_div(a.ring, CD_KEYS);
+    int splits = 1;
+    while (splits < 16 && splits * 2 <= tiles && splits * heads * a.rows < 148) splits *= 2;
     cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = dim3(splits, a.G * ceil_div(per, CD_HEADS), a.rows);
+    cfg.gridDim = dim3(splits, heads, a.rows);
     cfg.blockDim = dim3(CD_THREADS);
-    cfg.dynamicSmemBytes = chunk_decode_smem(dk, dv, stages);
+    cfg.dynamicSmemBytes = chunk_decode_smem(a.dimp, a.vdimp, stages);
     cfg.stream = st;
     cudaLaunchAttribute attr[2];
     attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
@@ -556,37 +562,39 @@ static int launch_chunk_decode(const ChunkAttnArgs& a, int splits, cudaStream_t 
     attr[1].val.clusterDim.y = attr[1].val.clusterDim.z = 1;
     cfg.attrs = attr;
     cfg.numAttrs = 2;
-    const cudaError_t le = cudaLaunchKernelEx(&cfg, chunk_attn_decode_kernel<DV>, a, stages);
+    const cudaError_t le = cudaLaunchKernelEx(&cfg, chunk_attn_decode_kernel<DV>, map_k, map_v, a, stages);
     return le != cudaSuccess ? (int)le : (int)cudaGetLastError();
 }
 
 GLMB_API size_t glmb_chunk_attn_args_sizeof(void) { return sizeof(ChunkAttnArgs); }
 
+static int g_chunk_prefill_tc = 1;
+// 1 (default): tcgen05 prefill kernel where the head sizes allow; 0: the mma.sync kernel.
+GLMB_API void glmb_set_chunk_prefill_tc(int enabled) { g_chunk_prefill_tc = enabled ? 1 : 0; }
+
 // bf16, rows of one sequence at consecutive positions; head sizes up to 256.
 GLMB_API int glmb_chunk_attn_prefill(const ChunkAttnArgs* args, void* stream) {
     const ChunkAttnArgs a = *args;
-    if (!chunk_args_ok(a) || !a.k_new || !a.v_new || a.dim > 256 || a.vdim > 256) return 1;
-    if (a.vdim <= 64) return launch_chunk_prefill<64>(a, (cudaStream_t)stream);
-    if (a.vdim <= 128) return launch_chunk_prefill<128>(a, (cudaStream_t)stream);
+    if (!chunk_args_ok(a) || a.decode || a.dimp > 256 || a.vdimp > 256) return 1;
+    if (g_chunk_prefill_tc && a.dimp <= 128 && a.vdimp <= 128 && a.scale > 0.f) return launch_chunk_attn_tcgen05(a, (cudaStream_t)stream);
+    if (a.vdimp <= 64) return launch_chunk_prefill<64>(a, (cudaStream_t)stream);
+    if (a.vdimp <= 128) return launch_chunk_prefill<128>(a, (cudaStream_t)stream);
     return launch_chunk_prefill<256>(a, (cudaStream_t)stream);
 }
 
 // bf16, one row per sequence, every key in the ring; head sizes up to 256.
 GLMB_API int glmb_chunk_attn_decode(const ChunkAttnArgs* args, void* stream) {
     const ChunkAttnArgs a = *args;
-    if (!chunk_args_ok(a) || a.k_new || a.v_new || a.dim > 256 || a.vdim > 256) return 1;
-    // CTAs per cluster: enough that a full ring leaves each warp a few blocks of keys, at most the portable cluster size
-    int splits = 1;
-    while (splits < 8 && a.ring > splits * CD_WARPS * CD_KEYS) splits *= 2;
-    if (a.vdim <= 64) return launch_chunk_decode<64>(a, splits, (cudaStream_t)stream);
-    if (a.vdim <= 128) return launch_chunk_decode<128>(a, splits, (cudaStream_t)stream);
-    return launch_chunk_decode<256>(a, splits, (cudaStream_t)stream);
+    if (!chunk_args_ok(a) || !a.decode || a.dimp > 256 || a.vdimp > 256) return 1;
+    if (a.vdimp <= 64) return launch_chunk_decode<64>(a, (cudaStream_t)stream);
+    if (a.vdimp <= 128) return launch_chunk_decode<128>(a, (cudaStream_t)stream);
+    return launch_chunk_decode<256>(a, (cudaStream_t)stream);
 }
 
 // Any head size (values up to 1024 columns), bf16 or fp32.
 GLMB_API int glmb_chunk_attn_any(const ChunkAttnArgs* args, int is_f32, void* stream) {
     const ChunkAttnArgs a = *args;
-    if (!chunk_args_ok(a) || !a.k_new != !a.v_new || a.vdim > CX_THREADS * CX_COLS || a.dim > 8192) return 1;
+    if (!chunk_args_ok(a) || a.vdim > CX_THREADS * CX_COLS || a.dim > 8192) return 1;
     const dim3 grid(a.rows, a.H);
     const size_t smem = (size_t)a.dim * sizeof(float);
     if (is_f32) GLMB_LAUNCH(chunk_attn_any_kernel<float>, grid, CX_THREADS, smem, (cudaStream_t)stream, a);

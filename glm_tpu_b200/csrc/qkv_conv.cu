@@ -6,13 +6,16 @@
 //   (a, b) -> (a cos - b sin, b cos + a sin)               dimensions i and i + dims/2 of every q and k head, fp32 table
 //   v       = (1 - lambda) v + lambda v_first
 //
-// A block owns one head (of q, k or v) and RB consecutive rows.  Prefill: the rows are one sequence; the rows' own history comes from
-// the projection, that of the first rows from the state, and the block of the first rows also advances the state once it has read it
-// (no other block reads it: RB >= taps - 1).  Decode: every row is its own sequence (lane), RB = 1.
+// A block owns one head (of q, k or v) and some consecutive rows.  Prefill: the rows are one sequence; the rows' own history comes from
+// the projection, that of the first rows from the state, and the block of the first rows also advances the state once it has read it (no
+// other block reads it: a block holds at least taps - 1 rows).  Decode: every row is its own sequence (lane), one row per block.
 //
-// Keys and values go to the lane's ring (slot = position mod ring size: with chunked attention a ring of one chunk holds everything a
-// later token can see) and, in prefill, to linear buffers that the attention reads for the rows of this step.  Rows before `ring_from`
-// stay out of the ring: their slots may still hold keys that queries of this very step need; ring_store writes them afterwards.
+//   qkv_conv_kernel       any sizes, decode and prefill: convolution into shared memory, then rotation / mixing / stores
+//   qkv_conv_rows_kernel  prefill, head sizes in multiples of 8, up to 4 taps: a thread slides down a strip of rows with two 8-channel
+//                         vectors (for rotated dimensions the two halves of a pair), its taps and its window in registers
+//
+// Keys and values go to the lane's ring (slot = position mod ring size: with chunked attention a ring of one chunk holds everything a later
+// token can see) or, when `k_lin` is set, to linear buffers, row by row.
 #include "common.cuh"
 #include "vec8.cuh"
 
@@ -26,31 +29,79 @@ struct QkvConvArgs {
     void* state;                                 // [lanes, taps - 1, C]
     const int *row_pos, *row_lane, *row_active;  // row_active may be NULL
     const float2* rot; int rot_dims;             // [capacity, rot_dims / 2] (cos, sin)
-    void *q, *k_new, *v_new;                     // [rows, H, dimp], [rows, G, dimp], [rows, G, vdimp]; k_new / v_new NULL in decode
+    void* q;                                     // [rows, H, dimp]
+    void *k_lin, *v_lin;                         // [rows, G, dimp], [rows, G, vdimp], or NULL: keys and values go to the ring
     void *k_ring, *v_ring; int ring;             // [lanes, ring, G, dimp], [lanes, ring, G, vdimp]
     void* v_first; int v_mode; float mix;        // [rows, G, vdimp]; 0: not used, 1: store this layer's values, 2: mix with them
-    int H, G, dim, dimp, vdim, vdimp, rows, decode, ring_from, capacity, lanes, rows_per_block;
+    int H, G, dim, dimp, vdim, vdimp, rows, decode, capacity, lanes, rows_per_block;
     uint32_t* status;
 };
+
+struct QcHead { int kind, slot, hd, hdp, chan0, C; };  // kind 0: q, 1: k, 2: v
+
+__device__ __forceinline__ QcHead qc_head(const QkvConvArgs& a, int head) {
+    QcHead h;
+    h.kind = head < a.H ? 0 : head < a.H + a.G ? 1 : 2;
+    h.hd = h.kind == 2 ? a.vdim : a.dim;
+    h.hdp = h.kind == 2 ? a.vdimp : a.dimp;
+    h.slot = h.kind == 0 ? head : h.kind == 1 ? head - a.H : head - a.H - a.G;
+    h.C = (a.H + a.G) * a.dim + a.G * a.vdim;
+    h.chan0 = h.kind == 0 ? h.slot * a.dim : h.kind == 1 ? (a.H + h.slot) * a.dim : (a.H + a.G) * a.dim + h.slot * a.vdim;
+    return h;
+}
+
+__device__ __forceinline__ int qc_lane(const QkvConvArgs& a, int row) {
+    const int lane = a.row_lane[row];
+    if (lane >= 0 && lane < a.lanes) return lane;
+    if (threadIdx.x == 0) raise_status(a.status, GLMB_STATUS_BAD_INDEX);
+    return min(max(lane, 0), a.lanes - 1);
+}
+
+// The state's next rows are the last taps - 1 rows up to the end of the step that starts at row `first` and has `seq` rows.
+template <typename T>
+__device__ __forceinline__ void qc_advance_state(const QkvConvArgs& a, const QcHead& h, T* state, int first, int seq) {
+    const T* proj = reinterpret_cast<const T*>(a.proj);
+    const int keep = a.taps - 1;
+    for (int c = threadIdx.x; c < h.hd; c += QC_THREADS)
+        for (int j = 0; j < keep; ++j)  // ascending: entry j only reads later entries
+            state[(int64_t)j * h.C + c] = seq + j < keep ? state[(int64_t)(j + seq) * h.C + c]
+                                                         : proj[(int64_t)(first + seq - keep + j) * a.proj_stride + h.chan0 + c];
+}
+
+// Eight finished channels of one row to where they belong; values are mixed on the way.
+template <typename T>
+__device__ __forceinline__ void qc_store(const QkvConvArgs& a, const QcHead& h, int row, int pos, int lane, bool keep, int c, float (&o)[8]) {
+    if (h.kind == 0) {
+        store8(reinterpret_cast<T*>(a.q) + ((int64_t)row * a.H + h.slot) * h.hdp + c, o);
+        return;
+    }
+    const int64_t at = ((int64_t)row * a.G + h.slot) * h.hdp + c;
+    if (h.kind == 2 && a.v_mode) {
+        T* vf = reinterpret_cast<T*>(a.v_first) + at;
+        if (a.v_mode == 1) {
+            store8(vf, o);
+        } else {
+            float f[8];
+            load8(vf, f);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) o[e] = (1.f - a.mix) * o[e] + a.mix * f[e];
+        }
+    }
+    T* lin = reinterpret_cast<T*>(h.kind == 1 ? a.k_lin : a.v_lin);
+    if (lin) store8(lin + at, o);
+    else if (keep) store8(reinterpret_cast<T*>(h.kind == 1 ? a.k_ring : a.v_ring) + (((int64_t)lane * a.ring + pos % a.ring) * a.G + h.slot) * h.hdp + c, o);
+}
 
 template <typename T, int VEC>
 __global__ void __launch_bounds__(QC_THREADS) qkv_conv_kernel(QkvConvArgs a) {
     GLMB_PDL_PROLOGUE();
     extern __shared__ float y_s[];  // [rows_per_block][hd]
-    const int head = blockIdx.y;
-    const int kind = head < a.H ? 0 : head < a.H + a.G ? 1 : 2;
-    const int hd = kind == 2 ? a.vdim : a.dim, hdp = kind == 2 ? a.vdimp : a.dimp;
-    const int slot = kind == 0 ? head : kind == 1 ? head - a.H : head - a.H - a.G;
-    const int C = (a.H + a.G) * a.dim + a.G * a.vdim;
-    const int chan0 = kind == 0 ? slot * a.dim : kind == 1 ? (a.H + slot) * a.dim : (a.H + a.G) * a.dim + slot * a.vdim;
+    const QcHead h = qc_head(a, blockIdx.y);
+    const int hd = h.hd, C = h.C, chan0 = h.chan0;
     const int r0 = blockIdx.x * a.rows_per_block;
     const int n = min(a.rows_per_block, a.rows - r0);
     const T* proj = reinterpret_cast<const T*>(a.proj);
-    int lane = a.row_lane[a.decode ? r0 : 0];
-    if (lane < 0 || lane >= a.lanes) {
-        if (threadIdx.x == 0) raise_status(a.status, GLMB_STATUS_BAD_INDEX);
-        lane = min(max(lane, 0), a.lanes - 1);
-    }
+    const int lane = qc_lane(a, a.decode ? r0 : 0);
     T* state = reinterpret_cast<T*>(a.state) + (int64_t)lane * (a.taps - 1) * C + chan0;
     const bool active = !a.row_active || a.row_active[a.decode ? r0 : 0] != 0;
 
@@ -84,17 +135,10 @@ __global__ void __launch_bounds__(QC_THREADS) qkv_conv_kernel(QkvConvArgs a) {
     }
     __syncthreads();
 
-    // ---- the state moves on: its next rows are the last taps - 1 rows up to the end of this step ----------
-    if (active && (a.decode || blockIdx.x == 0) && a.row_pos[a.decode ? r0 : 0] >= 0) {
-        const int seq = a.decode ? 1 : a.rows, first = a.decode ? r0 : 0, keep = a.taps - 1;
-        for (int c = threadIdx.x; c < hd; c += QC_THREADS)
-            for (int j = 0; j < keep; ++j)  // ascending: entry j only reads later entries
-                state[(int64_t)j * C + c] = seq + j < keep ? state[(int64_t)(j + seq) * C + c]
-                                                           : proj[(int64_t)(first + seq - keep + j) * a.proj_stride + chan0 + c];
-    }
+    if (active && (a.decode || blockIdx.x == 0) && a.row_pos[a.decode ? r0 : 0] >= 0) qc_advance_state(a, h, state, a.decode ? r0 : 0, a.decode ? 1 : a.rows);
 
     // ---- rotation / value mixing, stores ------------------------------------------------------------------
-    const int half = a.rot_dims / 2, outs = hdp / 8;
+    const int half = a.rot_dims / 2, outs = h.hdp / 8;
     for (int i = threadIdx.x; i < n * outs; i += QC_THREADS) {
         const int r = i / outs, c = (i % outs) * 8;
         const int row = r0 + r;
@@ -110,61 +154,118 @@ __global__ void __launch_bounds__(QC_THREADS) qkv_conv_kernel(QkvConvArgs a) {
         for (int e = 0; e < 8; ++e) {
             const int d = c + e;
             float v = d < hd ? y[d] : 0.f;
-            if (kind < 2 && d < a.rot_dims) {
+            if (h.kind < 2 && d < a.rot_dims) {
                 const bool low = d < half;
                 const float2 cs = a.rot[(int64_t)pos * half + (low ? d : d - half)];
                 v = low ? v * cs.x - y[d + half] * cs.y : v * cs.x + y[d - half] * cs.y;
             }
             o[e] = v;
         }
-        if (kind == 0) {
-            store8(reinterpret_cast<T*>(a.q) + ((int64_t)row * a.H + slot) * hdp + c, o);
-            continue;
-        }
-        const int64_t at = ((int64_t)row * a.G + slot) * hdp + c;
-        if (kind == 2 && a.v_mode) {
-            T* vf = reinterpret_cast<T*>(a.v_first) + at;
-            if (a.v_mode == 1) {
-                store8(vf, o);
-            } else {
-                float f[8];
-                load8(vf, f);
-#pragma unroll
-                for (int e = 0; e < 8; ++e) o[e] = (1.f - a.mix) * o[e] + a.mix * f[e];
-            }
-        }
-        T* fresh = reinterpret_cast<T*>(kind == 1 ? a.k_new : a.v_new);
-        if (fresh) store8(fresh + at, o);
-        if (active && !bad && row >= a.ring_from) {
-            T* ring = reinterpret_cast<T*>(kind == 1 ? a.k_ring : a.v_ring);
-            store8(ring + (((int64_t)lane * a.ring + pos % a.ring) * a.G + slot) * hdp + c, o);
-        }
+        qc_store<T>(a, h, row, pos, lane, active && !bad, c, o);
     }
 }
 
-// Rows [from, rows) of the linear key / value buffers of a step into the lane's ring.
+// ---------------------------------------------------------------------------------------------------
+#define QR_TAPS 4
+#define QR_STRIP 8  // rows a thread slides over
+
 template <typename T>
-__global__ void __launch_bounds__(256)
-ring_store_kernel(const T* __restrict__ k_new, const T* __restrict__ v_new, const int* __restrict__ row_pos, const int* __restrict__ row_lane,
-                  T* __restrict__ k_ring, T* __restrict__ v_ring, int ring, int k_row, int v_row, int from, int rows, int lanes, int capacity) {
+__global__ void __launch_bounds__(QC_THREADS) qkv_conv_rows_kernel(QkvConvArgs a) {
     GLMB_PDL_PROLOGUE();
-    const int lane = row_lane[0];
-    if (lane < 0 || lane >= lanes) return;
-    const int vecs = (k_row + v_row) / 8;
-    const int64_t total = (int64_t)(rows - from) * vecs;
-    for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
-        const int row = from + (int)(i / vecs), c = (int)(i % vecs) * 8;
-        const int pos = row_pos[row];
-        if (pos < 0 || pos >= capacity) continue;
-        const int64_t slot = (int64_t)lane * ring + pos % ring;
-        float v[8];
-        if (c < k_row) {
-            load8(k_new + (int64_t)row * k_row + c, v);
-            store8(k_ring + slot * k_row + c, v);
-        } else {
-            load8(v_new + (int64_t)row * v_row + c - k_row, v);
-            store8(v_ring + slot * v_row + c - k_row, v);
+    const QcHead h = qc_head(a, blockIdx.y);
+    const T* proj = reinterpret_cast<const T*>(a.proj) + h.chan0;
+    const int lane = qc_lane(a, 0), start = a.row_pos[0], keep = a.taps - 1;
+    T* state = reinterpret_cast<T*>(a.state) + (int64_t)lane * keep * h.C + h.chan0;
+    // pairs of channel vectors: the rotated halves of q and k first, then the rest two by two
+    const int vecs = h.hd / 8, half = h.kind < 2 ? a.rot_dims / 2 : 0, rot_pairs = half / 8, plain = vecs - 2 * rot_pairs;
+    const int pairs = rot_pairs + (plain + 1) / 2, strips = QC_THREADS / pairs;
+    const int pair = threadIdx.x % pairs, strip = threadIdx.x / pairs;
+    const bool rotated = pair < rot_pairs;
+    const int c0 = rotated ? pair * 8 : half * 2 + (pair - rot_pairs) * 16, c1 = rotated ? c0 + half : c0 + 8;
+    const bool both = c1 < h.hd;
+    const int block_rows = strips * QR_STRIP, first = blockIdx.x * block_rows + strip * QR_STRIP, last = min(first + QR_STRIP, a.rows);
+    if (strip < strips && first < a.rows) {
+        float w0[QR_TAPS][8], w1[QR_TAPS][8], u0[QR_TAPS][8], u1[QR_TAPS][8];  // window: u[QR_TAPS - 1] is the current row
+        auto fetch = [&](int row, float (&x)[8], float (&y)[8]) {
+            const T* src = nullptr;
+            if (row >= 0) src = proj + (int64_t)row * a.proj_stride;
+            else if (start + row >= 0) src = state + (int64_t)(keep + row) * h.C;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) x[e] = y[e] = 0.f;
+            if (src) {
+                load8(src + c0, x);
+                if (both) load8(src + c1, y);
+            }
+        };
+#pragma unroll
+        for (int j = 0; j < QR_TAPS; ++j) {
+            const int tap = j - (QR_TAPS - a.taps);  // fewer taps: the oldest ones are zero
+#pragma unroll
+            for (int e = 0; e < 8; ++e) w0[j][e] = w1[j][e] = u0[j][e] = u1[j][e] = 0.f;
+            if (tap >= 0) {
+                load8(a.conv_w + (int64_t)tap * h.C + h.chan0 + c0, w0[j]);
+                if (both) load8(a.conv_w + (int64_t)tap * h.C + h.chan0 + c1, w1[j]);
+                if (j < QR_TAPS - 1) fetch(first - (QR_TAPS - 1 - j), u0[j], u1[j]);
+            }
         }
+        for (int row = first; row < last; ++row) {
+            fetch(row, u0[QR_TAPS - 1], u1[QR_TAPS - 1]);
+            float y0[8], y1[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+                for (int j = 0; j < QR_TAPS; ++j) { s0 = fmaf(w0[j][e], u0[j][e], s0); s1 = fmaf(w1[j][e], u1[j][e], s1); }
+                y0[e] = s0;
+                y1[e] = s1;
+            }
+            int pos = a.row_pos[row];
+            const bool bad = pos < 0 || pos >= a.capacity;
+            if (bad) {
+                raise_status(a.status, GLMB_STATUS_BAD_INDEX);
+                pos = min(max(pos, 0), a.capacity - 1);
+            }
+            if (rotated) {
+                const float4* table = reinterpret_cast<const float4*>(a.rot + (int64_t)pos * half + c0);
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const float4 cs = table[e];
+                    const float p = y0[2 * e], q = y1[2 * e], r = y0[2 * e + 1], s = y1[2 * e + 1];
+                    y0[2 * e] = p * cs.x - q * cs.y;
+                    y1[2 * e] = q * cs.x + p * cs.y;
+                    y0[2 * e + 1] = r * cs.z - s * cs.w;
+                    y1[2 * e + 1] = s * cs.z + r * cs.w;
+                }
+            }
+            qc_store<T>(a, h, row, pos, lane, !bad, c0, y0);
+            if (both) qc_store<T>(a, h, row, pos, lane, !bad, c1, y1);
+            if (pair == 0 && h.hdp > h.hd) {  // the padding of the head row
+                float zero[8];
+#pragma unroll
+                for (int e = 0; e < 8; ++e) zero[e] = 0.f;
+                for (int c = h.hd; c < h.hdp; c += 8) qc_store<T>(a, h, row, pos, lane, !bad, c, zero);
+            }
+#pragma unroll
+            for (int j = 0; j + 1 < QR_TAPS; ++j)
+#pragma unroll
+                for (int e = 0; e < 8; ++e) { u0[j][e] = u0[j + 1][e]; u1[j][e] = u1[j + 1][e]; }
+        }
+    }
+    if (blockIdx.x == 0) {
+        __syncthreads();  // the first rows have read the state
+        if (start >= 0) qc_advance_state(a, h, state, 0, a.rows);
+    }
+}
+
+// ---------------------------------------------------------------------------------------------------
+// Two contiguous runs of cache rows from one place to another (a ring's current chunk to a linear buffer or back): 16-byte pieces.
+__global__ void __launch_bounds__(256)
+kv_copy_kernel(const uint4* __restrict__ k_src, uint4* __restrict__ k_dst, int64_t k_pieces, const uint4* __restrict__ v_src, uint4* __restrict__ v_dst,
+               int64_t v_pieces) {
+    GLMB_PDL_PROLOGUE();
+    for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < k_pieces + v_pieces; i += (int64_t)gridDim.x * blockDim.x) {
+        if (i < k_pieces) k_dst[i] = k_src[i];
+        else v_dst[i - k_pieces] = v_src[i - k_pieces];
     }
 }
 
@@ -178,13 +279,26 @@ GLMB_API int glmb_qkv_conv(const QkvConvArgs* args, int is_f32, void* stream) {
     const int widest = a.dim > a.vdim ? a.dim : a.vdim;
     if (a.rows < 1 || a.H < 1 || a.G < 1 || a.H % a.G || a.dim < 1 || a.vdim < 1 || (a.dimp & 7) || (a.vdimp & 7) || a.dimp < a.dim || a.vdimp < a.vdim) return 1;
     if (a.taps < 1 || a.taps > glmb_qkv_conv_max_taps(widest) || a.rot_dims < 0 || (a.rot_dims & 1) || a.rot_dims > a.dim || a.ring < 1) return 1;
-    if (a.decode && (a.k_new || a.v_new)) return 1;
+    if ((a.dimp & 15) || (a.vdimp & 15) || !a.k_lin != !a.v_lin || (a.decode && a.k_lin)) return 1;
     if (a.v_mode && !a.v_first) return 1;
+    const bool vec = !(a.dim & 7) && !(a.vdim & 7) && !(a.proj_stride & 7);
+    cudaStream_t st = (cudaStream_t)stream;
+    const int pairs = a.rot_dims / 16 + ((widest / 8 - a.rot_dims / 8) + 1) / 2;
+    if (vec && !a.decode && a.taps <= QR_TAPS && !(a.rot_dims & 15) && widest <= 1024 && pairs <= QC_THREADS) {
+        // strips per block differ between head kinds (their pair counts do): the grid covers the kind with the shortest block
+        auto blocks_of = [&](int hd, int rot) {
+            const int p = rot / 16 + ((hd / 8 - rot / 8) + 1) / 2;
+            return ceil_div(a.rows, QC_THREADS / p * QR_STRIP);
+        };
+        const int bq = blocks_of(a.dim, a.rot_dims), bv = blocks_of(a.vdim, 0);
+        const dim3 grid(bq > bv ? bq : bv, a.H + 2 * a.G);
+        if (is_f32) GLMB_LAUNCH(qkv_conv_rows_kernel<float>, grid, QC_THREADS, 0, st, a);
+        else GLMB_LAUNCH(qkv_conv_rows_kernel<bf16>, grid, QC_THREADS, 0, st, a);
+        return (int)cudaGetLastError();
+    }
     a.rows_per_block = a.decode ? 1 : min(QC_MAX_ROWS, QC_SMEM_FLOATS / widest);
     const dim3 grid(ceil_div(a.rows, a.rows_per_block), a.H + 2 * a.G);
     const size_t smem = (size_t)a.rows_per_block * widest * sizeof(float);
-    const bool vec = !(a.dim & 7) && !(a.vdim & 7) && !(a.proj_stride & 7);
-    cudaStream_t st = (cudaStream_t)stream;
     if (is_f32) {
         if (vec) GLMB_LAUNCH((qkv_conv_kernel<float, 8>), grid, QC_THREADS, smem, st, a);
         else GLMB_LAUNCH((qkv_conv_kernel<float, 1>), grid, QC_THREADS, smem, st, a);
@@ -195,17 +309,10 @@ GLMB_API int glmb_qkv_conv(const QkvConvArgs* args, int is_f32, void* stream) {
     return (int)cudaGetLastError();
 }
 
-// k_row, v_row: elements of a key / value row (all heads, padded: multiples of 8).
-GLMB_API int glmb_ring_store(const void* k_new, const void* v_new, const int* row_pos, const int* row_lane, void* k_ring, void* v_ring, int ring,
-                             int k_row, int v_row, int from, int rows, int lanes, int capacity, int is_f32, void* stream) {
-    if (rows < 1 || from < 0 || from >= rows || ring < 1 || (k_row & 7) || (v_row & 7) || rows - from > ring) return 1;
-    const int64_t blocks = ((int64_t)(rows - from) * ((k_row + v_row) / 8) + 255) / 256;
-    const int grid = blocks < 148 * 8 ? (int)blocks : 148 * 8;
-    if (is_f32)
-        GLMB_LAUNCH(ring_store_kernel<float>, grid, 256, 0, (cudaStream_t)stream, (const float*)k_new, (const float*)v_new, row_pos, row_lane,
-                    (float*)k_ring, (float*)v_ring, ring, k_row, v_row, from, rows, lanes, capacity);
-    else
-        GLMB_LAUNCH(ring_store_kernel<bf16>, grid, 256, 0, (cudaStream_t)stream, (const bf16*)k_new, (const bf16*)v_new, row_pos, row_lane,
-                    (bf16*)k_ring, (bf16*)v_ring, ring, k_row, v_row, from, rows, lanes, capacity);
+GLMB_API int glmb_kv_copy(const void* k_src, void* k_dst, int64_t k_bytes, const void* v_src, void* v_dst, int64_t v_bytes, void* stream) {
+    if (k_bytes < 16 || v_bytes < 16 || (k_bytes & 15) || (v_bytes & 15)) return 1;
+    const int64_t pieces = (k_bytes + v_bytes) / 16, blocks = (pieces + 255) / 256;
+    GLMB_LAUNCH(kv_copy_kernel, (unsigned)(blocks < 148 * 8 ? blocks : 148 * 8), 256, 0, (cudaStream_t)stream, (const uint4*)k_src, (uint4*)k_dst, k_bytes / 16,
+                (const uint4*)v_src, (uint4*)v_dst, v_bytes / 16);
     return (int)cudaGetLastError();
 }

@@ -40,11 +40,9 @@ __global__ void __launch_bounds__(256)
 glu_rows_kernel(const T* __restrict__ gate, const T* __restrict__ up, int64_t in_stride, T* __restrict__ act, int64_t out_stride, int rows, int n,
                 int kind) {
     GLMB_PDL_PROLOGUE();
-    const int per_row = n / 8;
-    const int64_t total = (int64_t)rows * per_row;
-    for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
-        const int64_t r = i / per_row;
-        const int c = (int)(i % per_row) * 8;
+    const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
+    if (c >= n) return;
+    for (int r = blockIdx.y; r < rows; r += gridDim.y) {
         float g[8], u[8];
         load8(gate + r * in_stride + c, g);
         load8(up + r * in_stride + c, u);
@@ -59,8 +57,7 @@ GLMB_API int glmb_glu_rows(const void* gate, const void* up, int64_t in_stride, 
                            void* stream) {
     if (rows < 1 || n < 8 || (n & 7) || (in_stride & 7) || (out_stride & 7) || (kind != GLU_SILU && kind != GLU_GELU_TANH)) return 1;
     if ((reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(up) | reinterpret_cast<uintptr_t>(act)) & 15) return 1;
-    const int64_t blocks = ((int64_t)rows * (n / 8) + 255) / 256;
-    const int grid = blocks < 148 * 8 ? (int)blocks : 148 * 8;
+    const dim3 grid(ceil_div(n / 8, 256), rows < 32768 ? rows : 32768);
     if (is_f32)
         GLMB_LAUNCH(glu_rows_kernel<float>, grid, 256, 0, (cudaStream_t)stream, (const float*)gate, (const float*)up, in_stride, (float*)act, out_stride,
                     rows, n, kind);

@@ -11,8 +11,9 @@ Per layer, five launches in decode:
     chunk_attention   over the lane's ring
     skinny_bf16       [attention | feed-forward] @ [W_o | W_down]: the fp32 update of the residual
 
-In prefill the projections run on the tcgen05 GEMM (gate / up and activation are two launches), the attention reads the step's own rows
-from linear buffers and older ones from the ring, and rows of a chunk that began inside the step enter the ring afterwards.
+In prefill the projections run on the tcgen05 GEMM (gate / up and activation are two launches).  A step whose rows lie in one chunk of a layer
+attends over the lane's ring itself; one that crosses into another chunk attends over a linear buffer (the chunk so far, copied from the
+ring, then the step's rows), and the rows of the last chunk enter the ring afterwards.
 
 The residual, norms, angles, scores, softmax and sums are fp32 in every mode.  ``weights.dtype`` selects the rest: bf16 operands with fp32
 accumulation, or fp32 throughout (plain FMA kernels: the 32-bit path exists to check the model, not to serve it).
@@ -26,7 +27,7 @@ import torch
 
 from glm_tpu_b200.config.cache import RingCacheConfig
 from glm_tpu_b200.exceptions import PlanValidationError
-from glm_tpu_b200.models.namizen.weights import NamizenWeights, pad8
+from glm_tpu_b200.models.namizen.weights import NamizenWeights, pad8, pad16
 from glm_tpu_b200.ops import native
 from glm_tpu_b200.parallel.peer import PeerGroup
 from glm_tpu_b200.runner.lane_state import RING, LaneRegisters
@@ -62,12 +63,13 @@ class NamizenWorkspace:
         self.h1, self.h2 = t(rows, model.width), t(rows, model.width)
         # flat buffers: every layer views them with its own row size
         self.proj = t(rows * max(pad8(m.qkv_width) for m in mixers))
-        self.q = t(rows * max(m.heads * pad8(m.dim) for m in mixers))
-        # columns past a head row's or a branch's own width must stay finite (zero weights meet them): zeroed once per layer shape below
+        self.q = t(rows * max(m.heads * pad16(m.dim) for m in mixers))
         self.branches = {cols: t(rows, cols) for cols in {(lw.attn_cols + lw.ff_cols) for lw in model.w.layers}}
-        self.k_new = t(rows * max(m.kv_heads * pad8(m.dim) for m in mixers)) if prefill else None
-        self.v_new = t(rows * max(m.kv_heads * pad8(m.vdim) for m in mixers)) if prefill else None
-        self.v_first = t(rows * max([m.kv_heads * pad8(m.vdim) for m in mixers if m.v_mix] or [8]))
+        # linear keys and values of a prefill step that crosses a chunk
+        lin = [model.cache.linear_rows(i, rows) if prefill else 0 for i in range(g.num_layers)]
+        self.k_lin = t(max(n * m.kv_heads * pad16(m.dim) for n, m in zip(lin, mixers)))
+        self.v_lin = t(max(n * m.kv_heads * pad16(m.vdim) for n, m in zip(lin, mixers)))
+        self.v_first = t(rows * max([m.kv_heads * pad16(m.vdim) for m in mixers if m.v_mix] or [8]))
         self.gate_up = t(rows * 2 * max(lw.ff_cols for lw in model.w.layers)) if prefill or model.is_f32 else None
         self.logits = torch.zeros((rows if not prefill else 0, pad8(g.vocab_size)), dtype=torch.float32, device=dev)
         self.local_best = torch.zeros(rows, dtype=torch.int64, device=dev)
@@ -115,7 +117,7 @@ class NamizenModel:
             native.gemm_bf16_tc(x, w, out, status=self.peer.status_ptr)
 
     def _attention(self, ws: NamizenWorkspace, state: RingState, layer: int, proj: torch.Tensor, out: torch.Tensor, rows: int, row_pos, row_lane,
-                   row_active, decode: bool, start: int) -> None:
+                   row_active, decode: bool, start: int, lane: int) -> None:
         m, lw, cache = self.g.layers[layer].mixer, self.w.layers[layer], self.cache
         first = self.g.first_mixing_layer
         a = native.QkvConvArgs()
@@ -127,28 +129,42 @@ class NamizenModel:
         a.q = ws.q.data_ptr()
         a.k_ring, a.v_ring, a.ring = state.k[layer].data_ptr(), state.v[layer].data_ptr(), cache.ring(layer)
         a.v_first, a.v_mode, a.mix = ws.v_first.data_ptr(), (0 if not m.v_mix else 1 if layer == first else 2), lw.mix
-        a.H, a.G, a.dim, a.dimp, a.vdim, a.vdimp = m.heads, m.kv_heads, m.dim, pad8(m.dim), m.vdim, pad8(m.vdim)
+        a.H, a.G, a.dim, a.dimp, a.vdim, a.vdimp = m.heads, m.kv_heads, m.dim, pad16(m.dim), m.vdim, pad16(m.vdim)
         a.rows, a.decode, a.capacity, a.lanes = rows, int(decode), cache.context_capacity, cache.lanes
         a.status = self.peer.status_ptr
-        keep, later = 0, False
-        if not decode:
-            a.k_new, a.v_new = ws.k_new.data_ptr(), ws.v_new.data_ptr()
-            keep, later = cache.ring_from(layer, start, rows)
-        a.ring_from = rows if later else keep
-        native.qkv_conv(a, self.is_f32)
         b = native.ChunkAttnArgs()
-        b.q, b.k_new, b.v_new, b.k_ring, b.v_ring = a.q, a.k_new, a.v_new, a.k_ring, a.v_ring
-        b.sink = lw.sink.data_ptr()
+        b.q, b.sink = a.q, lw.sink.data_ptr()
         b.row_pos, b.row_lane, b.row_active = a.row_pos, a.row_lane, a.row_active
         b.out, b.out_stride = out.data_ptr(), out.stride(0)
         b.rows, b.H, b.G, b.dim, b.dimp, b.vdim, b.vdimp = rows, m.heads, m.kv_heads, m.dim, a.dimp, m.vdim, a.vdimp
-        b.chunk, b.ring, b.capacity, b.lanes, b.scale = cache.chunk(layer), a.ring, a.capacity, a.lanes, m.scale
+        b.decode, b.chunk, b.ring, b.capacity, b.lanes, b.scale = a.decode, cache.chunk(layer), a.ring, a.capacity, a.lanes, m.scale
         b.status = self.peer.status_ptr
+        if decode:
+            b.k, b.v = a.k_ring, a.v_ring
+            native.qkv_conv(a, self.is_f32)
+            native.chunk_attention(b, self.is_f32, plain=self.plain_attention)
+            return
+        k_row, v_row = (m.kv_heads * padded * state.k[layer].element_size() for padded in (a.dimp, a.vdimp))  # bytes of a cached row
+        k_lane, v_lane = a.k_ring + lane * a.ring * k_row, a.v_ring + lane * a.ring * v_row
+        b.start, b.base = start, cache.first_position(layer, start)
+        b.keys = start + rows - b.base
+        across = cache.crossing(layer, start, rows)
+        if across is None:
+            b.k, b.v = k_lane, v_lane
+            native.qkv_conv(a, self.is_f32)
+            native.chunk_attention(b, self.is_f32, plain=self.plain_attention)
+            return
+        before, after = across
+        b.k, b.v = ws.k_lin.data_ptr(), ws.v_lin.data_ptr()
+        if before:
+            native.kv_copy(k_lane, b.k, before * k_row, v_lane, b.v, before * v_row)
+        a.k_lin, a.v_lin = b.k + before * k_row, b.v + before * v_row
+        native.qkv_conv(a, self.is_f32)
         native.chunk_attention(b, self.is_f32, plain=self.plain_attention)
-        if later:
-            native.ring_store(a, keep, self.is_f32)
+        tail = b.keys - after
+        native.kv_copy(b.k + tail * k_row, k_lane, after * k_row, b.v + tail * v_row, v_lane, after * v_row)
 
-    def _layer(self, ws, state, layer: int, rows: int, row_pos, row_lane, row_active, decode: bool, start: int) -> None:
+    def _layer(self, ws, state, layer: int, rows: int, row_pos, row_lane, row_active, decode: bool, start: int, lane: int) -> None:
         """Both branches of a layer from ``ws.h1`` / ``ws.h2``; the fp32 update of the residual lands in ``ws.update``."""
         lw = self.w.layers[layer]
         both = ws.branches[lw.attn_cols + lw.ff_cols][:rows]
@@ -169,7 +185,7 @@ class NamizenModel:
                 gate_up = ws.gate_up[: rows * 2 * lw.ff_cols].view(rows, 2 * lw.ff_cols)
                 self._mm(h2, lw.gate_up, gate_up)
                 native.glu_rows(gate_up[:, : lw.ff_cols], gate_up[:, lw.ff_cols :], act, native.GLU_GELU_TANH)
-        self._attention(ws, state, layer, proj, both, rows, row_pos, row_lane, row_active, decode, start)
+        self._attention(ws, state, layer, proj, both, rows, row_pos, row_lane, row_active, decode, start, lane)
         self._mm(both, lw.out, ws.update[:rows])
 
     # ------------------------------------------------------------------------------ whole model
@@ -182,12 +198,14 @@ class NamizenModel:
         """
         g, w, eps = self.g, self.w, self.g.norm_eps
         start = 0 if decode else max_ctx - rows
+        if not decode and not (0 <= start and max_ctx <= self.cache.context_capacity and lane_of_rows is not None and 0 <= lane_of_rows < self.cache.lanes):
+            raise ValueError("prefill rows lie within the context of one lane")
         residual, update = ws.residual[:rows], None
         for i, lw in enumerate(w.layers):
             source = dict(tokens=tokens, table=w.embed, vocab=g.vocab_size) if i == 0 else dict(update=update)
             native.parallel_norm(residual, g.hidden_size, lw.norm1, ws.h1[:rows], eps, w2=lw.norm2, out2=ws.h2 if lw.norm2 is not None else None,
                                  status=self.peer.status_ptr, **source)
-            self._layer(ws, state, i, rows, row_pos, row_lane, row_active, decode, start)
+            self._layer(ws, state, i, rows, row_pos, row_lane, row_active, decode, start, lane_of_rows)
             update = ws.update[:rows]
             if self.trace is not None:
                 self.trace.setdefault("residual", {})[i] = (residual + update)[:, : g.hidden_size].clone()

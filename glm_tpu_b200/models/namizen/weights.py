@@ -26,6 +26,10 @@ def pad8(n: int) -> int:
     return (n + 7) // 8 * 8
 
 
+def pad16(n: int) -> int:
+    return (n + 15) // 16 * 16
+
+
 class SourceTensors(Mapping):
     """``name -> tensor`` over the ``*.safetensors`` files of a directory; a tensor is streamed to ``device`` when it is looked up."""
 

@@ -74,21 +74,22 @@ class QkvConvArgs(C.Structure):
         ("state", C.c_void_p),
         ("row_pos", C.c_void_p), ("row_lane", C.c_void_p), ("row_active", C.c_void_p),
         ("rot", C.c_void_p), ("rot_dims", C.c_int),
-        ("q", C.c_void_p), ("k_new", C.c_void_p), ("v_new", C.c_void_p),
+        ("q", C.c_void_p), ("k_lin", C.c_void_p), ("v_lin", C.c_void_p),
         ("k_ring", C.c_void_p), ("v_ring", C.c_void_p), ("ring", C.c_int),
         ("v_first", C.c_void_p), ("v_mode", C.c_int), ("mix", C.c_float),
         ("H", C.c_int), ("G", C.c_int), ("dim", C.c_int), ("dimp", C.c_int), ("vdim", C.c_int), ("vdimp", C.c_int), ("rows", C.c_int),
-        ("decode", C.c_int), ("ring_from", C.c_int), ("capacity", C.c_int), ("lanes", C.c_int), ("rows_per_block", C.c_int),
+        ("decode", C.c_int), ("capacity", C.c_int), ("lanes", C.c_int), ("rows_per_block", C.c_int),
         ("status", C.c_void_p),
     ]
 
 
 class ChunkAttnArgs(C.Structure):
     _fields_ = [
-        ("q", C.c_void_p), ("k_new", C.c_void_p), ("v_new", C.c_void_p), ("k_ring", C.c_void_p), ("v_ring", C.c_void_p), ("sink", C.c_void_p),
+        ("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("sink", C.c_void_p),
         ("row_pos", C.c_void_p), ("row_lane", C.c_void_p), ("row_active", C.c_void_p),
         ("out", C.c_void_p), ("out_stride", C.c_int64),
         ("rows", C.c_int), ("H", C.c_int), ("G", C.c_int), ("dim", C.c_int), ("dimp", C.c_int), ("vdim", C.c_int), ("vdimp", C.c_int),
+        ("decode", C.c_int), ("start", C.c_int), ("base", C.c_int), ("keys", C.c_int),
         ("chunk", C.c_int), ("ring", C.c_int), ("capacity", C.c_int), ("lanes", C.c_int),
         ("scale", C.c_float),
         ("status", C.c_void_p),
@@ -439,19 +440,23 @@ def qkv_conv(args: QkvConvArgs, is_f32: bool) -> None:
     _check(lib().glmb_qkv_conv(C.byref(args), int(is_f32), _stream()), "qkv_conv")
 
 
-def ring_store(args: QkvConvArgs, first: int, is_f32: bool) -> None:
-    """Rows ``first ..`` of a step's linear key / value buffers into the lane's ring (``args`` of the ``qkv_conv`` that made them)."""
-    _check(lib().glmb_ring_store(C.c_void_p(args.k_new), C.c_void_p(args.v_new), C.c_void_p(args.row_pos), C.c_void_p(args.row_lane),
-                                 C.c_void_p(args.k_ring), C.c_void_p(args.v_ring), args.ring, args.G * args.dimp, args.G * args.vdimp, int(first),
-                                 args.rows, args.lanes, args.capacity, int(is_f32), _stream()), "ring_store")
+def kv_copy(k_src: int, k_dst: int, k_bytes: int, v_src: int, v_dst: int, v_bytes: int) -> None:
+    """Two contiguous runs of cache rows (addresses, bytes in multiples of 16) in one launch."""
+    _check(lib().glmb_kv_copy(C.c_void_p(k_src), C.c_void_p(k_dst), C.c_int64(k_bytes), C.c_void_p(v_src), C.c_void_p(v_dst), C.c_int64(v_bytes),
+                              _stream()), "kv_copy")
+
+
+def set_chunk_prefill_tc(enabled: int) -> None:
+    """1 (default): chunked prefill attention on tcgen05 where the head sizes allow; 0: on mma.sync."""
+    lib().glmb_set_chunk_prefill_tc(int(enabled))
 
 
 def chunk_attention(args: ChunkAttnArgs, is_f32: bool, *, plain: bool = False) -> None:
-    """Chunked causal attention with sinks.  bf16 heads up to 256 wide run on the tensor cores (``k_new`` set: prefill, otherwise decode);
+    """Chunked causal attention with sinks.  bf16 heads up to 256 wide run on the tensor cores (``args.decode`` says which);
     other head sizes, the 32-bit path and ``plain=True`` take the kernel that needs no particular size."""
-    if plain or is_f32 or max(args.dim, args.vdim) > 256:
+    if plain or is_f32 or max(args.dimp, args.vdimp) > 256:
         _check(lib().glmb_chunk_attn_any(C.byref(args), int(is_f32), _stream()), "chunk_attn_any")
-    elif args.k_new:
+    elif not args.decode:
         _check(lib().glmb_chunk_attn_prefill(C.byref(args), _stream()), "chunk_attn_prefill")
     else:
         _check(lib().glmb_chunk_attn_decode(C.byref(args), _stream()), "chunk_attn_decode")

@@ -9,7 +9,7 @@ import torch
 from glm_tpu_b200.config.cache import RingCacheConfig
 from glm_tpu_b200.exceptions import PlanValidationError
 from glm_tpu_b200.models.namizen.model import NamizenModel, NamizenWorkspace, RingState
-from glm_tpu_b200.models.namizen.weights import DeviceRandomTensors, NamizenWeights, pad8, resident_weights
+from glm_tpu_b200.models.namizen.weights import DeviceRandomTensors, NamizenWeights, pad8, pad16, resident_weights
 from glm_tpu_b200.parallel.peer import PeerGroup
 from glm_tpu_b200.runner.admission import project_live, project_ring_memory, require_admitted
 from glm_tpu_b200.runner.lane_runner import LaneRunner, RunnerReport
@@ -43,10 +43,12 @@ class NamizenRunner(LaneRunner):
 
     def _project(self, *, already_resident: int, mem_info=None) -> dict:
         g, item = self.g, self.cache.element_bytes
-        widest = max(pad8(m.qkv_width) + m.heads * pad8(m.dim) + 3 * m.kv_heads * pad8(max(m.dim, m.vdim)) + pad8(m.out_width) + 3 * pad8(layer.ff)
-                     for layer in g.layers for m in (layer.mixer,))
         rows = self.lanes + self.prefill_chunk
-        workspace = rows * (pad8(g.hidden_size) * (8 + 2 * item) + widest * item) + self.lanes * pad8(g.vocab_size) * 4
+        widest = max(pad8(m.qkv_width) + m.heads * pad16(m.dim) + m.kv_heads * pad16(m.vdim) + pad8(m.out_width) + 3 * pad8(layer.ff)
+                     for layer in g.layers for m in (layer.mixer,))
+        linear = max(self.cache.linear_rows(i, self.prefill_chunk) * m.kv_heads * (pad16(m.dim) + pad16(m.vdim))
+                     for i, layer in enumerate(g.layers) for m in (layer.mixer,))
+        workspace = rows * (pad8(g.hidden_size) * (8 + 2 * item) + widest * item) + linear * item + self.lanes * pad8(g.vocab_size) * 4
         rot = {(layer.mixer.rot_dims, layer.mixer.rot_base) for layer in g.layers}
         workspace += sum(dims * 4 * self.cache.context_capacity for dims, _ in rot)
         projection = project_ring_memory(self.cache, self.weights.bytes_resident, workspace)
