@@ -82,8 +82,8 @@ class NamizenGeometry:
         if self.vocab_size < 1 or self.hidden_size < 1 or not self.layers:
             raise ConfigValidationError("a Namizen model has a vocabulary, a width and at least one layer")
         mixing = [layer.mixer for layer in self.layers if layer.mixer.v_mix]
-        if any((m.kv_heads, m.vdim) != (mixing[0].kv_heads, mixing[0].vdim) for m in mixing):
-            raise ConfigValidationError("layers that mix values need the value heads of the first such layer")
+        if any(m.v_width != mixing[0].v_width for m in mixing):
+            raise ConfigValidationError("layers that mix values need as many value channels as the first such layer")
 
     @property
     def num_layers(self) -> int:

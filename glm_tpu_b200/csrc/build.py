@@ -67,7 +67,7 @@ def build(verbose: bool = False, force: bool = False, component: str | None = No
     with ThreadPoolExecutor(max_workers=min(8, len(sources) or 1)) as pool:
         objects = list(pool.map(compile_one, sources))
     if force or _stale(target, objects):
-        cmd = [NVCC, "-shared", "-o", str(target), *map(str, objects), "-lcudart"]
+        cmd = [NVCC, "-shared", "-Xlinker", "--no-undefined", "-o", str(target), *map(str, objects), "-lcudart"]
         done = subprocess.run(cmd, capture_output=True, text=True)
         if done.returncode != 0:
             raise RuntimeError(f"link failed:\n{done.stdout}\n{done.stderr}")

@@ -58,6 +58,13 @@ struct PeerComm {
     uint32_t* flags[GLMB_MAX_WORLD];  // flags[p]: rank p's flag buffer as mapped here
 };
 
+// The comm of a kernel that runs alone (no peers).
+static inline PeerComm single_comm() {
+    PeerComm c = {};
+    c.world = 1;
+    return c;
+}
+
 __device__ __forceinline__ void st_release_sys(uint32_t* p, uint32_t v) {
     asm volatile("st.release.sys.global.u32 [%0], %1;" ::"l"(p), "r"(v) : "memory");
 }

@@ -32,7 +32,7 @@ struct QkvConvArgs {
     void* q;                                     // [rows, H, dimp]
     void *k_lin, *v_lin;                         // [rows, G, dimp], [rows, G, vdimp], or NULL: keys and values go to the ring
     void *k_ring, *v_ring; int ring;             // [lanes, ring, G, dimp], [lanes, ring, G, vdimp]
-    void* v_first; int v_mode; float mix;        // [rows, G, vdimp]; 0: not used, 1: store this layer's values, 2: mix with them
+    void* v_first; int v_mode; float mix;        // [rows, G * vdim]; 0: not used, 1: store this layer's values, 2: mix with them
     int H, G, dim, dimp, vdim, vdimp, rows, decode, capacity, lanes, rows_per_block;
     uint32_t* status;
 };
@@ -76,15 +76,26 @@ __device__ __forceinline__ void qc_store(const QkvConvArgs& a, const QcHead& h, 
         return;
     }
     const int64_t at = ((int64_t)row * a.G + h.slot) * h.hdp + c;
-    if (h.kind == 2 && a.v_mode) {
-        T* vf = reinterpret_cast<T*>(a.v_first) + at;
-        if (a.v_mode == 1) {
-            store8(vf, o);
+    if (h.kind == 2 && a.v_mode) {  // by channel, whatever the heads: layers may cut the same channels into other heads
+        T* vf = reinterpret_cast<T*>(a.v_first) + ((int64_t)row * a.G + h.slot) * h.hd + c;
+        float f[8];
+        if (!(h.hd & 7)) {
+            if (c < h.hd) {
+                if (a.v_mode == 1) store8(vf, o);
+                else load8(vf, f);
+            }
         } else {
-            float f[8];
-            load8(vf, f);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) o[e] = (1.f - a.mix) * o[e] + a.mix * f[e];
+            for (int e = 0; e < 8; ++e)
+                if (c + e < h.hd) {
+                    if (a.v_mode == 1) from_f32(o[e], vf[e]);
+                    else f[e] = to_f32(vf[e]);
+                }
+        }
+        if (a.v_mode == 2) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e)
+                if (c + e < h.hd) o[e] = (1.f - a.mix) * o[e] + a.mix * f[e];
         }
     }
     T* lin = reinterpret_cast<T*>(h.kind == 1 ? a.k_lin : a.v_lin);

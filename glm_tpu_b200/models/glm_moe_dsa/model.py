@@ -677,7 +677,7 @@ class GlmMoeDsaModel:
 
     # ------------------------------------------------------------------------------ whole model
     def run_rows(self, ws: Workspace, state: DecoderState, tokens: torch.Tensor, row_pos: torch.Tensor, row_lane: torch.Tensor,
-                 row_active, rows: int, *, decode: bool, max_ctx: int, head_rows: slice | None = None, head: str = "logits",
+                 row_active, rows: int, *, decode: bool, max_ctx: int, head_rows: slice | torch.Tensor | None = None, head: str = "logits",
                  lane_of_rows: int | None = None):
         """Push ``rows`` token rows through the decoder.
 
@@ -706,7 +706,7 @@ class GlmMoeDsaModel:
             if self.trace is not None:
                 self.trace.setdefault("update", {})[i] = ws.update[:rows].clone()
         native.add_rmsnorm(update, ws.residual[:rows], self.w.final_norm, ws.x, g.rms_norm_eps)
-        hs = head_rows or slice(0, rows)
+        hs = slice(0, rows) if head_rows is None else head_rows  # a slice, or an index tensor
         xh = ws.x[hs]
         n = xh.shape[0]
         if head == "argmax":

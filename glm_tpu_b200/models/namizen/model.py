@@ -69,7 +69,7 @@ class NamizenWorkspace:
         lin = [model.cache.linear_rows(i, rows) if prefill else 0 for i in range(g.num_layers)]
         self.k_lin = t(max(n * m.kv_heads * pad16(m.dim) for n, m in zip(lin, mixers)))
         self.v_lin = t(max(n * m.kv_heads * pad16(m.vdim) for n, m in zip(lin, mixers)))
-        self.v_first = t(rows * max([m.kv_heads * pad16(m.vdim) for m in mixers if m.v_mix] or [8]))
+        self.v_first = t(rows * max([m.v_width for m in mixers if m.v_mix] or [8]))
         self.gate_up = t(rows * 2 * max(lw.ff_cols for lw in model.w.layers)) if prefill or model.is_f32 else None
         self.logits = torch.zeros((rows if not prefill else 0, pad8(g.vocab_size)), dtype=torch.float32, device=dev)
         self.local_best = torch.zeros(rows, dtype=torch.int64, device=dev)

@@ -68,16 +68,16 @@ def attention(h: torch.Tensor, mixer: dict, weight, first_values: torch.Tensor |
     heads, groups, dim, vdim = mixer["heads"], mixer["kv_heads"], mixer["dim"], mixer["vdim"]
     total = h.shape[0]
     q, k, v = (causal_conv(h @ weight(n).T, weight(n + ".conv")) for n in ("q", "k", "v"))
-    rot = mixer["rot"]
-    q = rotate_half(q.reshape(total, heads, dim), rot["dims"], rot["base"])
-    k = rotate_half(k.reshape(total, groups, dim), rot["dims"], rot["base"])
+    q, k = q.reshape(total, heads, dim), k.reshape(total, groups, dim)
+    if mixer.get("rot"):
+        q, k = (rotate_half(x, mixer["rot"]["dims"], mixer["rot"]["base"]) for x in (q, k))
     v = own = v.reshape(total, groups, vdim)
     if first_values is not None:
-        v = mix_values(v, first_values, weight("vmix"))
+        v = mix_values(v, first_values.reshape(total, groups, vdim), weight("vmix"))  # channel by channel, whatever the heads
     per = heads // groups
     k, v = k.repeat_interleave(per, dim=1), v.repeat_interleave(per, dim=1)
     scores = torch.einsum("ihd,jhd->hij", q, k) * mixer["scale"]
-    p = sink_softmax(scores, weight("sink"), chunk_mask(total, mixer["mask"]["size"]))
+    p = sink_softmax(scores, weight("sink"), chunk_mask(total, mixer["mask"]["size"] if mixer.get("mask") else total))
     out = torch.einsum("hij,jhd->ihd", p, v).reshape(total, heads * vdim)
     return out @ weight("o").T, own
 
