@@ -222,36 +222,30 @@ __global__ void __launch_bounds__(CP_THREADS) chunk_attn_prefill_kernel(ChunkAtt
 }
 
 // ---------------------------------------------------------------------------------------------------
-#define CD_WARPS 4
-#define CD_THREADS (CD_WARPS * 32)
 #define CD_HEADS 16
-#define CD_KEYS 64  // keys of a tile, 16 per warp
-#define CD_BOX (CD_KEYS * 128)  // bytes of a tile's 64-column box: 128-byte rows, 128-byte swizzle
+// A tile is 16 keys per warp: WARPS * 16 keys, in 64-column boxes of 128-byte rows (128-byte swizzle).
 
 static inline int cd_boxes(int padded) { return (padded + 63) / 64; }
-static inline size_t chunk_decode_smem(int dk, int dv, int stages) {
-    const size_t tiles = (size_t)stages * (cd_boxes(dk) + cd_boxes(dv)) * CD_BOX, merge = (size_t)CD_WARPS * CD_HEADS * dv * 4;
+static inline size_t chunk_decode_smem(int dk, int dv, int stages, int warps) {
+    const size_t tiles = (size_t)stages * (cd_boxes(dk) + cd_boxes(dv)) * warps * 16 * 128, merge = (size_t)warps * CD_HEADS * dv * 4;
     return 1024 + (tiles > merge ? tiles : merge) + (size_t)CD_HEADS * (dk + 8) * 2;
-}
-// 16-byte piece `c` of row `r` of a swizzled tile made of 64-column boxes
-__device__ __forceinline__ const unsigned char* cd_piece(const unsigned char* tile, int r, int c) {
-    return tile + (c >> 3) * CD_BOX + r * 128 + (((c & 7) ^ (r & 7)) << 4);
 }
 
 // grid (splits, key heads x blocks of 16 query heads, rows), cluster (splits, 1, 1).
-template <int DV>
-__global__ void __launch_bounds__(CD_THREADS)
+template <int DV, int WARPS>
+__global__ void __launch_bounds__(WARPS * 32)
 chunk_attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, ChunkAttnArgs a, int stages) {
+    constexpr int KEYS = WARPS * 16, BOX = KEYS * 128;
     cg::cluster_group cluster = cg::this_cluster();
     extern __shared__ unsigned char smem_raw[];
-    __shared__ float ml_s[CD_WARPS][CD_HEADS][2];  // (maximum, sum) per warp
-    __shared__ float cta_ml[CD_HEADS][2];
+    __shared__ float ml_s[WARPS][CD_HEADS][2];  // (maximum, sum) per warp
+    __shared__ __align__(8) float cta_ml[CD_HEADS][2];
     __shared__ __align__(8) uint64_t full_bar[4];
     const int dk = a.dimp, dv = a.vdimp, KP = dk + 8;
     const int kboxes = (dk + 63) / 64, vboxes = (dv + 63) / 64;
     unsigned char* tiles_s = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
-    const size_t stage_bytes = (size_t)(kboxes + vboxes) * CD_BOX;
-    const size_t tile_area = stages * stage_bytes, merge_area = (size_t)CD_WARPS * CD_HEADS * dv * 4;
+    const size_t stage_bytes = (size_t)(kboxes + vboxes) * BOX;
+    const size_t tile_area = stages * stage_bytes, merge_area = (size_t)WARPS * CD_HEADS * dv * 4;
     bf16* q_s = reinterpret_cast<bf16*>(tiles_s + (tile_area > merge_area ? tile_area : merge_area));
     if (threadIdx.x == 0) {
         for (int s = 0; s < stages; ++s) mbar_init(full_bar + s, 1);
@@ -267,22 +261,22 @@ chunk_attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
     const int pos = ca_pos(a, row), lane_id = ca_lane(a, row);
     const int keys = active ? pos % a.chunk + 1 : 0;  // slots 0 .. keys - 1 of the lane's ring
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3, mr = lane & 7, mi = lane >> 3;
-    const int tiles = (keys + CD_KEYS - 1) / CD_KEYS, mine = tiles > split ? (tiles - split - 1) / splits + 1 : 0;  // tiles split, split + splits, ..
+    const int tiles = (keys + KEYS - 1) / KEYS, mine = tiles > split ? (tiles - split - 1) / splits + 1 : 0;  // tiles split, split + splits, ..
 
     auto load_tile = [&](int i) {  // the i-th tile of this CTA, by one thread
         unsigned char* dst = tiles_s + (size_t)(i % stages) * stage_bytes;
         uint64_t* bar = full_bar + i % stages;
-        const int y = lane_id * a.ring + (split + i * splits) * CD_KEYS;
+        const int y = lane_id * a.ring + (split + i * splits) * KEYS;
         mbar_expect_tx(bar, (uint32_t)stage_bytes);
-        for (int b = 0; b < kboxes; ++b) tma_load_2d(dst + b * CD_BOX, &map_k, bar, group * dk + b * 64, y);
-        for (int b = 0; b < vboxes; ++b) tma_load_2d(dst + (kboxes + b) * CD_BOX, &map_v, bar, group * dv + b * 64, y);
+        for (int b = 0; b < kboxes; ++b) tma_load_2d(dst + b * BOX, &map_k, bar, group * dk + b * 64, y);
+        for (int b = 0; b < vboxes; ++b) tma_load_2d(dst + (kboxes + b) * BOX, &map_v, bar, group * dv + b * 64, y);
     };
     if (threadIdx.x == 0)
         for (int i = 0; i < min(stages, mine); ++i) load_tile(i);
     {
         const bf16* q = reinterpret_cast<const bf16*>(a.q) + ((int64_t)row * a.H + h0) * dk;
         const int pieces = dk / 8;
-        for (int i = threadIdx.x; i < CD_HEADS * pieces; i += CD_THREADS) {
+        for (int i = threadIdx.x; i < CD_HEADS * pieces; i += WARPS * 32) {
             const int r = i / pieces, c = i % pieces;
             *reinterpret_cast<uint4*>(q_s + r * KP + c * 8) = r < heads ? *reinterpret_cast<const uint4*>(q + (int64_t)r * dk + c * 8) : make_uint4(0, 0, 0, 0);
         }
@@ -295,29 +289,43 @@ chunk_attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
 #pragma unroll
     for (int j = 0; j < DV / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
     const bf16* qa = q_s + (mr + 8 * (mi & 1)) * KP + 8 * (mi >> 1);
+    // this lane's rows of a key / value fragment and its 16-byte pieces of a 128-byte row, as they lie swizzled
+    const int k_row = (mr + 8 * (mi >> 1)) * 128, v_row = (mr + 8 * (mi & 1)) * 128;
+    int k_col[4], v_col[4];
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+        k_col[c] = ((2 * c + (mi & 1)) ^ mr) << 4;
+        v_col[c] = ((2 * c + (mi >> 1)) ^ mr) << 4;
+    }
+    bool ok = true;
     for (int i = 0; i < mine; ++i) {
-        const int stage = i % stages, slot0 = (split + i * splits) * CD_KEYS;
-        if (!mbar_wait(full_bar + stage, (i / stages) & 1)) {
+        const int stage = i % stages, slot0 = (split + i * splits) * KEYS;
+        if (ok && !mbar_wait(full_bar + stage, (i / stages) & 1)) {
             if (lane == 0) raise_status(a.status, GLMB_STATUS_WAIT_TIMEOUT);
-            break;
+            ok = false;  // no more work for this warp, but it still meets the others at their barriers
         }
         unsigned char* kt = tiles_s + (size_t)stage * stage_bytes;
-        unsigned char* vt = kt + kboxes * CD_BOX;
-        const int w0 = warp * 16, left = keys - slot0 - w0;  // this warp's keys of the tile, how many of them exist
+        unsigned char* vt = kt + kboxes * BOX;
+        const int w0 = warp * 16, left = ok ? keys - slot0 - w0 : 0;  // this warp's keys of the tile, how many of them exist
         if (left > 0 && left < 16) {  // values past the last key meet zero weights: they must not be infinite or NaN
             for (int x = lane; x < (16 - left) * vboxes * 8; x += 32)
-                *reinterpret_cast<uint4*>(const_cast<unsigned char*>(cd_piece(vt, w0 + left + x / (vboxes * 8), x % (vboxes * 8)))) = make_uint4(0, 0, 0, 0);
+                *reinterpret_cast<uint4*>(vt + (x % (vboxes * 8) >> 3) * BOX + (w0 + left + x / (vboxes * 8)) * 128 + (x & 7) * 16) = make_uint4(0, 0, 0, 0);
             __syncwarp();
         }
         if (left > 0) {
             float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-            for (int k0 = 0; k0 < dk; k0 += 16) {
-                uint32_t qf[4], kf[4];
-                ldmatrix_x4(qf, qa + k0);
-                ldmatrix_x4(kf, cd_piece(kt, w0 + mr + 8 * (mi >> 1), k0 / 8 + (mi & 1)));
-                mma_bf16_16816(s[0], qf, kf[0], kf[1]);
-                mma_bf16_16816(s[1], qf, kf[2], kf[3]);
-            }
+            const bf16* qk = qa;
+            const unsigned char* kb = kt + w0 * 128 + k_row;
+            for (int k0 = 0; k0 < dk; k0 += 64, kb += BOX, qk += 64)
+#pragma unroll
+                for (int c = 0; c < 4; ++c)
+                    if (k0 + c * 16 < dk) {
+                        uint32_t qf[4], kf[4];
+                        ldmatrix_x4(qf, qk + c * 16);
+                        ldmatrix_x4(kf, kb + k_col[c]);
+                        mma_bf16_16816(s[0], qf, kf[0], kf[1]);
+                        mma_bf16_16816(s[1], qf, kf[2], kf[3]);
+                    }
             float mx[2] = {m[0], m[1]};
 #pragma unroll
             for (int j = 0; j < 2; ++j)
@@ -356,7 +364,7 @@ chunk_attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
                     o[j][0] *= fix[0]; o[j][1] *= fix[0]; o[j][2] *= fix[1]; o[j][3] *= fix[1];
                     o[j + 1][0] *= fix[0]; o[j + 1][1] *= fix[0]; o[j + 1][2] *= fix[1]; o[j + 1][3] *= fix[1];
                     uint32_t vf[4];
-                    ldmatrix_x4_trans(vf, cd_piece(vt, w0 + mr + 8 * (mi & 1), j + (mi >> 1)));
+                    ldmatrix_x4_trans(vf, vt + (j >> 3) * BOX + w0 * 128 + v_row + v_col[(j & 7) >> 1]);
                     mma_bf16_16816(o[j], hi, vf[0], vf[1]);
                     mma_bf16_16816(o[j + 1], hi, vf[2], vf[3]);
                     mma_bf16_16816(o[j], lw, vf[0], vf[1]);
@@ -387,39 +395,54 @@ chunk_attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
     // ---- warps of the CTA into warp 0's area ------------------------------------------------------------
     if (threadIdx.x < CD_HEADS) {
         float top = -INFINITY, sum = 0.f;
-        for (int w = 0; w < CD_WARPS; ++w) top = fmaxf(top, ml_s[w][threadIdx.x][0]);
-        for (int w = 0; w < CD_WARPS; ++w)
+        for (int w = 0; w < WARPS; ++w) top = fmaxf(top, ml_s[w][threadIdx.x][0]);
+        for (int w = 0; w < WARPS; ++w)
             if (ml_s[w][threadIdx.x][0] != -INFINITY) sum += ml_s[w][threadIdx.x][1] * exp2f(ml_s[w][threadIdx.x][0] - top);
         cta_ml[threadIdx.x][0] = top;
         cta_ml[threadIdx.x][1] = sum;
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < CD_HEADS * dv; i += CD_THREADS) {
+    for (int i = threadIdx.x; i < CD_HEADS * dv; i += WARPS * 32) {
         const int h = i / dv;
         const float top = cta_ml[h][0];
         float v = 0.f;
-        for (int w = 0; w < CD_WARPS; ++w)
+        for (int w = 0; w < WARPS; ++w)
             if (ml_s[w][h][0] != -INFINITY) v += o_s[(size_t)w * CD_HEADS * dv + i] * exp2f(ml_s[w][h][0] - top);
         o_s[i] = v;
     }
     cluster.sync();
     // ---- CTAs of the cluster: each finishes its share of the outputs, the sink joins here -----------------
-    const int total = heads * a.vdim;
-    bf16* out = reinterpret_cast<bf16*>(a.out) + (int64_t)row * a.out_stride + (int64_t)h0 * a.vdim;
-    for (int i = split * CD_THREADS + threadIdx.x; i < total; i += splits * CD_THREADS) {
-        const int h = i / a.vdim, c = i % a.vdim;
+    // First every CTA's (maximum, sum) of every head, all loads at once, then a weight per CTA and head.
+    __shared__ float part_s[16][CD_HEADS][2];
+    for (int i = threadIdx.x; i < splits * CD_HEADS; i += WARPS * 32) {
+        const float2 ml = *reinterpret_cast<const float2*>(cluster.map_shared_rank(&cta_ml[0][0], i / CD_HEADS) + (i % CD_HEADS) * 2);
+        part_s[i / CD_HEADS][i % CD_HEADS][0] = ml.x;
+        part_s[i / CD_HEADS][i % CD_HEADS][1] = ml.y;
+    }
+    __syncthreads();
+    if ((int)threadIdx.x < heads) {
+        const int h = threadIdx.x;
         const float sink2 = a.sink ? a.sink[h0 + h] * CA_LOG2E : -INFINITY;
         float top = sink2;
-        for (int p = 0; p < splits; ++p) top = fmaxf(top, cluster.map_shared_rank(&cta_ml[0][0], p)[h * 2]);
-        float sum = a.sink ? exp2f(sink2 - top) : 0.f, v = 0.f;
+        for (int p = 0; p < splits; ++p) top = fmaxf(top, part_s[p][h][0]);
+        float sum = a.sink ? exp2f(sink2 - top) : 0.f;
         for (int p = 0; p < splits; ++p) {
-            const float* pml = cluster.map_shared_rank(&cta_ml[0][0], p);
-            if (pml[h * 2] == -INFINITY) continue;
-            const float w = exp2f(pml[h * 2] - top);
-            sum += pml[h * 2 + 1] * w;
-            v += cluster.map_shared_rank(o_s, p)[h * dv + c] * w;
+            const float w = part_s[p][h][0] == -INFINITY ? 0.f : exp2f(part_s[p][h][0] - top);
+            sum += part_s[p][h][1] * w;
+            part_s[p][h][0] = w;
         }
-        out[i] = __float2bfloat16_rn(sum > 0.f ? v / sum : 0.f);
+        const float inv = sum > 0.f ? 1.f / sum : 0.f;
+        for (int p = 0; p < splits; ++p) part_s[p][h][0] *= inv;
+    }
+    __syncthreads();
+    const int total = heads * a.vdim;
+    bf16* out = reinterpret_cast<bf16*>(a.out) + (int64_t)row * a.out_stride + (int64_t)h0 * a.vdim;
+    for (int i = split * WARPS * 32 + threadIdx.x; i < total; i += splits * WARPS * 32) {
+        const int h = i / a.vdim, c = i % a.vdim;
+        float v = 0.f;
+#pragma unroll 16
+        for (int p = 0; p < splits; ++p) v = fmaf(cluster.map_shared_rank(o_s, p)[h * dv + c], part_s[p][h][0], v);
+        out[i] = __float2bfloat16_rn(v);
     }
     cluster.sync();  // nobody leaves while a peer may still read its shared memory
 }
@@ -527,32 +550,32 @@ static int launch_chunk_prefill(const ChunkAttnArgs& a, cudaStream_t st) {
     return (int)cudaGetLastError();
 }
 
-template <int DV>
+template <int DV, int WARPS>
 static int launch_chunk_decode(const ChunkAttnArgs& a, cudaStream_t st) {
     static DeviceOnce once;
-    cudaError_t e = chunk_smem_limit(chunk_attn_decode_kernel<DV>, once);
+    cudaError_t e = chunk_smem_limit(chunk_attn_decode_kernel<DV, WARPS>, once);
     if (e != cudaSuccess) return (int)e;
     static DeviceOnce wide;  // clusters of 16 are beyond the portable size
     const int wide_dev = wide.pending();
     if (wide_dev != DeviceOnce::SET) {
-        e = cudaFuncSetAttribute(chunk_attn_decode_kernel<DV>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+        e = cudaFuncSetAttribute(chunk_attn_decode_kernel<DV, WARPS>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
         if (e != cudaSuccess) return (int)e;
         wide.mark(wide_dev);
     }
     CUtensorMap map_k, map_v;
     const uint64_t ring_rows = (uint64_t)a.lanes * a.ring;
-    if (make_map(&map_k, a.k, ring_rows, (uint64_t)a.G * a.dimp, (uint64_t)a.G * a.dimp, CD_KEYS)) return 3;
-    if (make_map(&map_v, a.v, ring_rows, (uint64_t)a.G * a.vdimp, (uint64_t)a.G * a.vdimp, CD_KEYS)) return 3;
+    if (make_map(&map_k, a.k, ring_rows, (uint64_t)a.G * a.dimp, (uint64_t)a.G * a.dimp, WARPS * 16)) return 3;
+    if (make_map(&map_v, a.v, ring_rows, (uint64_t)a.G * a.vdimp, (uint64_t)a.G * a.vdimp, WARPS * 16)) return 3;
     int stages = 4;
-    while (stages > 2 && chunk_decode_smem(a.dimp, a.vdimp, stages) > 112 * 1024) --stages;
+    while (stages > 2 && chunk_decode_smem(a.dimp, a.vdimp, stages, WARPS) > 200 * 1024) --stages;
     // CTAs per cluster: enough that the grid reaches every SM, at least one tile each
-    const int heads = a.G * ceil_div(a.H / a.G, CD_HEADS), tiles = ceil_div(a.ring, CD_KEYS);
+    const int heads = a.G * ceil_div(a.H / a.G, CD_HEADS), tiles = ceil_div(a.ring, WARPS * 16);
     int splits = 1;
     while (splits < 16 && splits * 2 <= tiles && splits * heads * a.rows < 148) splits *= 2;
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(splits, heads, a.rows);
-    cfg.blockDim = dim3(CD_THREADS);
-    cfg.dynamicSmemBytes = chunk_decode_smem(a.dimp, a.vdimp, stages);
+    cfg.blockDim = dim3(WARPS * 32);
+    cfg.dynamicSmemBytes = chunk_decode_smem(a.dimp, a.vdimp, stages, WARPS);
     cfg.stream = st;
     cudaLaunchAttribute attr[2];
     attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
@@ -562,7 +585,7 @@ static int launch_chunk_decode(const ChunkAttnArgs& a, cudaStream_t st) {
     attr[1].val.clusterDim.y = attr[1].val.clusterDim.z = 1;
     cfg.attrs = attr;
     cfg.numAttrs = 2;
-    const cudaError_t le = cudaLaunchKernelEx(&cfg, chunk_attn_decode_kernel<DV>, map_k, map_v, a, stages);
+    const cudaError_t le = cudaLaunchKernelEx(&cfg, chunk_attn_decode_kernel<DV, WARPS>, map_k, map_v, a, stages);
     return le != cudaSuccess ? (int)le : (int)cudaGetLastError();
 }
 
@@ -586,9 +609,10 @@ GLMB_API int glmb_chunk_attn_prefill(const ChunkAttnArgs* args, void* stream) {
 GLMB_API int glmb_chunk_attn_decode(const ChunkAttnArgs* args, void* stream) {
     const ChunkAttnArgs a = *args;
     if (!chunk_args_ok(a) || !a.decode || a.dimp > 256 || a.vdimp > 256) return 1;
-    if (a.vdimp <= 64) return launch_chunk_decode<64>(a, (cudaStream_t)stream);
-    if (a.vdimp <= 128) return launch_chunk_decode<128>(a, (cudaStream_t)stream);
-    return launch_chunk_decode<256>(a, (cudaStream_t)stream);
+    if (a.dimp > 128) return launch_chunk_decode<256, 4>(a, (cudaStream_t)stream);
+    if (a.vdimp <= 64) return launch_chunk_decode<64, 8>(a, (cudaStream_t)stream);
+    if (a.vdimp <= 128) return launch_chunk_decode<128, 8>(a, (cudaStream_t)stream);
+    return launch_chunk_decode<256, 4>(a, (cudaStream_t)stream);
 }
 
 // Any head size (values up to 1024 columns), bf16 or fp32.

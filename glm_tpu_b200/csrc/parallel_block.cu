@@ -15,27 +15,29 @@
 #include "gemv_core.cuh"
 #include "vec8.cuh"
 
-#define PN_THREADS 256
-#define PN_REGS 2  // 8-element vectors of a row each thread keeps in registers (2 x 8 x 256 = 4096 columns); wider rows are read again
+// THREADS x REGS 8-element vectors of a row stay in registers (4096 columns either way); wider rows are read again.  Few rows: more threads
+// per row, and the weights are asked for before the sum of squares is known; many rows: smaller CTAs, more of them per SM.
+#define PN_FEW_ROWS 16
 
+template <int THREADS>
 __device__ __forceinline__ float pn_block_sum(float v, float* scratch) {
     v = warp_sum(v);
     if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = v;
     __syncthreads();
     float t = 0.f;
 #pragma unroll
-    for (int w = 0; w < PN_THREADS / 32; ++w) t += scratch[w];
+    for (int w = 0; w < THREADS / 32; ++w) t += scratch[w];
     return t;
 }
 
 // One CTA per row.  `padded` columns are stored (a multiple of 8, zeros past `width`); the mean is over `width`.
-template <typename T>
-__global__ void __launch_bounds__(PN_THREADS)
+template <typename T, int THREADS, int REGS>
+__global__ void __launch_bounds__(THREADS)
 parallel_norm_kernel(const int* __restrict__ tokens, const T* __restrict__ table, int vocab, const float* __restrict__ update,
                      float* __restrict__ residual, int width, int padded, const T* __restrict__ w1, const T* __restrict__ w2,
                      T* __restrict__ out1, T* __restrict__ out2, float eps, uint32_t* status) {
     GLMB_PDL_PROLOGUE();
-    __shared__ float scratch[PN_THREADS / 32];
+    __shared__ float scratch[THREADS / 32];
     const int64_t base = (int64_t)blockIdx.x * padded;
     float* res = residual + base;
     const T* source = nullptr;
@@ -47,10 +49,15 @@ parallel_norm_kernel(const int* __restrict__ tokens, const T* __restrict__ table
         }
         source = table + (int64_t)id * padded;
     }
-    float keep[PN_REGS][8];
+    float keep[REGS][8], wa[8], wb[8];
+    constexpr bool early = REGS == 1;
+    if (early && (int)threadIdx.x * 8 < padded) {  // the weights of the first vector
+        load8(w1 + threadIdx.x * 8, wa);
+        if (w2) load8(w2 + threadIdx.x * 8, wb);
+    }
     float ss = 0.f;
     int slot = 0;
-    for (int v = threadIdx.x * 8; v < padded; v += PN_THREADS * 8, ++slot) {
+    for (int v = threadIdx.x * 8; v < padded; v += THREADS * 8, ++slot) {
         float x[8];
         if (source) {
             load8(source + v, x);
@@ -67,36 +74,36 @@ parallel_norm_kernel(const int* __restrict__ tokens, const T* __restrict__ table
 #pragma unroll
         for (int e = 0; e < 8; ++e) ss = fmaf(x[e], x[e], ss);
 #pragma unroll
-        for (int s = 0; s < PN_REGS; ++s)
+        for (int s = 0; s < REGS; ++s)
             if (s == slot)
 #pragma unroll
                 for (int e = 0; e < 8; ++e) keep[s][e] = x[e];
     }
-    const float mean = pn_block_sum(ss, scratch) / (float)width;
+    const float mean = pn_block_sum<THREADS>(ss, scratch) / (float)width;
     const float denom = sqrtf(mean + eps);
     slot = 0;
-    for (int v = threadIdx.x * 8; v < padded; v += PN_THREADS * 8, ++slot) {
+    for (int v = threadIdx.x * 8; v < padded; v += THREADS * 8, ++slot) {
         float x[8];
-        if (slot < PN_REGS) {
+        if (slot < REGS) {
 #pragma unroll
-            for (int s = 0; s < PN_REGS; ++s)
+            for (int s = 0; s < REGS; ++s)
                 if (s == slot)
 #pragma unroll
                     for (int e = 0; e < 8; ++e) x[e] = keep[s][e];
         } else {
             load8(res + v, x);  // written by this same thread above
         }
-        float a[8], y[8];
+        float y[8];
 #pragma unroll
         for (int e = 0; e < 8; ++e) x[e] = x[e] / denom;
-        load8(w1 + v, a);
+        if (slot || !early) load8(w1 + v, wa);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) y[e] = x[e] * a[e];
+        for (int e = 0; e < 8; ++e) y[e] = x[e] * wa[e];
         store8(out1 + base + v, y);
         if (w2) {
-            load8(w2 + v, a);
+            if (slot || !early) load8(w2 + v, wb);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) y[e] = x[e] * a[e];
+            for (int e = 0; e < 8; ++e) y[e] = x[e] * wb[e];
             store8(out2 + base + v, y);
         }
     }
@@ -181,12 +188,18 @@ GLMB_API int glmb_parallel_norm(const int* tokens, const void* table, int vocab,
                                 int padded, const void* w1, const void* w2, void* out1, void* out2, float eps, int is_f32, uint32_t* status,
                                 void* stream) {
     if (rows < 1 || width < 1 || padded < width || (padded & 7) || (tokens && update) || (tokens && (!table || vocab < 1)) || (w2 && !out2)) return 1;
-    if (is_f32)
-        GLMB_LAUNCH(parallel_norm_kernel<float>, rows, PN_THREADS, 0, (cudaStream_t)stream, tokens, (const float*)table, vocab, update, residual, width,
-                    padded, (const float*)w1, (const float*)w2, (float*)out1, (float*)out2, eps, status);
-    else
-        GLMB_LAUNCH(parallel_norm_kernel<bf16>, rows, PN_THREADS, 0, (cudaStream_t)stream, tokens, (const bf16*)table, vocab, update, residual, width,
-                    padded, (const bf16*)w1, (const bf16*)w2, (bf16*)out1, (bf16*)out2, eps, status);
+    cudaStream_t st = (cudaStream_t)stream;
+#define CALL(T, THREADS, REGS)                                                                                                             \
+    GLMB_LAUNCH((parallel_norm_kernel<T, THREADS, REGS>), rows, THREADS, 0, st, tokens, (const T*)table, vocab, update, residual, width, padded, \
+                (const T*)w1, (const T*)w2, (T*)out1, (T*)out2, eps, status)
+    if (rows <= PN_FEW_ROWS) {
+        if (is_f32) CALL(float, 512, 1);
+        else CALL(bf16, 512, 1);
+    } else {
+        if (is_f32) CALL(float, 256, 2);
+        else CALL(bf16, 256, 2);
+    }
+#undef CALL
     return (int)cudaGetLastError();
 }
 

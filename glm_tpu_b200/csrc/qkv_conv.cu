@@ -11,8 +11,8 @@
 // other block reads it: a block holds at least taps - 1 rows).  Decode: every row is its own sequence (lane), one row per block.
 //
 //   qkv_conv_kernel       any sizes, decode and prefill: convolution into shared memory, then rotation / mixing / stores
-//   qkv_conv_rows_kernel  prefill, head sizes in multiples of 8, up to 4 taps: a thread slides down a strip of rows with two 8-channel
-//                         vectors (for rotated dimensions the two halves of a pair), its taps and its window in registers
+//   qkv_conv_rows_kernel  prefill, head sizes in multiples of 8, up to 4 taps: a thread takes a strip of rows with two 8-channel
+//                         vectors (for rotated dimensions the two halves of a pair), its taps, rows and history in registers
 //
 // Keys and values go to the lane's ring (slot = position mod ring size: with chunked attention a ring of one chunk holds everything a later
 // token can see) or, when `k_lin` is set, to linear buffers, row by row.
@@ -178,7 +178,31 @@ __global__ void __launch_bounds__(QC_THREADS) qkv_conv_kernel(QkvConvArgs a) {
 
 // ---------------------------------------------------------------------------------------------------
 #define QR_TAPS 4
-#define QR_STRIP 8  // rows a thread slides over
+#define QR_STRIP 4  // consecutive rows of a thread
+
+// Eight elements as they come from memory.
+template <typename T> struct Raw8;
+template <> struct Raw8<bf16> {
+    uint4 v;
+    __device__ __forceinline__ void clear() { v = make_uint4(0, 0, 0, 0); }
+    __device__ __forceinline__ void load(const bf16* p) { v = *reinterpret_cast<const uint4*>(p); }
+    __device__ __forceinline__ void get(float (&x)[8]) const {
+        x[0] = bf16_lo(v.x); x[1] = bf16_hi(v.x); x[2] = bf16_lo(v.y); x[3] = bf16_hi(v.y);
+        x[4] = bf16_lo(v.z); x[5] = bf16_hi(v.z); x[6] = bf16_lo(v.w); x[7] = bf16_hi(v.w);
+    }
+};
+template <> struct Raw8<float> {
+    float v[8];
+    __device__ __forceinline__ void clear() {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] = 0.f;
+    }
+    __device__ __forceinline__ void load(const float* p) { load8(p, v); }
+    __device__ __forceinline__ void get(float (&x)[8]) const {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] = v[e];
+    }
+};
 
 template <typename T>
 __global__ void __launch_bounds__(QC_THREADS) qkv_conv_rows_kernel(QkvConvArgs a) {
@@ -196,51 +220,57 @@ __global__ void __launch_bounds__(QC_THREADS) qkv_conv_rows_kernel(QkvConvArgs a
     const bool both = c1 < h.hd;
     const int block_rows = strips * QR_STRIP, first = blockIdx.x * block_rows + strip * QR_STRIP, last = min(first + QR_STRIP, a.rows);
     if (strip < strips && first < a.rows) {
-        float w0[QR_TAPS][8], w1[QR_TAPS][8], u0[QR_TAPS][8], u1[QR_TAPS][8];  // window: u[QR_TAPS - 1] is the current row
-        auto fetch = [&](int row, float (&x)[8], float (&y)[8]) {
-            const T* src = nullptr;
-            if (row >= 0) src = proj + (int64_t)row * a.proj_stride;
-            else if (start + row >= 0) src = state + (int64_t)(keep + row) * h.C;
+        // every row of the strip and its history is asked for at once: one memory round trip per strip
+        Raw8<T> u0[QR_STRIP + QR_TAPS - 1], u1[QR_STRIP + QR_TAPS - 1];
 #pragma unroll
-            for (int e = 0; e < 8; ++e) x[e] = y[e] = 0.f;
+        for (int i = 0; i < QR_STRIP + QR_TAPS - 1; ++i) {
+            const int row = first + i - (QR_TAPS - 1);
+            const T* src = nullptr;
+            if (row >= 0 && row < last) src = proj + (int64_t)row * a.proj_stride;
+            else if (row < 0 && row >= -keep && start + row >= 0) src = state + (int64_t)(keep + row) * h.C;
+            u0[i].clear();
+            u1[i].clear();
             if (src) {
-                load8(src + c0, x);
-                if (both) load8(src + c1, y);
+                u0[i].load(src + c0);
+                if (both) u1[i].load(src + c1);
             }
-        };
+        }
+        float w0[QR_TAPS][8], w1[QR_TAPS][8];
 #pragma unroll
         for (int j = 0; j < QR_TAPS; ++j) {
             const int tap = j - (QR_TAPS - a.taps);  // fewer taps: the oldest ones are zero
 #pragma unroll
-            for (int e = 0; e < 8; ++e) w0[j][e] = w1[j][e] = u0[j][e] = u1[j][e] = 0.f;
+            for (int e = 0; e < 8; ++e) w0[j][e] = w1[j][e] = 0.f;
             if (tap >= 0) {
                 load8(a.conv_w + (int64_t)tap * h.C + h.chan0 + c0, w0[j]);
                 if (both) load8(a.conv_w + (int64_t)tap * h.C + h.chan0 + c1, w1[j]);
-                if (j < QR_TAPS - 1) fetch(first - (QR_TAPS - 1 - j), u0[j], u1[j]);
             }
         }
-        for (int row = first; row < last; ++row) {
-            fetch(row, u0[QR_TAPS - 1], u1[QR_TAPS - 1]);
+        const bool bad_start = start < 0 || start + a.rows > a.capacity;
+        if (bad_start) raise_status(a.status, GLMB_STATUS_BAD_INDEX);
+#pragma unroll
+        for (int i = 0; i < QR_STRIP; ++i) {
+            const int row = first + i;
+            if (row >= last) break;
             float y0[8], y1[8];
 #pragma unroll
-            for (int e = 0; e < 8; ++e) {
-                float s0 = 0.f, s1 = 0.f;
+            for (int e = 0; e < 8; ++e) y0[e] = y1[e] = 0.f;
 #pragma unroll
-                for (int j = 0; j < QR_TAPS; ++j) { s0 = fmaf(w0[j][e], u0[j][e], s0); s1 = fmaf(w1[j][e], u1[j][e], s1); }
-                y0[e] = s0;
-                y1[e] = s1;
+            for (int j = 0; j < QR_TAPS; ++j) {
+                float x[8];
+                u0[i + j].get(x);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) y0[e] = fmaf(w0[j][e], x[e], y0[e]);
+                u1[i + j].get(x);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) y1[e] = fmaf(w1[j][e], x[e], y1[e]);
             }
-            int pos = a.row_pos[row];
-            const bool bad = pos < 0 || pos >= a.capacity;
-            if (bad) {
-                raise_status(a.status, GLMB_STATUS_BAD_INDEX);
-                pos = min(max(pos, 0), a.capacity - 1);
-            }
+            const int pos = min(max(start + row, 0), a.capacity - 1);
             if (rotated) {
                 const float4* table = reinterpret_cast<const float4*>(a.rot + (int64_t)pos * half + c0);
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
-                    const float4 cs = table[e];
+                    const float4 cs = __ldg(table + e);
                     const float p = y0[2 * e], q = y1[2 * e], r = y0[2 * e + 1], s = y1[2 * e + 1];
                     y0[2 * e] = p * cs.x - q * cs.y;
                     y1[2 * e] = q * cs.x + p * cs.y;
@@ -248,18 +278,14 @@ __global__ void __launch_bounds__(QC_THREADS) qkv_conv_rows_kernel(QkvConvArgs a
                     y1[2 * e + 1] = s * cs.z + r * cs.w;
                 }
             }
-            qc_store<T>(a, h, row, pos, lane, !bad, c0, y0);
-            if (both) qc_store<T>(a, h, row, pos, lane, !bad, c1, y1);
+            qc_store<T>(a, h, row, pos, lane, !bad_start, c0, y0);
+            if (both) qc_store<T>(a, h, row, pos, lane, !bad_start, c1, y1);
             if (pair == 0 && h.hdp > h.hd) {  // the padding of the head row
                 float zero[8];
 #pragma unroll
                 for (int e = 0; e < 8; ++e) zero[e] = 0.f;
-                for (int c = h.hd; c < h.hdp; c += 8) qc_store<T>(a, h, row, pos, lane, !bad, c, zero);
+                for (int c = h.hd; c < h.hdp; c += 8) qc_store<T>(a, h, row, pos, lane, !bad_start, c, zero);
             }
-#pragma unroll
-            for (int j = 0; j + 1 < QR_TAPS; ++j)
-#pragma unroll
-                for (int e = 0; e < 8; ++e) { u0[j][e] = u0[j + 1][e]; u1[j][e] = u1[j + 1][e]; }
         }
     }
     if (blockIdx.x == 0) {
