@@ -568,10 +568,11 @@ static int launch_chunk_decode(const ChunkAttnArgs& a, cudaStream_t st) {
     if (make_map(&map_v, a.v, ring_rows, (uint64_t)a.G * a.vdimp, (uint64_t)a.G * a.vdimp, WARPS * 16)) return 3;
     int stages = 4;
     while (stages > 2 && chunk_decode_smem(a.dimp, a.vdimp, stages, WARPS) > 200 * 1024) --stages;
-    // CTAs per cluster: enough that the grid reaches every SM, at least one tile each
-    const int heads = a.G * ceil_div(a.H / a.G, CD_HEADS), tiles = ceil_div(a.ring, WARPS * 16);
+    // CTAs per cluster: enough that the grid reaches every SM, at least one tile each.  A cluster of 16 only while few are launched: the
+    // GPU places a handful of them at a time, and eight waited for one another (20 us before the first key, 10 us with eight per cluster).
+    const int heads = a.G * ceil_div(a.H / a.G, CD_HEADS), tiles = ceil_div(a.ring, WARPS * 16), most = heads * a.rows <= 4 ? 16 : 8;
     int splits = 1;
-    while (splits < 16 && splits * 2 <= tiles && splits * heads * a.rows < 148) splits *= 2;
+    while (splits < most && splits * 2 <= tiles && splits * heads * a.rows < 148) splits *= 2;
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(splits, heads, a.rows);
     cfg.blockDim = dim3(WARPS * 32);
