@@ -231,21 +231,29 @@ static inline size_t chunk_decode_smem(int dk, int dv, int stages, int warps) {
     return 1024 + (tiles > merge ? tiles : merge) + (size_t)CD_HEADS * (dk + 8) * 2;
 }
 
+__device__ __forceinline__ uint32_t movmatrix_trans(uint32_t x) {  // 8 x 8 matrix of 16-bit elements, transposed across the warp
+    uint32_t y;
+    asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(y) : "r"(x));
+    return y;
+}
+
 // grid (splits, key heads x blocks of 16 query heads, rows), cluster (splits, 1, 1).
-template <int DV, int WARPS>
+// A warp's 16 keys are the M of both products (scores: keys x heads; output: value columns x heads), the query heads the N (NT tiles of 8):
+// with the handful of query heads that share a key head, few multiplications are spent on padding.
+template <int DV, int WARPS, int NT>
 __global__ void __launch_bounds__(WARPS * 32)
 chunk_attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, ChunkAttnArgs a, int stages) {
-    constexpr int KEYS = WARPS * 16, BOX = KEYS * 128;
+    constexpr int KEYS = WARPS * 16, BOX = KEYS * 128, HEADS = NT * 8;
     cg::cluster_group cluster = cg::this_cluster();
     extern __shared__ unsigned char smem_raw[];
-    __shared__ float ml_s[WARPS][CD_HEADS][2];  // (maximum, sum) per warp
-    __shared__ __align__(8) float cta_ml[CD_HEADS][2];
+    __shared__ float ml_s[WARPS][HEADS][2];  // (maximum, sum) per warp
+    __shared__ __align__(8) float cta_ml[HEADS][2];
     __shared__ __align__(8) uint64_t full_bar[4];
     const int dk = a.dimp, dv = a.vdimp, KP = dk + 8;
     const int kboxes = (dk + 63) / 64, vboxes = (dv + 63) / 64;
     unsigned char* tiles_s = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
     const size_t stage_bytes = (size_t)(kboxes + vboxes) * BOX;
-    const size_t tile_area = stages * stage_bytes, merge_area = (size_t)WARPS * CD_HEADS * dv * 4;
+    const size_t tile_area = stages * stage_bytes, merge_area = (size_t)WARPS * HEADS * dv * 4;
     bf16* q_s = reinterpret_cast<bf16*>(tiles_s + (tile_area > merge_area ? tile_area : merge_area));
     if (threadIdx.x == 0) {
         for (int s = 0; s < stages; ++s) mbar_init(full_bar + s, 1);
@@ -276,7 +284,7 @@ chunk_attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
     {
         const bf16* q = reinterpret_cast<const bf16*>(a.q) + ((int64_t)row * a.H + h0) * dk;
         const int pieces = dk / 8;
-        for (int i = threadIdx.x; i < CD_HEADS * pieces; i += WARPS * 32) {
+        for (int i = threadIdx.x; i < HEADS * pieces; i += WARPS * 32) {
             const int r = i / pieces, c = i % pieces;
             *reinterpret_cast<uint4*>(q_s + r * KP + c * 8) = r < heads ? *reinterpret_cast<const uint4*>(q + (int64_t)r * dk + c * 8) : make_uint4(0, 0, 0, 0);
         }
@@ -284,18 +292,34 @@ chunk_attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
     __syncthreads();
 
     const float scale2 = a.scale * CA_LOG2E;
-    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-    float o[DV / 8][4];
+    float m[NT][2], l[NT][2];  // of heads 8 n + 2 t4 + e, equal on the lanes that share t4 (m) or this lane's keys (l)
+    float o[DV / 16][NT][4];   // value columns 16 j + g, + 8; heads 8 n + 2 t4, + 1
 #pragma unroll
-    for (int j = 0; j < DV / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
-    const bf16* qa = q_s + (mr + 8 * (mi & 1)) * KP + 8 * (mi >> 1);
+    for (int n = 0; n < NT; ++n) {
+        m[n][0] = m[n][1] = -INFINITY;
+        l[n][0] = l[n][1] = 0.f;
+#pragma unroll
+        for (int j = 0; j < DV / 16; ++j) o[j][n][0] = o[j][n][1] = o[j][n][2] = o[j][n][3] = 0.f;
+    }
     // this lane's rows of a key / value fragment and its 16-byte pieces of a 128-byte row, as they lie swizzled
-    const int k_row = (mr + 8 * (mi >> 1)) * 128, v_row = (mr + 8 * (mi & 1)) * 128;
+    const int k_row = (mr + 8 * (mi & 1)) * 128, v_row = (mr + 8 * (mi >> 1)) * 128;
     int k_col[4], v_col[4];
 #pragma unroll
     for (int c = 0; c < 4; ++c) {
-        k_col[c] = ((2 * c + (mi & 1)) ^ mr) << 4;
-        v_col[c] = ((2 * c + (mi >> 1)) ^ mr) << 4;
+        k_col[c] = ((2 * c + (mi >> 1)) ^ mr) << 4;
+        v_col[c] = ((2 * c + (mi & 1)) ^ mr) << 4;
+    }
+    const bf16* q_lane = q_s + (mr + (NT == 2 ? 8 * (mi >> 1) : 0)) * KP + 8 * (mi & 1);
+    constexpr int QSTEPS = DV <= 128 ? 8 : 1;  // query fragments of head sizes up to 128 stay in registers
+    uint32_t qf[QSTEPS][2 * NT];
+    auto load_q = [&](uint32_t (&f)[2 * NT], int k0) {
+        if constexpr (NT == 2) ldmatrix_x4(f, q_lane + k0);
+        else ldmatrix_x2(f, q_lane + k0);
+    };
+    if constexpr (QSTEPS > 1) {
+#pragma unroll
+        for (int c = 0; c < QSTEPS; ++c)
+            if (c * 16 < dk) load_q(qf[c], c * 16);
     }
     bool ok = true;
     for (int i = 0; i < mine; ++i) {
@@ -313,62 +337,71 @@ chunk_attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
             __syncwarp();
         }
         if (left > 0) {
-            float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-            const bf16* qk = qa;
+            float s[NT][4];  // keys g, g + 8; heads 8 n + 2 t4, + 1
+#pragma unroll
+            for (int n = 0; n < NT; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
             const unsigned char* kb = kt + w0 * 128 + k_row;
-            for (int k0 = 0; k0 < dk; k0 += 64, kb += BOX, qk += 64)
+            auto step = [&](const uint32_t (&f)[2 * NT], const unsigned char* at) {
+                uint32_t kf[4];
+                ldmatrix_x4(kf, at);
 #pragma unroll
-                for (int c = 0; c < 4; ++c)
-                    if (k0 + c * 16 < dk) {
-                        uint32_t qf[4], kf[4];
-                        ldmatrix_x4(qf, qk + c * 16);
-                        ldmatrix_x4(kf, kb + k_col[c]);
-                        mma_bf16_16816(s[0], qf, kf[0], kf[1]);
-                        mma_bf16_16816(s[1], qf, kf[2], kf[3]);
-                    }
-            float mx[2] = {m[0], m[1]};
+                for (int n = 0; n < NT; ++n) mma_bf16_16816(s[n], kf, f[2 * n], f[2 * n + 1]);
+            };
+            if constexpr (QSTEPS > 1) {
 #pragma unroll
-            for (int j = 0; j < 2; ++j)
+                for (int c = 0; c < QSTEPS; ++c)
+                    if (c * 16 < dk) step(qf[c], kb + (c >> 2) * BOX + k_col[c & 3]);
+            } else {
+                for (int k0 = 0; k0 < dk; k0 += 64, kb += BOX)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const float x = j * 8 + 2 * t4 + (e & 1) >= left ? -INFINITY : s[j][e] * scale2;
-                    s[j][e] = x;
-                    mx[e >> 1] = fmaxf(mx[e >> 1], x);
-                }
-            float fix[2];
-#pragma unroll
-            for (int i2 = 0; i2 < 2; ++i2) {
-                mx[i2] = fmaxf(mx[i2], __shfl_xor_sync(0xffffffffu, mx[i2], 1));
-                mx[i2] = fmaxf(mx[i2], __shfl_xor_sync(0xffffffffu, mx[i2], 2));
-                fix[i2] = exp2f(m[i2] - mx[i2]);  // at least one key exists: the maximum is finite
-                m[i2] = mx[i2];
+                    for (int c = 0; c < 4; ++c)
+                        if (k0 + c * 16 < dk) {
+                            load_q(qf[0], k0 + c * 16);
+                            step(qf[0], kb + k_col[c]);
+                        }
             }
-            float sum[2] = {0.f, 0.f};
+            uint32_t hi[NT][2], lw[NT][2];  // weights as the second operand: keys x heads
+            float fix[NT][2];
 #pragma unroll
-            for (int j = 0; j < 2; ++j)
+            for (int n = 0; n < NT; ++n) {
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    s[j][e] = exp2f(s[j][e] - m[e >> 1]);
-                    sum[e >> 1] += s[j][e];
+                for (int e = 0; e < 4; ++e) s[n][e] = g + 8 * (e >> 1) >= left ? -INFINITY : s[n][e] * scale2;
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    float top = fmaxf(s[n][e], s[n][2 + e]);
+                    top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 4));
+                    top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 8));
+                    top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 16));
+                    top = fmaxf(top, m[n][e]);  // at least one key exists: finite
+                    fix[n][e] = exp2f(m[n][e] - top);
+                    m[n][e] = top;
+                    s[n][e] = exp2f(s[n][e] - top);
+                    s[n][2 + e] = exp2f(s[n][2 + e] - top);
+                    l[n][e] = l[n][e] * fix[n][e] + s[n][e] + s[n][2 + e];
                 }
-            l[0] = l[0] * fix[0] + sum[0];
-            l[1] = l[1] * fix[1] + sum[1];
-            uint32_t hi[4], lw[4];
-            ca_split(s[0][0], s[0][1], hi[0], lw[0]);
-            ca_split(s[0][2], s[0][3], hi[1], lw[1]);
-            ca_split(s[1][0], s[1][1], hi[2], lw[2]);
-            ca_split(s[1][2], s[1][3], hi[3], lw[3]);
 #pragma unroll
-            for (int j = 0; j < DV / 8; j += 2)
-                if (j * 8 < dv) {
-                    o[j][0] *= fix[0]; o[j][1] *= fix[0]; o[j][2] *= fix[1]; o[j][3] *= fix[1];
-                    o[j + 1][0] *= fix[0]; o[j + 1][1] *= fix[0]; o[j + 1][2] *= fix[1]; o[j + 1][3] *= fix[1];
+                for (int e = 0; e < 2; ++e) {
+                    uint32_t x, y;
+                    ca_split(s[n][2 * e], s[n][2 * e + 1], x, y);
+                    hi[n][e] = movmatrix_trans(x);
+                    lw[n][e] = movmatrix_trans(y);
+                }
+            }
+            bool moved = false;
+#pragma unroll
+            for (int n = 0; n < NT; ++n) moved |= fix[n][0] != 1.f || fix[n][1] != 1.f;
+            moved = __any_sync(0xffffffffu, moved);
+#pragma unroll
+            for (int j = 0; j < DV / 16; ++j)
+                if (j * 16 < dv) {
                     uint32_t vf[4];
-                    ldmatrix_x4_trans(vf, vt + (j >> 3) * BOX + w0 * 128 + v_row + v_col[(j & 7) >> 1]);
-                    mma_bf16_16816(o[j], hi, vf[0], vf[1]);
-                    mma_bf16_16816(o[j + 1], hi, vf[2], vf[3]);
-                    mma_bf16_16816(o[j], lw, vf[0], vf[1]);
-                    mma_bf16_16816(o[j + 1], lw, vf[2], vf[3]);
+                    ldmatrix_x4_trans(vf, vt + (j >> 2) * BOX + w0 * 128 + v_row + v_col[j & 3]);
+#pragma unroll
+                    for (int n = 0; n < NT; ++n) {
+                        if (moved) { o[j][n][0] *= fix[n][0]; o[j][n][1] *= fix[n][1]; o[j][n][2] *= fix[n][0]; o[j][n][3] *= fix[n][1]; }
+                        mma_bf16_16816(o[j][n], vf, hi[n][0], hi[n][1]);
+                        mma_bf16_16816(o[j][n], vf, lw[n][0], lw[n][1]);
+                    }
                 }
         }
         if (i + stages < mine) {  // every warp has read the stage: fill it again
@@ -377,23 +410,27 @@ chunk_attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
         }
     }
 #pragma unroll
-    for (int i = 0; i < 2; ++i) {
-        l[i] += __shfl_xor_sync(0xffffffffu, l[i], 1);
-        l[i] += __shfl_xor_sync(0xffffffffu, l[i], 2);
-        if (t4 == 0) { ml_s[warp][g + 8 * i][0] = m[i]; ml_s[warp][g + 8 * i][1] = l[i]; }
-    }
+    for (int n = 0; n < NT; ++n)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            float sum = l[n][e];
+            sum += __shfl_xor_sync(0xffffffffu, sum, 4);
+            sum += __shfl_xor_sync(0xffffffffu, sum, 8);
+            sum += __shfl_xor_sync(0xffffffffu, sum, 16);
+            if (g == 0) { ml_s[warp][n * 8 + 2 * t4 + e][0] = m[n][e]; ml_s[warp][n * 8 + 2 * t4 + e][1] = sum; }
+        }
     __syncthreads();  // every warp has left the tiles: the merge area takes their place
     float* o_s = reinterpret_cast<float*>(tiles_s);  // [warp][head][dv]
 #pragma unroll
-    for (int j = 0; j < DV / 8; ++j)
-        if (j * 8 < dv) {
-            float* d = o_s + ((size_t)warp * CD_HEADS + g) * dv + j * 8 + 2 * t4;
-            *reinterpret_cast<float2*>(d) = make_float2(o[j][0], o[j][1]);
-            *reinterpret_cast<float2*>(d + 8 * dv) = make_float2(o[j][2], o[j][3]);
-        }
+    for (int j = 0; j < DV / 16; ++j)
+        if (j * 16 < dv)
+#pragma unroll
+            for (int n = 0; n < NT; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) o_s[((size_t)warp * HEADS + n * 8 + 2 * t4 + (e & 1)) * dv + j * 16 + g + 8 * (e >> 1)] = o[j][n][e];
     __syncthreads();
     // ---- warps of the CTA into warp 0's area ------------------------------------------------------------
-    if (threadIdx.x < CD_HEADS) {
+    if (threadIdx.x < HEADS) {
         float top = -INFINITY, sum = 0.f;
         for (int w = 0; w < WARPS; ++w) top = fmaxf(top, ml_s[w][threadIdx.x][0]);
         for (int w = 0; w < WARPS; ++w)
@@ -402,22 +439,22 @@ chunk_attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
         cta_ml[threadIdx.x][1] = sum;
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < CD_HEADS * dv; i += WARPS * 32) {
+    for (int i = threadIdx.x; i < HEADS * dv; i += WARPS * 32) {
         const int h = i / dv;
         const float top = cta_ml[h][0];
         float v = 0.f;
         for (int w = 0; w < WARPS; ++w)
-            if (ml_s[w][h][0] != -INFINITY) v += o_s[(size_t)w * CD_HEADS * dv + i] * exp2f(ml_s[w][h][0] - top);
+            if (ml_s[w][h][0] != -INFINITY) v += o_s[(size_t)w * HEADS * dv + i] * exp2f(ml_s[w][h][0] - top);
         o_s[i] = v;
     }
     cluster.sync();
     // ---- CTAs of the cluster: each finishes its share of the outputs, the sink joins here -----------------
     // First every CTA's (maximum, sum) of every head, all loads at once, then a weight per CTA and head.
-    __shared__ float part_s[16][CD_HEADS][2];
-    for (int i = threadIdx.x; i < splits * CD_HEADS; i += WARPS * 32) {
-        const float2 ml = *reinterpret_cast<const float2*>(cluster.map_shared_rank(&cta_ml[0][0], i / CD_HEADS) + (i % CD_HEADS) * 2);
-        part_s[i / CD_HEADS][i % CD_HEADS][0] = ml.x;
-        part_s[i / CD_HEADS][i % CD_HEADS][1] = ml.y;
+    __shared__ float part_s[16][HEADS][2];
+    for (int i = threadIdx.x; i < splits * HEADS; i += WARPS * 32) {
+        const float2 ml = *reinterpret_cast<const float2*>(cluster.map_shared_rank(&cta_ml[0][0], i / HEADS) + (i % HEADS) * 2);
+        part_s[i / HEADS][i % HEADS][0] = ml.x;
+        part_s[i / HEADS][i % HEADS][1] = ml.y;
     }
     __syncthreads();
     if ((int)threadIdx.x < heads) {
@@ -550,15 +587,15 @@ static int launch_chunk_prefill(const ChunkAttnArgs& a, cudaStream_t st) {
     return (int)cudaGetLastError();
 }
 
-template <int DV, int WARPS>
+template <int DV, int WARPS, int NT>
 static int launch_chunk_decode(const ChunkAttnArgs& a, cudaStream_t st) {
     static DeviceOnce once;
-    cudaError_t e = chunk_smem_limit(chunk_attn_decode_kernel<DV, WARPS>, once);
+    cudaError_t e = chunk_smem_limit(chunk_attn_decode_kernel<DV, WARPS, NT>, once);
     if (e != cudaSuccess) return (int)e;
     static DeviceOnce wide;  // clusters of 16 are beyond the portable size
     const int wide_dev = wide.pending();
     if (wide_dev != DeviceOnce::SET) {
-        e = cudaFuncSetAttribute(chunk_attn_decode_kernel<DV, WARPS>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+        e = cudaFuncSetAttribute(chunk_attn_decode_kernel<DV, WARPS, NT>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
         if (e != cudaSuccess) return (int)e;
         wide.mark(wide_dev);
     }
@@ -586,7 +623,7 @@ static int launch_chunk_decode(const ChunkAttnArgs& a, cudaStream_t st) {
     attr[1].val.clusterDim.y = attr[1].val.clusterDim.z = 1;
     cfg.attrs = attr;
     cfg.numAttrs = 2;
-    const cudaError_t le = cudaLaunchKernelEx(&cfg, chunk_attn_decode_kernel<DV, WARPS>, map_k, map_v, a, stages);
+    const cudaError_t le = cudaLaunchKernelEx(&cfg, chunk_attn_decode_kernel<DV, WARPS, NT>, map_k, map_v, a, stages);
     return le != cudaSuccess ? (int)le : (int)cudaGetLastError();
 }
 
@@ -610,10 +647,11 @@ GLMB_API int glmb_chunk_attn_prefill(const ChunkAttnArgs* args, void* stream) {
 GLMB_API int glmb_chunk_attn_decode(const ChunkAttnArgs* args, void* stream) {
     const ChunkAttnArgs a = *args;
     if (!chunk_args_ok(a) || !a.decode || a.dimp > 256 || a.vdimp > 256) return 1;
-    if (a.dimp > 128) return launch_chunk_decode<256, 4>(a, (cudaStream_t)stream);
-    if (a.vdimp <= 64) return launch_chunk_decode<64, 8>(a, (cudaStream_t)stream);
-    if (a.vdimp <= 128) return launch_chunk_decode<128, 8>(a, (cudaStream_t)stream);
-    return launch_chunk_decode<256, 4>(a, (cudaStream_t)stream);
+    const bool few = a.H / a.G <= 8;
+    cudaStream_t st = (cudaStream_t)stream;
+    if (a.dimp > 128 || a.vdimp > 128) return few ? launch_chunk_decode<256, 4, 1>(a, st) : launch_chunk_decode<256, 4, 2>(a, st);
+    if (a.vdimp <= 64) return few ? launch_chunk_decode<64, 8, 1>(a, st) : launch_chunk_decode<64, 8, 2>(a, st);
+    return few ? launch_chunk_decode<128, 8, 1>(a, st) : launch_chunk_decode<128, 8, 2>(a, st);
 }
 
 // Any head size (values up to 1024 columns), bf16 or fp32.
