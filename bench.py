@@ -23,8 +23,8 @@ Two measurements:
   votes over gloo and the token line written and flushed by rank 0.  The rate is the engine's own report (decode tokens /
   decode wall seconds, slowest rank), which is how the published 13.57 tokens/s is defined.
 
-``--design namizen`` measures another workload instead: prefill and decode throughput of the Namizen family beside this one at equal size
-(``glm_tpu_b200/benchmarks/design_bench.py``), one GPU, one JSON line.
+``--design namizen`` and ``--design zikevik`` measure another workload instead: prefill and decode throughput of that family beside this one at
+equal size (``glm_tpu_b200/benchmarks/design_bench.py``), one GPU, one JSON line.
 
 ``--impl reference`` reports why the JAX/Pallas TPU reference cannot run on this machine.
 """
@@ -122,10 +122,10 @@ def design_arm(args) -> int:
     if args.gpus != 1:
         raise SystemExit("--design runs on one GPU")
     build()
-    out = design_bench.run(args.sizes.split(","), steps=args.steps, warmup=args.warmup, sampler=ClockSampler(0))
+    out = design_bench.run(args.sizes.split(","), steps=args.steps, warmup=args.warmup, design=args.design, sampler=ClockSampler(0))
     last = out["sizes"][args.sizes.split(",")[-1]]
     print(json.dumps({
-        "metric": "Namizen prefill and decode tokens/s beside GLM-MoE-DSA (dense layers) at equal size", "value": last["namizen"]["prefill"]["tok_s"],
+        "metric": f"{args.design.capitalize()} prefill and decode tokens/s beside GLM-MoE-DSA at equal size", "value": last[args.design]["prefill"]["tok_s"],
         "unit": "prefill tokens/s (last size)", "higher_is_better": True, "n_gpus": 1, "steps": args.steps, "warmup": args.warmup, "dtype": "bf16",
         "data": "synthetic: random weights, random prompt ids, random cache rows at the decode depth", **out}))
     return 0
@@ -307,8 +307,8 @@ def main() -> int:
     ap.add_argument("--kv-layout", default="auto", choices=["auto", "striped", "replicated"],
                     help="latent cache: a replica per GPU (no attention exchange) or striped by position over the GPUs")
     ap.add_argument("--decode-path", default="auto", choices=["auto", "kernels", "phases", "mega"])
-    ap.add_argument("--design", choices=["namizen"], help="measure this family beside GLM-MoE-DSA at equal size instead of the headline workload")
-    ap.add_argument("--sizes", default="small,medium,large", help="with --design: which of the sizes small, medium, large")
+    ap.add_argument("--design", choices=["namizen", "zikevik"], help="measure this family beside GLM-MoE-DSA at equal size instead of the headline workload")
+    ap.add_argument("--sizes", default="small,medium,large", help="with --design: which of the sizes small, medium, large (Zikevik also: routed)")
     args = ap.parse_args()
     if args.design:
         return design_arm(args)

@@ -202,3 +202,62 @@ class RingCacheConfig:
                     count *= n
                 total += count * self.element_bytes
         return total
+
+
+@dataclass(frozen=True)
+class HybridCacheConfig:
+    """Caches of a model whose layers are recurrent or attend over a shared latent, one GPU.
+
+    A latent layer keeps one row per position and lane, ``[normalized latent | rotated key part]``, both parts padded to a multiple of 16
+    elements (whole tensor-core steps, 16-byte vectors).  A recurrent layer keeps, per lane and whatever the context, an fp32 state per head
+    (stored ``[vdim, dim]``: a value channel's row of key channels, padded to a multiple of 32) and the last ``taps - 1`` projected rows of its
+    convolution.
+
+    ``geometry.layers[i].mixer`` gives the layer's sizes; a recurrent mixer has ``conv_width``, a latent one ``kv_rank``.
+    """
+
+    geometry: object
+    context_capacity: int
+    lanes: int = 1
+    element_bytes: int = 2
+    page: int = 1
+
+    def __post_init__(self) -> None:
+        if self.context_capacity < 1 or not 1 <= self.lanes <= 8:
+            raise PlanValidationError("the context capacity must be positive and the lanes between 1 and 8")
+
+    def _mixer(self, layer: int):
+        return self.geometry.layers[layer].mixer
+
+    def is_latent(self, layer: int) -> bool:
+        return hasattr(self._mixer(layer), "kv_rank")
+
+    def latent_columns(self, layer: int) -> tuple[int, int]:
+        """Padded columns of the latent and of the rotated key part."""
+        m = self._mixer(layer)
+        return (-(-m.kv_rank // 16) * 16, -(-m.rot_dim // 16) * 16)
+
+    def latent_shape(self, layer: int) -> tuple[int, int, int]:
+        return (self.lanes, self.context_capacity, sum(self.latent_columns(layer)))
+
+    def state_shape(self, layer: int) -> tuple[int, int, int, int]:
+        m = self._mixer(layer)
+        return (self.lanes, m.heads, m.vdim, -(-m.dim // 32) * 32)
+
+    def conv_shape(self, layer: int) -> tuple[int, int, int]:
+        m = self._mixer(layer)
+        return (self.lanes, m.conv - 1, m.conv_width)
+
+    def layer_bytes(self, layer: int) -> int:
+        def count(shape):
+            n = 1
+            for x in shape:
+                n *= x
+            return n
+
+        if self.is_latent(layer):
+            return count(self.latent_shape(layer)) * self.element_bytes
+        return count(self.state_shape(layer)) * 4 + count(self.conv_shape(layer)) * self.element_bytes
+
+    def cache_bytes_per_gpu(self) -> int:
+        return sum(self.layer_bytes(i) for i in range(len(self.geometry.layers)))

@@ -14,7 +14,8 @@
 //                              TMA and are dealt to the cluster's CTAs, the partial softmax states meet in distributed shared memory
 //   chunk_attn_any_kernel      any head size and element type, one CTA per (row, head): the 32-bit path and larger heads
 //
-// The running maximum starts at the sink and the sum gets the sink's term once; the sink has no value.
+// The running maximum starts at the sink and the sum gets the sink's term once; the sink has no value.  A gate per row and head may scale
+// the output.
 #include <cooperative_groups.h>
 
 #include "attention_core.cuh"
@@ -51,6 +52,11 @@ __device__ __forceinline__ void ca_store2(bf16* p, float x, float y, bool both, 
         p[0] = __float2bfloat16_rn(x);
         if (both) p[1] = __float2bfloat16_rn(y);
     }
+}
+
+template <typename T>
+__device__ __forceinline__ float ca_gate(const ChunkAttnArgs& a, int row, int head) {
+    return a.gate ? sigmoidf_precise(to_f32(reinterpret_cast<const T*>(a.gate)[(int64_t)row * a.gate_stride + head])) : 1.f;
 }
 
 // ---------------------------------------------------------------------------------------------------
@@ -96,12 +102,12 @@ __global__ void __launch_bounds__(CP_THREADS) chunk_attn_prefill_kernel(ChunkAtt
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     {
-        const bf16* q = reinterpret_cast<const bf16*>(a.q) + ((int64_t)r0 * a.H + head) * a.dimp;
+        const bf16* q = reinterpret_cast<const bf16*>(a.q) + (int64_t)r0 * a.q_stride + (int64_t)head * a.dimp;
         const int pieces = dk / 8;
         for (int i = tid; i < CP_ROWS * pieces; i += CP_THREADS) {
             const int r = i / pieces, c = i % pieces;
             bf16* d = q_s + r * KP + c * 8;
-            if (r < nrows) cp_async16(d, q + (int64_t)r * a.H * a.dimp + c * 8);
+            if (r < nrows) cp_async16(d, q + (int64_t)r * a.q_stride + c * 8);
             else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
         }
     }
@@ -212,7 +218,7 @@ __global__ void __launch_bounds__(CP_THREADS) chunk_attn_prefill_kernel(ChunkAtt
         if (r >= nrows) continue;
         bf16* dst = reinterpret_cast<bf16*>(a.out) + (int64_t)(r0 + r) * a.out_stride + (int64_t)head * a.vdim;
         const bool aligned = !(reinterpret_cast<uintptr_t>(dst) & 3);
-        const float inv = 1.f / l[i];
+        const float inv = ca_gate<bf16>(a, r0 + r, head) / l[i];
 #pragma unroll
         for (int j = 0; j < DV / 8; ++j) {
             const int c = j * 8 + 2 * t4;
@@ -282,7 +288,7 @@ chunk_attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
     if (threadIdx.x == 0)
         for (int i = 0; i < min(stages, mine); ++i) load_tile(i);
     {
-        const bf16* q = reinterpret_cast<const bf16*>(a.q) + ((int64_t)row * a.H + h0) * dk;
+        const bf16* q = reinterpret_cast<const bf16*>(a.q) + (int64_t)row * a.q_stride + (int64_t)h0 * dk;
         const int pieces = dk / 8;
         for (int i = threadIdx.x; i < HEADS * pieces; i += WARPS * 32) {
             const int r = i / pieces, c = i % pieces;
@@ -468,7 +474,7 @@ chunk_attn_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
             sum += part_s[p][h][1] * w;
             part_s[p][h][0] = w;
         }
-        const float inv = sum > 0.f ? 1.f / sum : 0.f;
+        const float inv = sum > 0.f ? ca_gate<bf16>(a, row, h0 + h) / sum : 0.f;
         for (int p = 0; p < splits; ++p) part_s[p][h][0] *= inv;
     }
     __syncthreads();
@@ -500,7 +506,7 @@ __global__ void __launch_bounds__(CX_THREADS) chunk_attn_any_kernel(ChunkAttnArg
     const int pos = a.decode ? ca_pos(a, row) : a.start + row;
     const int key0 = pos / a.chunk * a.chunk, keys = active ? pos - key0 + 1 : 0;
     const int64_t row0 = a.decode ? (int64_t)ca_lane(a, row) * a.ring : key0 - a.base;  // where the first visible key lies
-    const T* q = reinterpret_cast<const T*>(a.q) + ((int64_t)row * a.H + head) * a.dimp;
+    const T* q = reinterpret_cast<const T*>(a.q) + (int64_t)row * a.q_stride + (int64_t)head * a.dimp;
     for (int d = threadIdx.x; d < a.dim; d += CX_THREADS) q_f[d] = to_f32(q[d]);
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -551,17 +557,23 @@ __global__ void __launch_bounds__(CX_THREADS) chunk_attn_any_kernel(ChunkAttnArg
         __syncthreads();
     }
     T* out = reinterpret_cast<T*>(a.out) + (int64_t)row * a.out_stride + (int64_t)head * a.vdim;
+    const float gate = ca_gate<T>(a, row, head);
 #pragma unroll
     for (int i = 0; i < CX_COLS; ++i) {
         const int c = threadIdx.x + i * CX_THREADS;
-        if (c < a.vdim) from_f32(l > 0.f ? acc[i] / l : 0.f, out[c]);
+        if (c < a.vdim) from_f32(l > 0.f ? acc[i] / l * gate : 0.f, out[c]);
     }
 }
 
 // ===================================================================================================
+static ChunkAttnArgs chunk_args(const ChunkAttnArgs* args) {
+    ChunkAttnArgs a = *args;
+    if (!a.q_stride) a.q_stride = (int64_t)a.H * a.dimp;
+    return a;
+}
 static bool chunk_args_ok(const ChunkAttnArgs& a) {
     if (a.rows < 1 || a.H < 1 || a.G < 1 || a.H % a.G || a.dim < 1 || a.vdim < 1 || (a.dimp & 15) || (a.vdimp & 15) || a.dimp < a.dim || a.vdimp < a.vdim ||
-        a.chunk < 1 || !a.q || !a.k || !a.v || !a.out)
+        a.chunk < 1 || !a.q || !a.k || !a.v || !a.out || (a.q_stride & 7))
         return false;
     if (a.decode) return a.ring >= 1 && a.capacity >= 1 && a.lanes >= 1 && (a.ring == a.chunk || a.ring == a.capacity) && a.row_pos && a.row_lane;
     // every key a row can see lies in the buffers
@@ -635,7 +647,7 @@ GLMB_API void glmb_set_chunk_prefill_tc(int enabled) { g_chunk_prefill_tc = enab
 
 // bf16, rows of one sequence at consecutive positions; head sizes up to 256.
 GLMB_API int glmb_chunk_attn_prefill(const ChunkAttnArgs* args, void* stream) {
-    const ChunkAttnArgs a = *args;
+    ChunkAttnArgs a = chunk_args(args);
     if (!chunk_args_ok(a) || a.decode || a.dimp > 256 || a.vdimp > 256) return 1;
     if (g_chunk_prefill_tc && a.dimp <= 128 && a.vdimp <= 128 && a.scale > 0.f) return launch_chunk_attn_tcgen05(a, (cudaStream_t)stream);
     if (a.vdimp <= 64) return launch_chunk_prefill<64>(a, (cudaStream_t)stream);
@@ -645,7 +657,7 @@ GLMB_API int glmb_chunk_attn_prefill(const ChunkAttnArgs* args, void* stream) {
 
 // bf16, one row per sequence, every key in the ring; head sizes up to 256.
 GLMB_API int glmb_chunk_attn_decode(const ChunkAttnArgs* args, void* stream) {
-    const ChunkAttnArgs a = *args;
+    ChunkAttnArgs a = chunk_args(args);
     if (!chunk_args_ok(a) || !a.decode || a.dimp > 256 || a.vdimp > 256) return 1;
     const bool few = a.H / a.G <= 8;
     cudaStream_t st = (cudaStream_t)stream;
@@ -656,7 +668,7 @@ GLMB_API int glmb_chunk_attn_decode(const ChunkAttnArgs* args, void* stream) {
 
 // Any head size (values up to 1024 columns), bf16 or fp32.
 GLMB_API int glmb_chunk_attn_any(const ChunkAttnArgs* args, int is_f32, void* stream) {
-    const ChunkAttnArgs a = *args;
+    ChunkAttnArgs a = chunk_args(args);
     if (!chunk_args_ok(a) || a.vdim > CX_THREADS * CX_COLS || a.dim > 8192) return 1;
     const dim3 grid(a.rows, a.H);
     const size_t smem = (size_t)a.dim * sizeof(float);

@@ -242,7 +242,9 @@ chunk_attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
             } else {
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
                 if (a.sink) l += fa_exp2(sink2 - m);
-                const float inv = 1.f / l;
+                float inv = 1.f / l;
+                if (a.gate && row < range[t].rows)
+                    inv *= sigmoidf_precise(__bfloat162float(reinterpret_cast<const bf16*>(a.gate)[(int64_t)(r0 + t * FA_TILE + row) * a.gate_stride + head]));
                 bf16* dst = reinterpret_cast<bf16*>(a.out) + (int64_t)(r0 + t * FA_TILE + row) * a.out_stride + (int64_t)head * a.vdim;
                 const bool vec = !(reinterpret_cast<uintptr_t>(dst) & 15);
                 for (int c = 0; c < a.vdimp; c += 16) {
@@ -274,7 +276,7 @@ chunk_attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
 
 int launch_chunk_attn_tcgen05(const ChunkAttnArgs& a, cudaStream_t stream) {
     CUtensorMap map_q, map_k, map_v;
-    if (make_map(&map_q, a.q, (uint64_t)a.rows, (uint64_t)a.H * a.dimp, (uint64_t)a.H * a.dimp, FA_TILE)) return 3;
+    if (make_map(&map_q, a.q, (uint64_t)a.rows, (uint64_t)a.H * a.dimp, (uint64_t)a.q_stride, FA_TILE)) return 3;
     if (make_map(&map_k, a.k, (uint64_t)a.keys, (uint64_t)a.G * a.dimp, (uint64_t)a.G * a.dimp, FA_TILE)) return 3;
     if (make_map(&map_v, a.v, (uint64_t)a.keys, (uint64_t)a.G * a.vdimp, (uint64_t)a.G * a.vdimp, FA_TILE)) return 3;
     static DeviceOnce once;

@@ -15,13 +15,13 @@
 // ---------------------------------------------------------------------------------------------------
 // One warp per row.  E <= 1024.
 __global__ void __launch_bounds__(128)
-router_topk_kernel(const float* __restrict__ logits, const float* __restrict__ bias, int rows, int E, int top_k,
+router_topk_kernel(const float* __restrict__ logits, int64_t stride, const float* __restrict__ bias, int rows, int E, int top_k, int normalize,
                    int* __restrict__ ids, float* __restrict__ weights) {
     GLMB_PDL_PROLOGUE();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int r = blockIdx.x * (blockDim.x >> 5) + warp;
     if (r >= rows) return;
-    const float* lg = logits + (int64_t)r * E;
+    const float* lg = logits + (int64_t)r * stride;
     const int per = (E + 31) / 32;  // <= 32
     uint32_t taken = 0;             // bit i: this lane's i-th expert (e = lane + 32*i) is already chosen
     float picked_sum = 0.f;
@@ -34,7 +34,7 @@ router_topk_kernel(const float* __restrict__ logits, const float* __restrict__ b
             const int e = lane + 32 * i;
             if (e < E && !((taken >> i) & 1u)) {
                 const float sc = sigmoidf_precise(lg[e]);
-                const uint32_t key = orderable_u32(__fadd_rn(sc, bias[e]));
+                const uint32_t key = orderable_u32(__fadd_rn(sc, bias ? bias[e] : 0.f));
                 if (best_e == 0x7fffffff || key > best_key) { best_key = key; best_e = e; best_score = sc; }
             }
         }
@@ -51,18 +51,18 @@ router_topk_kernel(const float* __restrict__ logits, const float* __restrict__ b
         picked_sum += best_score;
         if (lane == 0) ids[(int64_t)r * top_k + s] = best_e == 0x7fffffff ? 0 : best_e;
     }
-    if (lane < top_k) weights[(int64_t)r * top_k + lane] = my_score / (picked_sum + 1e-20f);
+    if (lane < top_k) weights[(int64_t)r * top_k + lane] = normalize ? my_score / (picked_sum + 1e-20f) : my_score;
 }
 
 // Same selection for E <= 256: every lane loads its (up to 8) logits once and keeps score and key in registers (router_core.cuh).
 __global__ void __launch_bounds__(128)
-router_topk256_kernel(const float* __restrict__ logits, const float* __restrict__ bias, int rows, int E, int top_k,
+router_topk256_kernel(const float* __restrict__ logits, int64_t stride, const float* __restrict__ bias, int rows, int E, int top_k, int normalize,
                       int* __restrict__ ids, float* __restrict__ weights) {
     GLMB_PDL_PROLOGUE();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int r = blockIdx.x * (blockDim.x >> 5) + warp;
     if (r >= rows) return;
-    router_topk256_row<false>(logits + (int64_t)r * E, bias, E, top_k, ids + (int64_t)r * top_k, weights + (int64_t)r * top_k, lane);
+    router_topk256_row<false>(logits + (int64_t)r * stride, bias, E, top_k, normalize != 0, ids + (int64_t)r * top_k, weights + (int64_t)r * top_k, lane);
 }
 
 // ---------------------------------------------------------------------------------------------------
@@ -211,13 +211,14 @@ __global__ void fill_uniform_f32_kernel(float* __restrict__ out, int64_t n, uint
 }
 
 // ===================================================================================================
-GLMB_API int glmb_router_topk(const float* logits, const float* bias, int rows, int E, int top_k, int* ids, float* weights,
-                              void* stream) {
-    if (E > 1024 || top_k > 32 || top_k > E) return 1;
+// logits: rows of E scores, `stride` apart; bias may be NULL; normalize: the weights are the chosen scores over their sum.
+GLMB_API int glmb_router_topk(const float* logits, int64_t stride, const float* bias, int rows, int E, int top_k, int normalize, int* ids,
+                              float* weights, void* stream) {
+    if (E > 1024 || top_k > 32 || top_k > E || stride < E) return 1;
     if (E <= 256)
-        GLMB_LAUNCH(router_topk256_kernel, ceil_div(rows, 4), 128, 0, (cudaStream_t)stream, logits, bias, rows, E, top_k, ids, weights);
+        GLMB_LAUNCH(router_topk256_kernel, ceil_div(rows, 4), 128, 0, (cudaStream_t)stream, logits, stride, bias, rows, E, top_k, normalize, ids, weights);
     else
-        GLMB_LAUNCH(router_topk_kernel, ceil_div(rows, 4), 128, 0, (cudaStream_t)stream, logits, bias, rows, E, top_k, ids, weights);
+        GLMB_LAUNCH(router_topk_kernel, ceil_div(rows, 4), 128, 0, (cudaStream_t)stream, logits, stride, bias, rows, E, top_k, normalize, ids, weights);
     return (int)cudaGetLastError();
 }
 

@@ -35,7 +35,7 @@ template <typename T, int THREADS, int REGS>
 __global__ void __launch_bounds__(THREADS)
 parallel_norm_kernel(const int* __restrict__ tokens, const T* __restrict__ table, int vocab, const float* __restrict__ update,
                      float* __restrict__ residual, int width, int padded, const T* __restrict__ w1, const T* __restrict__ w2,
-                     T* __restrict__ out1, T* __restrict__ out2, float eps, uint32_t* status) {
+                     T* __restrict__ out1, T* __restrict__ out2, float eps, float table_scale, float w_offset, uint32_t* status) {
     GLMB_PDL_PROLOGUE();
     __shared__ float scratch[THREADS / 32];
     const int64_t base = (int64_t)blockIdx.x * padded;
@@ -61,6 +61,8 @@ parallel_norm_kernel(const int* __restrict__ tokens, const T* __restrict__ table
         float x[8];
         if (source) {
             load8(source + v, x);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) x[e] *= table_scale;
         } else {
             load8(res + v, x);
             if (update) {
@@ -98,12 +100,12 @@ parallel_norm_kernel(const int* __restrict__ tokens, const T* __restrict__ table
         for (int e = 0; e < 8; ++e) x[e] = x[e] / denom;
         if (slot || !early) load8(w1 + v, wa);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) y[e] = x[e] * wa[e];
+        for (int e = 0; e < 8; ++e) y[e] = x[e] * (w_offset + wa[e]);
         store8(out1 + base + v, y);
         if (w2) {
             if (slot || !early) load8(w2 + v, wb);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) y[e] = x[e] * wb[e];
+            for (int e = 0; e < 8; ++e) y[e] = x[e] * (w_offset + wb[e]);
             store8(out2 + base + v, y);
         }
     }
@@ -183,15 +185,16 @@ dual_proj_kernel(const bf16* __restrict__ x1, const bf16* __restrict__ x2, int64
 
 // ===================================================================================================
 // tokens != NULL: the residual starts from the embedding `table` [vocab, padded]; update != NULL: residual += update first.
+// The embedding is multiplied by table_scale; w_offset is added to the weights (1 for weights stored around zero).
 // w2 / out2 may be NULL (one normalized output).  All rows are `padded` elements (a multiple of 8), 16-byte aligned.
 GLMB_API int glmb_parallel_norm(const int* tokens, const void* table, int vocab, const float* update, float* residual, int rows, int width,
-                                int padded, const void* w1, const void* w2, void* out1, void* out2, float eps, int is_f32, uint32_t* status,
-                                void* stream) {
+                                int padded, const void* w1, const void* w2, void* out1, void* out2, float eps, float table_scale, float w_offset,
+                                int is_f32, uint32_t* status, void* stream) {
     if (rows < 1 || width < 1 || padded < width || (padded & 7) || (tokens && update) || (tokens && (!table || vocab < 1)) || (w2 && !out2)) return 1;
     cudaStream_t st = (cudaStream_t)stream;
 #define CALL(T, THREADS, REGS)                                                                                                             \
     GLMB_LAUNCH((parallel_norm_kernel<T, THREADS, REGS>), rows, THREADS, 0, st, tokens, (const T*)table, vocab, update, residual, width, padded, \
-                (const T*)w1, (const T*)w2, (T*)out1, (T*)out2, eps, status)
+                (const T*)w1, (const T*)w2, (T*)out1, (T*)out2, eps, table_scale, w_offset, status)
     if (rows <= PN_FEW_ROWS) {
         if (is_f32) CALL(float, 512, 1);
         else CALL(bf16, 512, 1);

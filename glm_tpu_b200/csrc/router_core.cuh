@@ -4,16 +4,17 @@
 #include "common.cuh"
 
 // Router choice of one row by one warp (E <= 256): sigmoid scores, the correction bias enters the choice only, ties to the lowest
-// expert id, fp32 weights normalised over the chosen scores.  FRESH: read the logits past the L1 (they were written by other CTAs of a launch still in flight).
+// expert id, fp32 weights: the chosen scores, normalised over them if asked.  bias may be NULL.  FRESH: read the logits past the L1 (they were written by other CTAs of a launch still in flight).
 template <bool FRESH>
-__device__ __forceinline__ void router_topk256_row(const float* lg, const float* bias, int E, int top_k, int* ids, float* weights, int lane) {
+__device__ __forceinline__ void router_topk256_row(const float* lg, const float* bias, int E, int top_k, bool normalize, int* ids, float* weights,
+                                                   int lane) {
     float lv[8], bv[8], sc[8];
     uint32_t key[8];
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
         const int e = lane + 32 * i;
         lv[i] = e < E ? (FRESH ? __ldcg(lg + e) : lg[e]) : 0.f;
-        bv[i] = e < E ? bias[e] : 0.f;
+        bv[i] = bias && e < E ? bias[e] : 0.f;
     }
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
@@ -46,5 +47,5 @@ __device__ __forceinline__ void router_topk256_row(const float* lg, const float*
         picked_sum += best_score;
         if (lane == 0) ids[s] = best_e == 0x7fffffff ? 0 : best_e;
     }
-    if (lane < top_k) weights[lane] = my_score / (picked_sum + 1e-20f);
+    if (lane < top_k) weights[lane] = normalize ? my_score / (picked_sum + 1e-20f) : my_score;
 }

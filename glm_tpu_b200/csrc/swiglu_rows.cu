@@ -34,11 +34,11 @@ GLMB_API int glmb_swiglu_rows(const void* gate, const void* up, void* act, int64
 }
 
 // Gated activation of strided rows: act[r][i] = f(gate[r][i]) * up[r][i] for i < n (a multiple of 8), f by `kind` (vec8.cuh), arithmetic
-// in fp32 and one rounding.  gate and up may be the two halves of one projection's output, act the tail of a wider row.
+// in fp32 and one rounding; with `scale`, both are first multiplied by scale[r], or by scale[scale_at[r]] (0 where that is negative).  gate and up may be the two halves of one projection's output, act the tail of a wider row.
 template <typename T>
 __global__ void __launch_bounds__(256)
 glu_rows_kernel(const T* __restrict__ gate, const T* __restrict__ up, int64_t in_stride, T* __restrict__ act, int64_t out_stride, int rows, int n,
-                int kind) {
+                int kind, const float* __restrict__ scale, const int* __restrict__ scale_at) {
     GLMB_PDL_PROLOGUE();
     const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
     if (c >= n) return;
@@ -46,6 +46,12 @@ glu_rows_kernel(const T* __restrict__ gate, const T* __restrict__ up, int64_t in
         float g[8], u[8];
         load8(gate + r * in_stride + c, g);
         load8(up + r * in_stride + c, u);
+        if (scale) {
+            const int at = scale_at ? scale_at[r] : r;
+            const float w = at >= 0 ? scale[at] : 0.f;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) { g[e] *= w; u[e] *= w; }
+        }
 #pragma unroll
         for (int e = 0; e < 8; ++e) g[e] = glu_activation(kind, g[e]) * u[e];
         store8(act + r * out_stride + c, g);
@@ -53,16 +59,16 @@ glu_rows_kernel(const T* __restrict__ gate, const T* __restrict__ up, int64_t in
 }
 
 // n and both strides multiples of 8 elements, all pointers 16-byte aligned.
-GLMB_API int glmb_glu_rows(const void* gate, const void* up, int64_t in_stride, void* act, int64_t out_stride, int rows, int n, int kind, int is_f32,
-                           void* stream) {
+GLMB_API int glmb_glu_rows(const void* gate, const void* up, int64_t in_stride, void* act, int64_t out_stride, int rows, int n, int kind, const float* scale,
+                           const int* scale_at, int is_f32, void* stream) {
     if (rows < 1 || n < 8 || (n & 7) || (in_stride & 7) || (out_stride & 7) || (kind != GLU_SILU && kind != GLU_GELU_TANH)) return 1;
     if ((reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(up) | reinterpret_cast<uintptr_t>(act)) & 15) return 1;
     const dim3 grid(ceil_div(n / 8, 256), rows < 32768 ? rows : 32768);
     if (is_f32)
         GLMB_LAUNCH(glu_rows_kernel<float>, grid, 256, 0, (cudaStream_t)stream, (const float*)gate, (const float*)up, in_stride, (float*)act, out_stride,
-                    rows, n, kind);
+                    rows, n, kind, scale, scale_at);
     else
         GLMB_LAUNCH(glu_rows_kernel<bf16>, grid, 256, 0, (cudaStream_t)stream, (const bf16*)gate, (const bf16*)up, in_stride, (bf16*)act, out_stride,
-                    rows, n, kind);
+                    rows, n, kind, scale, scale_at);
     return (int)cudaGetLastError();
 }

@@ -27,7 +27,8 @@ import torch
 
 from glm_tpu_b200.config.cache import RingCacheConfig
 from glm_tpu_b200.exceptions import PlanValidationError
-from glm_tpu_b200.models.namizen.weights import NamizenWeights, pad8, pad16
+from glm_tpu_b200.model_loader.directory import pad8, pad16
+from glm_tpu_b200.models.namizen.weights import NamizenWeights
 from glm_tpu_b200.ops import native
 from glm_tpu_b200.parallel.peer import PeerGroup
 from glm_tpu_b200.runner.lane_state import RING, LaneRegisters

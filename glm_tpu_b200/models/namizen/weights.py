@@ -1,7 +1,6 @@
 """Namizen weights: the checkpoint mapping, random fixtures, and the tables one GPU keeps.
 
-The checkpoint is a flat ``name -> tensor`` mapping (``NamizenGeometry.tensor_shapes``), read from the safetensors files of a directory
-through the same streaming reader the packed checkpoints use.
+The checkpoint is a flat ``name -> tensor`` mapping (``NamizenGeometry.tensor_shapes``), e.g. ``model_loader.directory.SourceTensors``.
 
 Resident tables are laid out for the kernels: every row is padded to a multiple of 8 columns (zeros), so any width, head size or
 feed-forward size meets the alignment of the tensor-core and streaming kernels; q, k and v are one table, gate and up are one table, and the
@@ -13,41 +12,12 @@ from __future__ import annotations
 
 from collections.abc import Mapping
 from dataclasses import dataclass
-from pathlib import Path
 
 import torch
 
 from glm_tpu_b200.config.namizen import NamizenGeometry
 from glm_tpu_b200.exceptions import CheckpointValidationError
-from glm_tpu_b200.model_loader.sharded_state import format as fmt
-
-
-def pad8(n: int) -> int:
-    return (n + 7) // 8 * 8
-
-
-def pad16(n: int) -> int:
-    return (n + 15) // 16 * 16
-
-
-class SourceTensors(Mapping):
-    """``name -> tensor`` over the ``*.safetensors`` files of a directory; a tensor is streamed to ``device`` when it is looked up."""
-
-    def __init__(self, root: Path, device=None):
-        from glm_tpu_b200.model_loader.source_inventory import read_source_inventory
-
-        self.device = device
-        self._where = {name: t.shard for name, t in read_source_inventory(root).tensors.items()}
-        self._readers = {shard: fmt.TensorReader(Path(root) / shard) for shard in sorted(set(self._where.values()))}
-
-    def __getitem__(self, name: str) -> torch.Tensor:
-        return self._readers[self._where[name]].read(name, device=self.device)
-
-    def __iter__(self):
-        return iter(self._where)
-
-    def __len__(self) -> int:
-        return len(self._where)
+from glm_tpu_b200.model_loader.directory import pad8, padded
 
 
 def check_tensors(g: NamizenGeometry, tensors: Mapping, shape_of=None) -> None:
@@ -115,12 +85,6 @@ class NamizenWeights:
         self.bytes_resident = sum(t.numel() * t.element_size() for t in tables)
 
 
-def _padded(t: torch.Tensor, rows: int, cols: int, dtype, device) -> torch.Tensor:
-    out = torch.zeros((rows, cols), dtype=dtype, device=device)
-    out[: t.shape[0], : t.shape[1]] = t.to(device=device, dtype=dtype)
-    return out
-
-
 def resident_weights(g: NamizenGeometry, tensors: Mapping, device, dtype: torch.dtype = torch.bfloat16) -> NamizenWeights:
     """The tables of one GPU from a checkpoint mapping (each tensor is asked for once)."""
     check_tensors(g, tensors)
@@ -134,7 +98,7 @@ def resident_weights(g: NamizenGeometry, tensors: Mapping, device, dtype: torch.
         return t
 
     def row(name: str) -> torch.Tensor:
-        return _padded(get(name)[None, :], 1, Wp, dtype, dev)[0]
+        return padded(get(name)[None, :], 1, Wp, dtype, dev)[0]
 
     layers = []
     for i, spec in enumerate(g.layers):
@@ -161,28 +125,14 @@ def resident_weights(g: NamizenGeometry, tensors: Mapping, device, dtype: torch.
             norm1=row(p + ".norm1"), norm2=row(p + ".norm2") if spec.ff else None, qkv=qkv, conv=conv.contiguous(), gate_up=gate_up, out=out,
             sink=get(p + ".mix.sink").to(device=dev, dtype=torch.float32).contiguous(), mix=float(get(p + ".mix.vmix")) if mixes else 0.0,
             attn_cols=attn_cols, ff_cols=ff_cols))
-    return NamizenWeights(g, dtype, embed=_padded(get("embed"), g.vocab_size, Wp, dtype, dev), layers=layers, final_norm=row("final.norm"),
-                          head=_padded(get("head"), pad8(g.vocab_size), Wp, dtype, dev))
+    return NamizenWeights(g, dtype, embed=padded(get("embed"), g.vocab_size, Wp, dtype, dev), layers=layers, final_norm=row("final.norm"),
+                          head=padded(get("head"), pad8(g.vocab_size), Wp, dtype, dev))
 
 
-class DeviceRandomTensors(Mapping):
-    """Random bf16 tensors made on the GPU one at a time (speed measurements at full size: nothing passes through host memory)."""
-
-    def __init__(self, g: NamizenGeometry, device, seed: int = 0):
-        self._shapes, self.device, self.seed = g.tensor_shapes(), torch.device(device), seed
-
-    def __getitem__(self, name: str) -> torch.Tensor:
-        from glm_tpu_b200.ops import native
-
-        shape = self._shapes[name]
-        out = torch.empty(shape, dtype=torch.bfloat16, device=self.device)
-        norm = "norm" in name
-        std = 0.1 if norm else 1.0 if name == "embed" else shape[-1] ** -0.5 if shape else 0.0
-        native.fill_random_bf16(out, self.seed * 4096 + list(self._shapes).index(name), 1.0 if norm else 0.5 if not shape else 0.0, std)
-        return out
-
-    def __iter__(self):
-        return iter(self._shapes)
-
-    def __len__(self) -> int:
-        return len(self._shapes)
+def random_spread(name: str, shape) -> tuple[float, float]:
+    """Mean and standard deviation of the tensors that are made on the device (``DeviceRandomTensors``)."""
+    if "norm" in name:
+        return 1.0, 0.1
+    if not shape:
+        return 0.5, 0.0
+    return 0.0, 1.0 if name == "embed" else shape[-1] ** -0.5

@@ -14,6 +14,7 @@ from typing import Any, Callable, Mapping
 
 from glm_tpu_b200.config import model as glm_config
 from glm_tpu_b200.config import namizen as namizen_config
+from glm_tpu_b200.config import zikevik as zikevik_config
 from glm_tpu_b200.exceptions import ConfigValidationError
 
 
@@ -92,58 +93,89 @@ GLM = Family(
     small_enough_for_host=lambda g: g.num_layers <= 8 and g.hidden_size <= 1024, next_token=_glm_next_token)
 
 
-# ------------------------------------------------------------------------------------------------ Namizen
-def _namizen_load(path: Path, rank: int = 0, world: int = 1, *, pins=None, device=None):
-    from glm_tpu_b200.exceptions import CheckpointValidationError
-    from glm_tpu_b200.models.namizen.weights import SourceTensors
+# ------------------------------------------------------------------------------------------------ one-GPU families read from a directory
+def _load_directory(architecture: str):
+    def load(path: Path, rank: int = 0, world: int = 1, *, pins=None, device=None):
+        from glm_tpu_b200.exceptions import CheckpointValidationError
+        from glm_tpu_b200.model_loader.directory import SourceTensors
 
-    if any((pins or {}).values()):
-        raise CheckpointValidationError("the site pins a packed checkpoint; a Namizen directory has no manifest to pin")
-    return SourceTensors(path, device=device)
+        if any((pins or {}).values()):
+            raise CheckpointValidationError(f"the site pins a packed checkpoint; a {architecture} directory has no manifest to pin")
+        return SourceTensors(path, device=device)
 
-
-def _namizen_random(geometry, seed: int = 0):
-    from glm_tpu_b200.models.namizen.weights import random_checkpoint
-
-    return random_checkpoint(geometry, seed=seed)
+    return load
 
 
-def _namizen_next_token(geometry, checkpoint, capacity: int):
-    import torch
-
-    from glm_tpu_b200.oracle import namizen as oracle
-
-    config, tensors = geometry.to_config(), dict(checkpoint.items())
-    return lambda sequence: int(torch.argmax(oracle.forward(config, tensors, sequence, dtype=torch.float32)[-1]))
+def _matches(architecture: str):
+    return lambda config: config.get("architecture") == architecture
 
 
-def _namizen_runner(geometry, **kwargs):
-    from glm_tpu_b200.runner.namizen_runner import build
+def _is_directory_of(architecture: str):
+    def is_checkpoint(path: Path) -> bool:
+        try:
+            return _matches(architecture)(_read_config(path))
+        except ConfigValidationError:
+            return False
 
-    return build(geometry, **kwargs)
-
-
-def _namizen_matches(config: Mapping) -> bool:
-    return config.get("architecture") == namizen_config.ARCHITECTURE
-
-
-def _namizen_is_checkpoint(path: Path) -> bool:
-    try:
-        return _namizen_matches(_read_config(path))
-    except ConfigValidationError:
-        return False
+    return is_checkpoint
 
 
-NAMIZEN = Family(
-    name="namizen", architecture=namizen_config.ARCHITECTURE, geometry_type=namizen_config.NamizenGeometry,
-    presets={"namizen-tiny": namizen_config.tiny_namizen}, library_component="namizen", dtypes=("bfloat16", "float32"),
-    from_config=namizen_config.NamizenGeometry.from_config, matches=_namizen_matches, is_checkpoint=_namizen_is_checkpoint,
-    read_geometry=lambda path: namizen_config.NamizenGeometry.from_config(_read_config(path)),
-    load_checkpoint=_namizen_load, load_full_checkpoint=_namizen_load, random_checkpoint=_namizen_random,
-    small_enough_for_host=lambda g: g.num_layers <= 16 and g.hidden_size <= 1024, next_token=_namizen_next_token,
-    build_runner=_namizen_runner, multi_gpu=False)
+def _random_weights(package: str):
+    def random(geometry, seed: int = 0):
+        import importlib
 
-FAMILIES = (GLM, NAMIZEN)
+        return importlib.import_module(f"glm_tpu_b200.models.{package}.weights").random_checkpoint(geometry, seed=seed)
+
+    return random
+
+
+def _oracle_next_token(module: str):
+    def next_token(geometry, checkpoint, capacity: int):
+        import importlib
+
+        import torch
+
+        oracle = importlib.import_module(f"glm_tpu_b200.oracle.{module}")
+        config, tensors = geometry.to_config(), dict(checkpoint.items())
+        return lambda sequence: int(torch.argmax(oracle.forward(config, tensors, sequence, dtype=torch.float32)[-1]))
+
+    return next_token
+
+
+def _runner_of(module: str):
+    def build(geometry, **kwargs):
+        import importlib
+
+        return importlib.import_module(f"glm_tpu_b200.runner.{module}").build(geometry, **kwargs)
+
+    return build
+
+
+def _directory_family(name: str, architecture: str, geometry_type: type, presets: Mapping, read_geometry: Callable[[Path], Any]) -> Family:
+    """A family that runs on one GPU, from ``config.json`` and safetensors, with modules called after it."""
+    load = _load_directory(architecture)
+    return Family(
+        name=name, architecture=architecture, geometry_type=geometry_type, presets=presets, library_component=name, dtypes=("bfloat16", "float32"),
+        from_config=geometry_type.from_config, matches=_matches(architecture), is_checkpoint=_is_directory_of(architecture),
+        read_geometry=read_geometry, load_checkpoint=load, load_full_checkpoint=load, random_checkpoint=_random_weights(name),
+        small_enough_for_host=lambda g: g.num_layers <= 16 and g.hidden_size <= 1024, next_token=_oracle_next_token(name),
+        build_runner=_runner_of(f"{name}_runner"), multi_gpu=False)
+
+
+NAMIZEN = _directory_family("namizen", namizen_config.ARCHITECTURE, namizen_config.NamizenGeometry, {"namizen-tiny": namizen_config.tiny_namizen},
+                            lambda path: namizen_config.NamizenGeometry.from_config(_read_config(path)))
+
+
+def _zikevik_geometry(path: Path):
+    from glm_tpu_b200.model_loader.directory import SourceTensors
+
+    return zikevik_config.ZikevikGeometry.from_config(_read_config(path), SourceTensors(path).shapes)
+
+
+ZIKEVIK = _directory_family("zikevik", zikevik_config.ARCHITECTURE, zikevik_config.ZikevikGeometry, {"zikevik-tiny": zikevik_config.tiny_zikevik},
+                            _zikevik_geometry)
+
+FAMILIES = (GLM, NAMIZEN, ZIKEVIK)
 
 
 def family_of(geometry) -> Family:

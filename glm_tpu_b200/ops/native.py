@@ -85,9 +85,9 @@ class QkvConvArgs(C.Structure):
 
 class ChunkAttnArgs(C.Structure):
     _fields_ = [
-        ("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("sink", C.c_void_p),
+        ("q", C.c_void_p), ("q_stride", C.c_int64), ("k", C.c_void_p), ("v", C.c_void_p), ("sink", C.c_void_p),
         ("row_pos", C.c_void_p), ("row_lane", C.c_void_p), ("row_active", C.c_void_p),
-        ("out", C.c_void_p), ("out_stride", C.c_int64),
+        ("out", C.c_void_p), ("out_stride", C.c_int64), ("gate", C.c_void_p), ("gate_stride", C.c_int64),
         ("rows", C.c_int), ("H", C.c_int), ("G", C.c_int), ("dim", C.c_int), ("dimp", C.c_int), ("vdim", C.c_int), ("vdimp", C.c_int),
         ("decode", C.c_int), ("start", C.c_int), ("base", C.c_int), ("keys", C.c_int),
         ("chunk", C.c_int), ("ring", C.c_int), ("capacity", C.c_int), ("lanes", C.c_int),
@@ -95,6 +95,47 @@ class ChunkAttnArgs(C.Structure):
         ("status", C.c_void_p),
     ]
 
+
+class LatentArgs(C.Structure):
+    _fields_ = [
+        ("proj", C.c_void_p), ("proj_stride", C.c_int64),
+        ("off_kv", C.c_int), ("off_gate", C.c_int),
+        ("q_norm", C.c_void_p), ("kv_norm", C.c_void_p), ("rot", C.c_void_p),
+        ("row_pos", C.c_void_p), ("row_lane", C.c_void_p), ("row_active", C.c_void_p),
+        ("cq", C.c_void_p), ("cq_stride", C.c_int64),
+        ("cache", C.c_void_p), ("q", C.c_void_p), ("uk", C.c_void_p), ("qa", C.c_void_p), ("o_lat", C.c_void_p), ("uv", C.c_void_p),
+        ("out", C.c_void_p), ("out_stride", C.c_int64),
+        ("rows", C.c_int), ("H", C.c_int), ("dim", C.c_int), ("rot_dim", C.c_int), ("dimp", C.c_int), ("vdim", C.c_int), ("q_rank", C.c_int),
+        ("kv_rank", C.c_int), ("lat", C.c_int), ("pe", C.c_int), ("lanes", C.c_int), ("capacity", C.c_int),
+        ("eps", C.c_float),
+        ("status", C.c_void_p),
+    ]
+
+
+class DeltaArgs(C.Structure):
+    _fields_ = [
+        ("proj", C.c_void_p), ("proj_stride", C.c_int64),
+        ("off_b", C.c_int),
+        ("conv_w", C.c_void_p), ("taps", C.c_int),
+        ("conv_state", C.c_void_p),
+        ("a", C.c_void_p), ("a_stride", C.c_int64),
+        ("a_rate", C.c_void_p), ("dt_bias", C.c_void_p),
+        ("row_pos", C.c_void_p), ("row_lane", C.c_void_p), ("row_active", C.c_void_p),
+        ("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("lg", C.c_void_p), ("beta", C.c_void_p),
+        ("state", C.c_void_p), ("o", C.c_void_p),
+        ("gate", C.c_void_p), ("gate_stride", C.c_int64),
+        ("norm", C.c_void_p),
+        ("out", C.c_void_p), ("out_stride", C.c_int64),
+        ("H", C.c_int), ("G", C.c_int), ("dim", C.c_int), ("dimp", C.c_int), ("vdim", C.c_int), ("rows", C.c_int), ("decode", C.c_int),
+        ("lanes", C.c_int), ("capacity", C.c_int), ("rows_per_block", C.c_int),
+        ("eps", C.c_float),
+        ("status", C.c_void_p),
+    ]
+
+
+# argument structures and the entry point that gives their size in the library
+_STRUCTS = (("glmb_qkv_conv_args_sizeof", QkvConvArgs), ("glmb_chunk_attn_args_sizeof", ChunkAttnArgs), ("glmb_latent_args_sizeof", LatentArgs),
+            ("glmb_delta_args_sizeof", DeltaArgs))
 
 _lib = None
 
@@ -125,7 +166,9 @@ def lib() -> C.CDLL:
         _lib.glmb_peer_status_ptr.restype = C.c_void_p
         if hasattr(_lib, "glmb_indexer_rows_scratch_bytes"):  # a component library holds one family's kernels only
             _lib.glmb_indexer_rows_scratch_bytes.restype = C.c_int64
-        for entry, struct in (("glmb_qkv_conv_args_sizeof", QkvConvArgs), ("glmb_chunk_attn_args_sizeof", ChunkAttnArgs)):
+        for entry, struct in _STRUCTS:
+            if not hasattr(_lib, entry):  # a component library holds one family's kernels only
+                continue
             getattr(_lib, entry).restype = C.c_size_t
             if getattr(_lib, entry)() != C.sizeof(struct):
                 raise RuntimeError(f"{struct.__name__} layout differs between Python and the CUDA library")
@@ -351,11 +394,12 @@ def swiglu_rows(gate, up, act=None):
     return act
 
 
-def glu_rows(gate, up, act, kind):
-    """``act[r, :n] = f(gate[r]) * up[r]`` for strided rows (``kind``: ``GLU_SILU`` or ``GLU_GELU_TANH``); bf16 or fp32, fp32 arithmetic."""
+def glu_rows(gate, up, act, kind, *, scale=None, scale_at=None):
+    """``act[r, :n] = f(gate[r]) * up[r]`` for strided rows (``kind``: ``GLU_SILU`` or ``GLU_GELU_TANH``); bf16 or fp32, fp32 arithmetic.
+    ``scale`` (fp32) multiplies both inputs of row ``r`` by ``scale[r]``, or by ``scale[scale_at[r]]`` (0 where that index is negative)."""
     rows, n = gate.shape
     _check(lib().glmb_glu_rows(_p(gate), _p(up), C.c_int64(gate.stride(0)), _p(act), C.c_int64(act.stride(0)), rows, n, int(kind),
-                               int(gate.dtype == torch.float32), _stream()), "glu_rows")
+                               _p(scale), _p(scale_at), int(gate.dtype == torch.float32), _stream()), "glu_rows")
 
 
 def route_sort128(topk_ids, ebase: int, el: int, tiles, n_tiles, perm) -> None:
@@ -414,12 +458,14 @@ def add_rmsnorm(update, residual, weight, out, eps):
     _check(lib().glmb_add_rmsnorm(_p(update), _p(residual), _p(weight), _p(out), rows, H, f32(eps), _stream()), "add_rmsnorm")
 
 
-def parallel_norm(residual, width, w1, out1, eps, *, w2=None, out2=None, update=None, tokens=None, table=None, vocab=0, status=None):
-    """Both RMS-normalized inputs of a parallel layer from one fp32 residual: ``residual += update`` (fp32), or ``residual =
-    table[tokens]``, first; then ``out = residual / sqrt(mean(residual**2) + eps) * w``.  Rows are padded to a multiple of 8 columns."""
+def parallel_norm(residual, width, w1, out1, eps, *, w2=None, out2=None, update=None, tokens=None, table=None, vocab=0, table_scale=1.0,
+                  weight_offset=0.0, status=None):
+    """One or both RMS-normalized inputs of a layer from one fp32 residual: ``residual += update`` (fp32), or ``residual = table[tokens] *
+    table_scale``, first; then ``out = residual / sqrt(mean(residual**2) + eps) * (weight_offset + w)``.  Rows are padded to a multiple of 8
+    columns."""
     rows, padded = out1.shape
     _check(lib().glmb_parallel_norm(_p(tokens), _p(table), int(vocab), _p(update), _p(residual), rows, int(width), padded, _p(w1), _p(w2), _p(out1),
-                                    _p(out2), f32(eps), int(out1.dtype == torch.float32), _p(status), _stream()), "parallel_norm")
+                                    _p(out2), f32(eps), f32(table_scale), f32(weight_offset), int(out1.dtype == torch.float32), _p(status), _stream()), "parallel_norm")
 
 
 def dual_proj(x1, w, out, x2=None, wg=None, wu=None, act=None, kind=GLU_SILU):
@@ -492,6 +538,74 @@ def q_absorb(q_nope, rows, kv_b, heads_local, head_base, heads_total, nope, vdim
                             C.c_int64(q_full_offset), _comm(comm), sig, _stream()),
         "q_absorb",
     )
+
+
+# ----------------------------------------------------------------------------- attention over a shared latent, gated delta rule
+def latent_rows(args: LatentArgs, is_f32: bool) -> None:
+    """Projection rows -> normalized query latent, and the cache rows (normalized latent, rotated key part)."""
+    _check(lib().glmb_latent_rows(C.byref(args), int(is_f32), _stream()), "latent_rows")
+
+
+def latent_query(args: LatentArgs, is_f32: bool) -> None:
+    """Rotates the rotated part of every query head in place."""
+    _check(lib().glmb_latent_query(C.byref(args), int(is_f32), _stream()), "latent_query")
+
+
+def latent_absorb(args: LatentArgs, is_f32: bool) -> None:
+    """Query heads in the coordinates of the cache rows."""
+    _check(lib().glmb_latent_absorb(C.byref(args), int(is_f32), _stream()), "latent_absorb")
+
+
+def latent_value(args: LatentArgs, is_f32: bool) -> None:
+    """Per-head value projection of the attended latent, times the head's output gate."""
+    _check(lib().glmb_latent_value(C.byref(args), int(is_f32), _stream()), "latent_value")
+
+
+def delta_max_taps() -> int:
+    return int(lib().glmb_delta_max_taps())
+
+
+def delta_prep(args: DeltaArgs, is_f32: bool) -> None:
+    """Convolution, activation, unit vectors, decay and write strength of a delta-rule layer; advances the convolution's state."""
+    _check(lib().glmb_delta_prep(C.byref(args), int(is_f32), _stream()), "delta_prep")
+
+
+def delta_scan(args: DeltaArgs) -> None:
+    """The recurrence, token by token."""
+    _check(lib().glmb_delta_scan(C.byref(args), _stream()), "delta_scan")
+
+
+def delta_out(args: DeltaArgs, is_f32: bool) -> None:
+    """Norm per head and output gate of what the recurrence read."""
+    _check(lib().glmb_delta_out(C.byref(args), int(is_f32), _stream()), "delta_out")
+
+
+# ----------------------------------------------------------------------------- routed experts, unquantized, weight on the input
+def expert_glu(x, ids, weights, gate_up, act, kind, *, status=None):
+    """``act[route] = f(w x Wg_e^T) * (w x Wu_e^T)`` for the routes of ``ids`` / ``weights`` ``[rows, top]``; ``gate_up``: ``[E, 2 F, K]``."""
+    rows, top = ids.shape
+    E, F2, K = gate_up.shape
+    _check(lib().glmb_expert_glu(_p(x), C.c_int64(x.stride(0)), rows, top, _p(ids), _p(weights), _p(gate_up), E, F2 // 2, K, int(kind), _p(act),
+                                 int(x.dtype == torch.float32), _p(status), _stream()), "expert_glu")
+
+
+def expert_down(act, ids, down, out):
+    """``out[row] = sum over the row's routes of act[route] Wd_e^T`` (fp32); ``down``: ``[E, N, F]``."""
+    rows, top = ids.shape
+    E, N, F = down.shape
+    _check(lib().glmb_expert_down(_p(act), rows, top, _p(ids), _p(down), E, N, F, _p(out), C.c_int64(out.stride(0)), int(act.dtype == torch.float32),
+                                  _stream()), "expert_down")
+
+
+def gather_routes(src, perm, top, place, dst):
+    """Rows of ``src`` into the order of ``perm`` (route ids; zeros where negative); ``place`` becomes the inverse of ``perm``."""
+    _check(lib().glmb_gather_routes(_p(src), C.c_int64(src.stride(0)), _p(perm), dst.shape[0], int(top), _p(place), _p(dst), dst.shape[1], _stream()),
+           "gather_routes")
+
+
+def route_combine(y, place, top, out):
+    """``out[row] = sum over slots of y[place[row * top + slot]]`` (fp32, in slot order)."""
+    _check(lib().glmb_route_combine(_p(y), _p(place), out.shape[0], int(top), _p(out), out.shape[1], _stream()), "route_combine")
 
 
 # ----------------------------------------------------------------------------- indexer
@@ -642,9 +756,11 @@ def attn_final_merge(rows, L, heads_local, xpart_offset, o_lat, comm, sig=SIG_AT
 
 
 # ----------------------------------------------------------------------------- router / sampler / misc
-def router_topk(logits, bias, top_k, ids, weights):
+def router_topk(logits, bias, top_k, ids, weights, *, normalize=True):
+    """The ``top_k`` experts with the largest ``sigmoid(logits) + bias`` per row and their sigmoid scores, over their sum if ``normalize``."""
     rows, E = logits.shape
-    _check(lib().glmb_router_topk(_p(logits), _p(bias), rows, E, top_k, _p(ids), _p(weights), _stream()), "router_topk")
+    _check(lib().glmb_router_topk(_p(logits), C.c_int64(logits.stride(0)), _p(bias), rows, E, top_k, int(normalize), _p(ids), _p(weights), _stream()),
+           "router_topk")
 
 
 def argmax_rows(logits, rows, V, vocab_base, cand, cand_offset=0, comm=None, sig=SIG_SAMPLE, status=None):

@@ -83,8 +83,8 @@ def check_collective_plan(plan: list[dict], *, world: int, ar_slice_floats: int 
             raise PlanValidationError(f"unknown exchange kind {op['kind']!r}")
 
 
-def project_ring_memory(cache, weight_bytes: int, workspace: int, hbm_bytes: int = HBM_BYTES) -> dict:
-    """The same projection for a model with ring caches on one GPU (no staging)."""
+def project_local_memory(cache, weight_bytes: int, workspace: int, hbm_bytes: int = HBM_BYTES) -> dict:
+    """The same projection for a one-GPU family (no staging)."""
     caches = cache.cache_bytes_per_gpu()
     total = weight_bytes + caches + workspace
     return {"weights": int(weight_bytes), "caches": int(caches), "staging": 0, "workspace": int(workspace), "total": int(total),

@@ -17,6 +17,7 @@ from glm_tpu_b200.engine import request as rq
 from glm_tpu_b200.engine.llm_engine import LLMEngine
 from glm_tpu_b200.entrypoints.cli import trace as trace_cli
 from glm_tpu_b200.exceptions import CheckpointValidationError, ConfigValidationError, PlanValidationError, RequestValidationError
+from glm_tpu_b200.model_loader.directory import pad8
 from glm_tpu_b200.model_loader.sharded_state import format as fmt
 from glm_tpu_b200.models import registry
 from glm_tpu_b200.models.namizen import weights as nw
@@ -241,7 +242,7 @@ def test_resident_tables_from_a_directory(tmp_path):
     assert set(tensors) == set(ck) and all(torch.equal(tensors[n], ck[n]) for n in ck) and len(tensors) == len(ck)
     w = nw.resident_weights(g, tensors, "cpu", torch.float32)
     lw = w.layers[0]
-    assert lw.qkv.shape == (nw.pad8(3 * 21 * 2 + 3 * 13), 104) and torch.equal(lw.qkv[:63, :100], ck["l0.mix.q"].float()) and not lw.qkv[:, 100:].any()
+    assert lw.qkv.shape == (pad8(3 * 21 * 2 + 3 * 13), 104) and torch.equal(lw.qkv[:63, :100], ck["l0.mix.q"].float()) and not lw.qkv[:, 100:].any()
     assert torch.equal(lw.qkv[126 : 126 + 39, :100], ck["l0.mix.v"].float()) and torch.equal(lw.conv[0, 63:126], ck["l0.mix.k.conv"][:, 0].float())
     assert torch.equal(lw.out[:100, :39], ck["l0.mix.o"].float()) and torch.equal(lw.out[:100, 40 : 40 + 51], ck["l0.mlp.down"].float())
     assert not lw.out[:, 39].any() and lw.mix == 0.0 and w.layers[2].mix == float(ck["l2.mix.vmix"]) and w.layers[1].gate_up is None
