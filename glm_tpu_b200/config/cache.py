@@ -210,8 +210,8 @@ class HybridCacheConfig:
 
     A latent layer keeps one row per position and lane, ``[normalized latent | rotated key part]``, both parts padded to a multiple of 16
     elements (whole tensor-core steps, 16-byte vectors).  A recurrent layer keeps, per lane and whatever the context, an fp32 state per head
-    (stored ``[vdim, dim]``: a value channel's row of key channels, padded to a multiple of 32) and the last ``taps - 1`` projected rows of its
-    convolution.
+    (stored ``[vdim, dim]``: a value channel's row of key channels, padded to a multiple of 32) and a ring of the last ``taps`` projected
+    rows for its convolution.
 
     ``geometry.layers[i].mixer`` gives the layer's sizes; a recurrent mixer has ``conv_width``, a latent one ``kv_rank``.
     """
@@ -246,7 +246,7 @@ class HybridCacheConfig:
 
     def conv_shape(self, layer: int) -> tuple[int, int, int]:
         m = self._mixer(layer)
-        return (self.lanes, m.conv - 1, m.conv_width)
+        return (self.lanes, m.conv, m.conv_width)
 
     def layer_bytes(self, layer: int) -> int:
         def count(shape):

@@ -6,12 +6,13 @@
 // vectors per head (q also scaled by dim^-1/2); beta = sigmoid; log g = -rate softplus(a + bias).  What is read out is normalized per head
 // and gated.
 //
-//   delta_prep   projection -> q, k, v, log g, beta (any sizes, decode and prefill); advances the convolution's state
+//   delta_prep   projection -> q, k, v, log g, beta (any sizes, decode and prefill); the convolution's history moves on
 //   delta_scan   the recurrence token by token: a thread keeps 4 DQ key channels of one value channel in registers, eight threads share a
 //                value channel; the two sums over key channels of a token are reduced together (o_t = S'^T q_t + (q_t . k_t) u_t)
 //   delta_out    root-mean-square norm per head, output gate
 //
-// Prefill: the rows are consecutive tokens of one sequence.  Decode: every row is the next token of its own sequence (lane).  A sequence at
+// The convolution's history is a ring of `taps` projected rows per lane (slot = position mod taps): a decode step writes a slot that none of
+// its readers needs.  Prefill: the rows are consecutive tokens of one sequence.  Decode: every row is the next token of its own sequence (lane).  A sequence at
 // position 0 starts from zeros whatever its lane held before.
 #include "attention_core.cuh"
 #include "common.cuh"
@@ -49,14 +50,14 @@ __global__ void __launch_bounds__(DR_THREADS) delta_prep_kernel(DeltaArgs a) {
     const int chan0 = kind == 0 ? slot * a.dim : kind == 1 ? (a.G + slot) * a.dim : 2 * a.G * a.dim + slot * a.vdim;
     const T* proj = reinterpret_cast<const T*>(a.proj) + chan0;
     const int state_lane = delta_lane(a, a.decode ? r0 : 0), keep = a.taps - 1;
-    T* state = reinterpret_cast<T*>(a.conv_state) + (int64_t)state_lane * keep * C + chan0;
+    T* ring = reinterpret_cast<T*>(a.conv_state) + (int64_t)state_lane * a.taps * C + chan0;
     auto conv = [&](int row, int pos, int c) {
         float y = 0.f;
         for (int j = 0; j < a.taps; ++j) {
             const int back = keep - j;
             if (back > pos) continue;  // before the sequence's start
             const bool here = a.decode ? back == 0 : row >= back;
-            const T u = here ? proj[(int64_t)(row - back) * a.proj_stride + c] : state[(int64_t)(keep - back + (a.decode ? 0 : row)) * C + c];
+            const T u = here ? proj[(int64_t)(row - back) * a.proj_stride + c] : ring[(int64_t)((pos - back) % a.taps) * C + c];
             y = fmaf(a.conv_w[(int64_t)j * C + chan0 + c], to_f32(u), y);
         }
         return delta_silu(y);
@@ -83,12 +84,13 @@ __global__ void __launch_bounds__(DR_THREADS) delta_prep_kernel(DeltaArgs a) {
             if (lane + 32 * i < a.dimp) dst[lane + 32 * i] = y[i] * scale;
     }
     if (!a.decode && blockIdx.x > 0) return;
-    __syncthreads();  // the first rows have read the state (no other block does: a block holds at least taps - 1 rows)
-    const int first = a.decode ? r0 : 0, seq = a.decode ? 1 : a.rows;
+    __syncthreads();  // the first rows have read the ring (no other block does: a block holds at least taps - 1 rows)
+    const int first = a.decode ? r0 : 0, rows = a.decode ? 1 : a.rows, kept = min(keep, rows);
     if (!delta_writes(a, first)) return;
-    for (int c = threadIdx.x; c < hd; c += DR_THREADS)
-        for (int j = 0; j < keep; ++j)  // ascending: entry j only reads later entries
-            state[(int64_t)j * C + c] = seq + j < keep ? state[(int64_t)(j + seq) * C + c] : proj[(int64_t)(first + seq - keep + j) * a.proj_stride + c];
+    for (int i = threadIdx.x; i < kept * hd; i += DR_THREADS) {
+        const int row = first + rows - kept + i / hd;
+        ring[(int64_t)(a.row_pos[row] % a.taps) * C + i % hd] = proj[(int64_t)row * a.proj_stride + i % hd];
+    }
 }
 
 // ---------------------------------------------------------------------------------------------------
@@ -195,11 +197,30 @@ __global__ void __launch_bounds__(DR_THREADS) delta_out_kernel(DeltaArgs a) {
     if (unit >= (int64_t)a.rows * a.H) return;
     const int row = (int)(unit / a.H), h = (int)(unit % a.H);
     const float* o = a.o + unit * a.vdim;
+    const T* gate = reinterpret_cast<const T*>(a.gate) + (int64_t)row * a.gate_stride + h * a.vdim;
+    T* out = reinterpret_cast<T*>(a.out) + (int64_t)row * a.out_stride + h * a.vdim;
+    if (!(a.vdim & 7) && a.vdim <= 256) {  // eight channels per lane, everything asked for at once
+        const int c = lane * 8;
+        float x[8], z[8], w[8], ss = 0.f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] = 0.f;
+        if (c < a.vdim) {
+            load8(o + c, x);
+            load8(gate + c, z);
+            load8(a.norm + c, w);
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss = fmaf(x[e], x[e], ss);
+        const float denom = sqrtf(warp_sum(ss) / (float)a.vdim + a.eps);
+        if (c >= a.vdim) return;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] = x[e] / denom * w[e] * sigmoidf_precise(z[e]);
+        store8(out + c, x);
+        return;
+    }
     float ss = 0.f;
     for (int c = lane; c < a.vdim; c += 32) ss = fmaf(o[c], o[c], ss);
     const float denom = sqrtf(warp_sum(ss) / (float)a.vdim + a.eps);
-    const T* gate = reinterpret_cast<const T*>(a.gate) + (int64_t)row * a.gate_stride + h * a.vdim;
-    T* out = reinterpret_cast<T*>(a.out) + (int64_t)row * a.out_stride + h * a.vdim;
     for (int c = lane; c < a.vdim; c += 32) from_f32(o[c] / denom * a.norm[c] * sigmoidf_precise(to_f32(gate[c])), out[c]);
 }
 

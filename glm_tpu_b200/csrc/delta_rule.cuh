@@ -7,7 +7,7 @@ struct DeltaArgs {
     const void* proj; int64_t proj_stride;       // [rows, q | k | v | beta logits at off_b | ..]
     int off_b;
     const float* conv_w; int taps;               // [taps, C], C = 2 G dim + H vdim
-    void* conv_state;                            // [lanes, taps - 1, C]
+    void* conv_state;                            // [lanes, taps, C]: slot = position mod taps
     const float* a; int64_t a_stride;            // [rows, H dim]: the decay's projection, before bias and softplus
     const float *a_rate, *dt_bias;               // [H] (positive), [H dim]
     const int *row_pos, *row_lane, *row_active;  // row_active may be NULL

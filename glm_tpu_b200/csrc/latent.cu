@@ -8,34 +8,8 @@
 //
 // A cache row is [latent | rotated key part], both padded to a multiple of 16 columns (zeros).  Pairs (2i, 2i + 1) of the rotated part turn by
 // the (cos, sin) of a fp32 table.  Templates over the element type: bf16 for serving, fp32 for the 32-bit path.
-#include "common.cuh"
+#include "latent_args.cuh"
 #include "vec8.cuh"
-
-struct LatentArgs {
-    const void* proj; int64_t proj_stride;       // [rows, query latent at 0 | key/value latent, key part at off_kv | gate logits at off_gate | ..]
-    int off_kv, off_gate;
-    const float *q_norm, *kv_norm;               // [q_rank], [kv_rank]
-    const float2* rot;                           // [capacity, rot / 2] (cos, sin)
-    const int *row_pos, *row_lane, *row_active;  // row_active may be NULL
-    void* cq; int64_t cq_stride;                 // [rows, q_rank padded to cq_stride]
-    void* cache;                                 // [lanes, capacity, lat + pe]
-    void* q;                                     // [rows, H, dimp]: dim unrotated, rot rotated dimensions, zeros
-    const void* uk;                              // [H, dim, lat]
-    void* qa;                                    // [rows, H, lat + pe]
-    const void* o_lat;                           // [rows, H, kv_rank]
-    const void* uv;                              // [H, vdim, lat]
-    void* out; int64_t out_stride;               // [rows, H vdim]
-    int rows, H, dim, rot_dim, dimp, vdim, q_rank, kv_rank, lat, pe, lanes, capacity;
-    float eps;
-    uint32_t* status;
-};
-
-__device__ __forceinline__ int latent_pos(const LatentArgs& a, int row, bool& ok) {
-    const int pos = a.row_pos[row];
-    ok = pos >= 0 && pos < a.capacity;
-    if (!ok && threadIdx.x == 0) raise_status(a.status, GLMB_STATUS_BAD_INDEX);
-    return min(max(pos, 0), a.capacity - 1);
-}
 
 #define LR_THREADS 128
 __device__ __forceinline__ float lr_block_sum(float v, float* scratch) {
@@ -108,40 +82,56 @@ __global__ void __launch_bounds__(256) latent_query_kernel(LatentArgs a) {
     from_f32(v * cs.x + u * cs.y, q[1]);
 }
 
-// grid (pieces of 8 * LA_THREADS latent columns, H, blocks of R rows): a thread owns one column.
-#define LA_THREADS 64
+// grid (pieces of 256 latent columns, H, blocks of LA_ROWS rows): a lane owns eight columns, the warps share the unrotated dimensions.
+#define LA_WARPS 8
+#define LA_THREADS (LA_WARPS * 32)
 #define LA_ROWS 8
-template <typename T>
+template <typename T, int R>
 __global__ void __launch_bounds__(LA_THREADS) latent_absorb_kernel(LatentArgs a) {
-    GLMB_PDL_PROLOGUE();
-    extern __shared__ float q_f[];  // [LA_ROWS][dim]
-    const int h = blockIdx.y, r0 = blockIdx.z * LA_ROWS, rows = min(LA_ROWS, a.rows - r0), W = a.lat + a.pe;
+    asm volatile("griddepcontrol.launch_dependents;");
+    const int h = blockIdx.y, r0 = blockIdx.z * LA_ROWS, rows = min(R, a.rows - r0), W = a.lat + a.pe;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, c = (blockIdx.x * 32 + lane) * 8;
+    const T* w = reinterpret_cast<const T*>(a.uk) + (int64_t)h * a.dim * a.lat + c;
+    float w0[8];  // the weights do not depend on the kernel before: the first ones are asked for while it finishes
+    if (c < a.lat && warp < a.dim) load8(w + (int64_t)warp * a.lat, w0);
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    extern __shared__ __align__(16) float la_smem[];
+    float* part = la_smem;                       // [LA_WARPS][R][256]
+    float* q_f = la_smem + LA_WARPS * R * 256;   // [R][dim]
     const T* q = reinterpret_cast<const T*>(a.q) + ((int64_t)r0 * a.H + h) * a.dimp;
     T* qa = reinterpret_cast<T*>(a.qa) + ((int64_t)r0 * a.H + h) * W;
-    for (int i = threadIdx.x; i < LA_ROWS * a.dim; i += LA_THREADS) {
-        const int r = i / a.dim;
-        q_f[i] = r < rows ? to_f32(q[(int64_t)r * a.H * a.dimp + i % a.dim]) : 0.f;
-    }
+    for (int i = threadIdx.x; i < R * a.dim; i += LA_THREADS) q_f[i] = i / a.dim < rows ? to_f32(q[(int64_t)(i / a.dim) * a.H * a.dimp + i % a.dim]) : 0.f;
     __syncthreads();
-    const int c = (blockIdx.x * LA_THREADS + threadIdx.x) * 2;
-    if (c < a.lat) {
-        const T* w = reinterpret_cast<const T*>(a.uk) + (int64_t)h * a.dim * a.lat + c;
-        float acc[LA_ROWS][2] = {};
-#pragma unroll 8
-        for (int d = 0; d < a.dim; ++d) {
-            const float x = to_f32(w[(int64_t)d * a.lat]), y = to_f32(w[(int64_t)d * a.lat + 1]);
+    float acc[R][8];
 #pragma unroll
-            for (int r = 0; r < LA_ROWS; ++r) {
-                acc[r][0] = fmaf(q_f[r * a.dim + d], x, acc[r][0]);
-                acc[r][1] = fmaf(q_f[r * a.dim + d], y, acc[r][1]);
+    for (int r = 0; r < R; ++r)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[r][e] = 0.f;
+    if (c < a.lat)
+#pragma unroll 4
+        for (int d = warp; d < a.dim; d += LA_WARPS) {
+            float x[8];
+            if (d == warp) {
+#pragma unroll
+                for (int e = 0; e < 8; ++e) x[e] = w0[e];
+            } else {
+                load8(w + (int64_t)d * a.lat, x);
             }
+#pragma unroll
+            for (int r = 0; r < R; ++r)
+#pragma unroll
+                for (int e = 0; e < 8; ++e) acc[r][e] = fmaf(q_f[r * a.dim + d], x[e], acc[r][e]);
         }
 #pragma unroll
-        for (int r = 0; r < LA_ROWS; ++r)
-            if (r < rows) {
-                from_f32(acc[r][0], qa[(int64_t)r * a.H * W + c]);
-                from_f32(acc[r][1], qa[(int64_t)r * a.H * W + c + 1]);
-            }
+    for (int r = 0; r < R; ++r) store8(part + ((warp * R + r) * 32 + lane) * 8, acc[r]);
+    __syncthreads();
+    for (int i = threadIdx.x; i < R * 256; i += LA_THREADS) {
+        const int r = i / 256, col = blockIdx.x * 256 + i % 256;
+        if (r >= rows || col >= a.lat) continue;
+        float y = 0.f;
+#pragma unroll
+        for (int p = 0; p < LA_WARPS; ++p) y += part[p * R * 256 + i];
+        from_f32(y, qa[(int64_t)r * a.H * W + col]);
     }
     if (blockIdx.x) return;
     const int half = a.rot_dim / 2;
@@ -193,10 +183,6 @@ __global__ void __launch_bounds__(LV_WARPS * 32) latent_value_kernel(LatentArgs 
 }
 
 // ===================================================================================================
-static bool latent_ok(const LatentArgs& a) {
-    return a.rows >= 1 && a.rows <= 65535 && a.H >= 1 && a.H <= 65535 && a.dim >= 1 && a.rot_dim >= 2 && !(a.rot_dim & 1) && a.dimp >= a.dim + a.rot_dim && a.vdim >= 1 && a.q_rank >= 1 &&
-           a.kv_rank >= 1 && a.lat >= a.kv_rank && a.pe >= a.rot_dim && !(a.lat & 1) && !(a.pe & 1) && a.lanes >= 1 && a.capacity >= 1 && a.row_pos && a.row_lane;
-}
 #define LATENT_LAUNCH(kernel, grid, threads, smem)                                                         \
     do {                                                                                                   \
         if (is_f32) GLMB_LAUNCH(kernel<float>, grid, threads, smem, (cudaStream_t)stream, a);              \
@@ -216,10 +202,26 @@ GLMB_API int glmb_latent_query(const LatentArgs* args, int is_f32, void* stream)
     if (!latent_ok(a)) return 1;
     LATENT_LAUNCH(latent_query_kernel, dim3(ceil_div(a.H * (a.rot_dim / 2), 256), a.rows), 256, 0);
 }
+template <typename T, int R>
+static int launch_absorb(const LatentArgs& a, cudaStream_t st) {
+    const size_t smem = (size_t)(R * a.dim + LA_WARPS * R * 256) * sizeof(float);
+    static DeviceOnce once;
+    const int dev = once.pending();
+    if (dev != DeviceOnce::SET) {
+        const cudaError_t e = cudaFuncSetAttribute(latent_absorb_kernel<T, R>, cudaFuncAttributeMaxDynamicSharedMemorySize, (R * 1024 + LA_WARPS * R * 256) * 4);
+        if (e != cudaSuccess) return (int)e;
+        once.mark(dev);
+    }
+    GLMB_LAUNCH((latent_absorb_kernel<T, R>), dim3(ceil_div(a.lat, 256), a.H, ceil_div(a.rows, LA_ROWS)), LA_THREADS, smem, st, a);
+    return (int)cudaGetLastError();
+}
 GLMB_API int glmb_latent_absorb(const LatentArgs* args, int is_f32, void* stream) {
     const LatentArgs a = *args;
-    if (!latent_ok(a) || a.dim > 1024) return 1;
-    LATENT_LAUNCH(latent_absorb_kernel, dim3(ceil_div(a.lat, 2 * LA_THREADS), a.H, ceil_div(a.rows, LA_ROWS)), LA_THREADS, LA_ROWS * a.dim * sizeof(float));
+    if (!latent_ok(a) || a.dim > 1024 || (a.lat & 15) || (a.pe & 15)) return 1;
+    cudaStream_t st = (cudaStream_t)stream;
+    if (is_f32) return launch_absorb<float, 8>(a, st);
+    if (a.rows == 1) return launch_absorb<bf16, 1>(a, st);
+    return a.rows <= 4 ? launch_absorb<bf16, 4>(a, st) : launch_absorb<bf16, 8>(a, st);
 }
 GLMB_API int glmb_latent_value(const LatentArgs* args, int is_f32, void* stream) {
     const LatentArgs a = *args;

@@ -31,6 +31,7 @@ from glm_tpu_b200.parallel.peer import PeerGroup
 from glm_tpu_b200.runner.lane_state import RING, LaneRegisters
 
 EXPAND_BYTES = 1 << 30  # keys and values of as many heads at a time as fit here
+RECORD_BYTES = 64 << 20  # what the chunked recurrence keeps between its two kernels stays in the L2
 ABSORB_ROWS = native.MAX_ROWS  # steps of up to this many rows attend over the cache rows as they are
 MAX_EXPERTS, MAX_TOP = 256, 32  # limits of the route sort and the router kernel
 
@@ -51,6 +52,14 @@ class HybridState(LaneRegisters):
         return cls(**cls.registers(cache.lanes, device), latent=[make(cache.latent_shape(i), dtype) if cache.is_latent(i) else None for i in layers],
                    state=[None if cache.is_latent(i) else make(cache.state_shape(i), torch.float32) for i in layers],
                    conv=[None if cache.is_latent(i) else make(cache.conv_shape(i), dtype) for i in layers])
+
+
+def delta_record_bytes(m: DeltaSpec) -> int:
+    """Bytes per 16 tokens and head that the chunked recurrence keeps between its two kernels (0: other sizes, token by token)."""
+    dimp, blocks = pad_to(m.dim, 32), pad16(m.vdim) // 16
+    if m.dim > 128 or m.dim % 8 or m.vdim % 8 or m.conv > 4:
+        return 0
+    return 6 * 16 * (dimp + 8) * 2 + 4 * 16 * 24 * 2 + dimp * 4 + blocks * 16 * 20 * 4
 
 
 def expand_heads(m: LatentSpec, capacity: int, element_bytes: int) -> int:
@@ -81,6 +90,9 @@ def workspace_elements(g, cache: HybridCacheConfig, rows: int, *, prefill: bool,
             for name in ("dv", "do"):
                 need(f, name, rows * m.v_width)
             need(f, "beta", rows * m.heads)
+            if prefill and not is_f32 and delta_record_bytes(m):
+                chunks = min(-(-rows // 16), max(1, RECORD_BYTES // (m.heads * delta_record_bytes(m))))
+                need(f, "records", chunks * m.heads * delta_record_bytes(m) // 4)
         else:
             lat, pe = cache.latent_columns(i)
             need(t, "proj", rows * (pad8(m.q_rank) + pad8(m.kv_rank + m.rot_dim) + pad8(m.heads)))
@@ -89,6 +101,8 @@ def workspace_elements(g, cache: HybridCacheConfig, rows: int, *, prefill: bool,
             few = min(rows, ABSORB_ROWS) if prefill else rows
             need(t, "qa", few * m.heads * (lat + pe))
             need(t, "o_lat", few * m.heads * m.kv_rank)
+            need(f, "part_o", max(few, 16) * m.heads * lat)
+            need(f, "part_ml", max(few, 16) * m.heads * 2)
             if prefill and rows > ABSORB_ROWS:
                 heads = expand_heads(m, cache.context_capacity, cache.element_bytes)
                 need(t, "keys", cache.context_capacity * heads * pad16(m.dim + m.rot_dim))
@@ -206,8 +220,11 @@ class ZikevikModel:
         a.gate, a.gate_stride, a.norm = gate.data_ptr(), gate.stride(0), t.norm.data_ptr()
         a.out, a.out_stride = out.data_ptr(), out.stride(0)
         a.H, a.G, a.dim, a.dimp, a.vdim, a.decode, a.eps = m.heads, m.kv_heads, m.dim, pad_to(m.dim, 32), m.vdim, int(decode), self.g.norm_eps
-        native.delta_prep(a, self.is_f32)
-        native.delta_scan(a)
+        if not decode and "records" in ws.flat and delta_record_bytes(m) and not self.plain_kernels:
+            native.delta_chunk(a, ws.flat["records"])
+        else:
+            native.delta_prep(a, self.is_f32)
+            native.delta_scan(a)
         native.delta_out(a, self.is_f32)
         return out
 
@@ -236,6 +253,10 @@ class ZikevikModel:
             # one key head: the cache row is the key, its first columns are the value
             a.qa, a.o_lat = ws.flat["qa"].data_ptr(), ws.flat["o_lat"].data_ptr()
             native.latent_absorb(a, self.is_f32)
+            if not (self.is_f32 or self.plain_kernels) and native.latent_decode_takes(lat, pe):
+                a.sink, a.scale, a.part_o, a.part_ml = t.sink.data_ptr(), m.scale, ws.flat["part_o"].data_ptr(), ws.flat["part_ml"].data_ptr()
+                native.latent_decode(a)
+                return out
             b.q, b.k, b.v, b.out, b.out_stride = a.qa, a.cache, a.cache, a.o_lat, m.heads * m.kv_rank
             b.G, b.dim, b.dimp, b.vdim, b.vdimp, b.decode = 1, lat + pe, lat + pe, m.kv_rank, lat + pe, 1
             native.chunk_attention(b, self.is_f32, plain=self.plain_kernels)

@@ -105,9 +105,10 @@ class LatentArgs(C.Structure):
         ("cq", C.c_void_p), ("cq_stride", C.c_int64),
         ("cache", C.c_void_p), ("q", C.c_void_p), ("uk", C.c_void_p), ("qa", C.c_void_p), ("o_lat", C.c_void_p), ("uv", C.c_void_p),
         ("out", C.c_void_p), ("out_stride", C.c_int64),
+        ("sink", C.c_void_p), ("part_o", C.c_void_p), ("part_ml", C.c_void_p), ("parts", C.c_int),
         ("rows", C.c_int), ("H", C.c_int), ("dim", C.c_int), ("rot_dim", C.c_int), ("dimp", C.c_int), ("vdim", C.c_int), ("q_rank", C.c_int),
         ("kv_rank", C.c_int), ("lat", C.c_int), ("pe", C.c_int), ("lanes", C.c_int), ("capacity", C.c_int),
-        ("eps", C.c_float),
+        ("eps", C.c_float), ("scale", C.c_float),
         ("status", C.c_void_p),
     ]
 
@@ -561,6 +562,15 @@ def latent_value(args: LatentArgs, is_f32: bool) -> None:
     _check(lib().glmb_latent_value(C.byref(args), int(is_f32), _stream()), "latent_value")
 
 
+def latent_decode_takes(lat: int, pe: int) -> bool:
+    return lat <= 512 and lat + pe <= 640
+
+
+def latent_decode(args: LatentArgs) -> None:
+    """bf16, 1..8 rows: attention over the cache rows, sink, value projection and gate (two launches)."""
+    _check(lib().glmb_latent_decode(C.byref(args), _stream()), "latent_decode")
+
+
 def delta_max_taps() -> int:
     return int(lib().glmb_delta_max_taps())
 
@@ -568,6 +578,16 @@ def delta_max_taps() -> int:
 def delta_prep(args: DeltaArgs, is_f32: bool) -> None:
     """Convolution, activation, unit vectors, decay and write strength of a delta-rule layer; advances the convolution's state."""
     _check(lib().glmb_delta_prep(C.byref(args), int(is_f32), _stream()), "delta_prep")
+
+
+def delta_chunk_record(dim: int, vdim: int, taps: int) -> int:
+    """Bytes of a record of the chunked kernels (16 tokens of one head); 0: the sizes are not for them."""
+    return int(lib().glmb_delta_chunk_record(int(dim), int(vdim), int(taps)))
+
+
+def delta_chunk(args: DeltaArgs, records) -> None:
+    """bf16, consecutive rows of one sequence: projection to read-out in chunks of 16 tokens on the tensor cores; ``records`` is scratch."""
+    _check(lib().glmb_delta_chunk(C.byref(args), _p(records), C.c_int64(records.numel() * records.element_size()), _stream()), "delta_chunk")
 
 
 def delta_scan(args: DeltaArgs) -> None:

@@ -118,6 +118,13 @@ def gated_ff(h: torch.Tensor, weight, prefix: str = "") -> torch.Tensor:
     return (silu(h @ weight(prefix + "gate").T) * (h @ weight(prefix + "up").T)) @ weight(prefix + "down").T
 
 
+def router_margin(h: torch.Tensor, router: dict, weight) -> torch.Tensor:
+    """``[T]``: how far the last expert that is chosen lies above the first that is not (in router logits; infinite if all are chosen)."""
+    best = (h @ weight("router").T).sort(dim=-1, descending=True).values
+    top = router["top"]
+    return best[:, top - 1] - best[:, top] if top < router["experts"] else torch.full((h.shape[0],), float("inf"), dtype=h.dtype)
+
+
 def routed_experts(h: torch.Tensor, router: dict, weight) -> torch.Tensor:
     """Sigmoid scores; the best ``top`` experts each take the token scaled by its own score, and their outputs are added."""
     scores = torch.sigmoid(h @ weight("router").T)
@@ -134,8 +141,9 @@ def routed_experts(h: torch.Tensor, router: dict, weight) -> torch.Tensor:
 MIXERS = {"channel_delta": channel_delta, "latent_attention": latent_attention}
 
 
-def forward(config: dict, tensors: dict, tokens, *, dtype=torch.float64, layers_out: list | None = None) -> torch.Tensor:
-    """Logits ``[T, vocab]`` of a sequence; ``layers_out`` collects the residual after every layer."""
+def forward(config: dict, tensors: dict, tokens, *, dtype=torch.float64, layers_out: list | None = None, margins_out: list | None = None) -> torch.Tensor:
+    """Logits ``[T, vocab]`` of a sequence; ``layers_out`` collects the residual after every layer, ``margins_out`` the ``router_margin`` of every
+    routed layer."""
     get = lambda name: tensors[name].to(dtype)  # noqa: E731
     eps = config["norm"]["eps"]
     x = get("embed")[torch.as_tensor(list(tokens), dtype=torch.long)] * config["embedding"]["scale"]
@@ -147,6 +155,8 @@ def forward(config: dict, tensors: dict, tokens, *, dtype=torch.float64, layers_
         mlp = layer.get("mlp")
         if mlp is not None:
             h, weight = zero_centred_norm(x, get(f"l{j}.norm2"), eps), lambda n, j=j: get(f"l{j}.mlp.{n}")
+            if margins_out is not None and mlp["kind"] != "dense":
+                margins_out.append(router_margin(h, mlp["router"], weight))
             x = x + (gated_ff(h, weight) if mlp["kind"] == "dense" else routed_experts(h, mlp["router"], weight))
         if layers_out is not None:
             layers_out.append(x.clone())
