@@ -11,12 +11,14 @@
 //
 //   delta_chunk_prep   a CTA per (chunk, head): convolution, activation, unit vectors, decays, A, B and L in fp32; leaves one record with what
 //                      the scan multiplies, matrices as two bf16 pieces (value and remainder: 16 bits of mantissa)
-//   delta_chunk_scan   a warp keeps the fp32 state of 16 value channels in its accumulators ([value channel, key channel]: the accumulator
+//   delta_chunk_scan   two warps keep the fp32 state of 16 value channels in their accumulators ([value channel, key channel]: the accumulator
 //                      layout is the operand layout of the next product) and walks the chunks; records arrive by bulk copies, several chunks
 //                      ahead.  Products are hi.hi + hi.lo + lo.hi with fp32 sums.
 //
 // A record: [6][16][dimp + 8] bf16 (e^G k, e^G q, e^(G_last - G) k, each hi and lo), [4][16][24] bf16 (L hi, lo, B hi, lo), [dimp] fp32
 // (e^G_last), [vdim / 16][16][20] fp32 (V by blocks of 16 channels).  Row paddings stagger the banks for ldmatrix.
+#include <mutex>
+
 #include "attention_core.cuh"
 #include "delta_rule.cuh"
 #include "tcgen05.cuh"
@@ -27,6 +29,7 @@
 #define DC_TAPS 4
 #define DC_LB 24      // row of L and B
 #define DC_VB 20      // row of a value block
+#define DC_OVERLAP_CHUNKS 16  // longer steps prepare one segment while the one before is scanned
 #define DC_LOG2E 1.4426950408889634f
 
 struct DeltaChunkArgs {
@@ -34,7 +37,7 @@ struct DeltaChunkArgs {
     unsigned char* records;  // [chunks of the segment, H] records
     int row0, count;         // the segment: rows row0 .. row0 + count - 1 of the step (row0 a multiple of 16)
     int last;                // the segment ends the step
-    int warps;               // scan: blocks of 16 value channels per CTA
+    int blocks;              // scan: blocks of 16 value channels per CTA
 };
 
 __host__ __device__ static inline int dc_mats_bytes(int dimp) { return 6 * DC_TOKENS * (dimp + 8) * 2; }
@@ -63,8 +66,33 @@ __device__ __forceinline__ void dc_fold(float (&v)[32], int lane, int offset) {
     }
 }
 
+__device__ __forceinline__ float dc_silu(float z) { return __fdividef(z, 1.f + dc_exp2(-DC_LOG2E * z)); }
+
+// Token t's rows of the three operands that meet the state, by one warp.  scale_k, scale_q: what makes the token's key and query unit vectors.
+__device__ __forceinline__ void dc_operands(const float* q_s, const float* k_s, const float* g_s, int RS, int DP, int t, float scale_k, float scale_q,
+                                            uint32_t* mats, int lane) {
+    const int words = (DP + 8) / 2;
+    for (int d = lane * 2; d < DP; d += 64) {
+        const float2 g = *reinterpret_cast<const float2*>(g_s + t * RS + d), end = *reinterpret_cast<const float2*>(g_s + (DC_TOKENS - 1) * RS + d);
+        float2 k = *reinterpret_cast<const float2*>(k_s + t * RS + d), q = *reinterpret_cast<const float2*>(q_s + t * RS + d);
+        k.x *= scale_k; k.y *= scale_k; q.x *= scale_q; q.y *= scale_q;
+        const float e0 = dc_exp2(g.x), e1 = dc_exp2(g.y), f0 = dc_exp2(end.x - g.x), f1 = dc_exp2(end.y - g.y);
+        uint32_t* at = mats + t * words + d / 2;
+        uint32_t hi, lo;
+        dc_split(k.x * e0, k.y * e1, hi, lo);
+        at[0] = hi;
+        at[DC_TOKENS * words] = lo;
+        dc_split(q.x * e0, q.y * e1, hi, lo);
+        at[2 * DC_TOKENS * words] = hi;
+        at[3 * DC_TOKENS * words] = lo;
+        dc_split(k.x * f0, k.y * f1, hi, lo);
+        at[4 * DC_TOKENS * words] = hi;
+        at[5 * DC_TOKENS * words] = lo;
+    }
+}
+
 // grid (chunks, H)
-__global__ void __launch_bounds__(DC_THREADS) delta_chunk_prep_kernel(DeltaChunkArgs p) {
+__global__ void __launch_bounds__(DC_THREADS, 3) delta_chunk_prep_kernel(DeltaChunkArgs p) {
     GLMB_PDL_PROLOGUE();
     const DeltaArgs& a = p.d;
     extern __shared__ __align__(16) float smem_f[];
@@ -72,7 +100,7 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_prep_kernel(DeltaChunk
     float* q_s = smem_f;                        // [16][RS]
     float* k_s = q_s + DC_TOKENS * RS;
     float* g_s = k_s + DC_TOKENS * RS;          // log2 of the decays, then their running sum
-    __shared__ float A_s[DC_TOKENS][DC_TOKENS + 1], B_s[DC_TOKENS][DC_TOKENS + 1], beta_s[DC_TOKENS];
+    __shared__ float A_s[DC_TOKENS][DC_TOKENS + 1], B_s[DC_TOKENS][DC_TOKENS + 1], beta_s[DC_TOKENS], scale_s[2 * DC_TOKENS];
     const int h = blockIdx.y, kvh = h / (a.H / a.G), t0 = p.row0 + blockIdx.x * DC_TOKENS, n = min(DC_TOKENS, p.row0 + p.count - t0);
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int C = 2 * a.G * a.dim + a.H * a.vdim, keep = a.taps - 1;
@@ -82,17 +110,10 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_prep_kernel(DeltaChunk
     const int start = a.row_pos[0], seq = delta_lane(a, 0);
     const bf16* state = reinterpret_cast<const bf16*>(a.conv_state) + (int64_t)seq * a.taps * C;
 
-    // ---- decays ------------------------------------------------------------------------------------------
-    const float rate = a.a_rate[h] * DC_LOG2E;
-    for (int i = tid; i < DC_TOKENS * DP; i += DC_THREADS) {
-        const int t = i / DP, d = i % DP;
-        g_s[t * RS + d] = t < n && d < a.dim ? -rate * delta_softplus(a.a[(int64_t)(t0 + t) * a.a_stride + h * a.dim + d] + a.dt_bias[h * a.dim + d]) : 0.f;
-    }
-    if (tid < DC_TOKENS) beta_s[tid] = tid < n ? sigmoidf_precise(__bfloat162float(proj[(int64_t)(t0 + tid) * a.proj_stride + a.off_b + h])) : 0.f;
     // ---- convolution: a thread takes eight channels of four tokens -----------------------------------------
     const int kvec = a.dim / 8, vecs = 2 * kvec + a.vdim / 8;
     for (int i = tid; i < vecs * 4; i += DC_THREADS) {
-        const int vec = i % vecs, first = i / vecs * 4;
+        const int strip = i / vecs, vec = i - strip * vecs, first = strip * 4;
         const int kind = vec < kvec ? 0 : vec < 2 * kvec ? 1 : 2, c = (kind == 0 ? vec : kind == 1 ? vec - kvec : vec - 2 * kvec) * 8;
         const int chan = (kind == 0 ? kvh * a.dim : kind == 1 ? (a.G + kvh) * a.dim : 2 * a.G * a.dim + h * a.vdim) + c;
         uint4 u[4 + DC_TAPS - 1];
@@ -127,25 +148,43 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_prep_kernel(DeltaChunk
 #pragma unroll
         for (int t = 0; t < 4; ++t) {
 #pragma unroll
-            for (int e = 0; e < 8; ++e) y[t][e] = first + t < n ? delta_silu(y[t][e]) : 0.f;
+            for (int e = 0; e < 8; ++e) y[t][e] = first + t < n ? dc_silu(y[t][e]) : 0.f;
             if (kind == 2) store8(v_out + ((int64_t)(c / 16) * DC_TOKENS + first + t) * DC_VB + c % 16, y[t]);
             else store8((kind == 0 ? q_s : k_s) + (first + t) * RS + c, y[t]);
         }
     }
-    for (int i = tid; i < 2 * DC_TOKENS * (DP - a.dim); i += DC_THREADS) {  // padding of the key channels
-        const int r = i / (DP - a.dim), d = a.dim + i % (DP - a.dim);
-        (r < DC_TOKENS ? q_s : k_s)[(r % DC_TOKENS) * RS + d] = 0.f;
-    }
+    if (a.dim < DP)  // padding of the key channels
+        for (int r = warp; r < 2 * DC_TOKENS; r += DC_THREADS / 32)
+            for (int d = a.dim + lane; d < DP; d += 32) (r < DC_TOKENS ? q_s : k_s)[(r % DC_TOKENS) * RS + d] = 0.f;
     if (a.vdim % 16)  // the last value block's second half
         for (int i = tid; i < DC_TOKENS * 8; i += DC_THREADS) v_out[((int64_t)(a.vdim / 16) * DC_TOKENS + i / 8) * DC_VB + 8 + i % 8] = 0.f;
+    // ---- decays ------------------------------------------------------------------------------------------
+    const float rate = a.a_rate[h] * DC_LOG2E;
+    for (int d = lane; d < DP; d += 32) {
+        const float bias = d < a.dim ? a.dt_bias[h * a.dim + d] : 0.f;
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+            const int t = warp + x * (DC_THREADS / 32);
+            g_s[t * RS + d] = t < n && d < a.dim ? -rate * delta_softplus(a.a[(int64_t)(t0 + t) * a.a_stride + h * a.dim + d] + bias) : 0.f;
+        }
+    }
+    if (tid < DC_TOKENS) beta_s[tid] = tid < n ? sigmoidf_precise(__bfloat162float(proj[(int64_t)(t0 + tid) * a.proj_stride + a.off_b + h])) : 0.f;
     __syncthreads();
-    // ---- unit vectors (a warp per row), running sums of the decays ------------------------------------------
-    for (int r = warp; r < 2 * DC_TOKENS; r += DC_THREADS / 32) {
-        float* x = (r < DC_TOKENS ? q_s : k_s) + (r % DC_TOKENS) * RS;
-        float ss = 0.f;
-        for (int d = lane; d < DP; d += 32) ss = fmaf(x[d], x[d], ss);
-        const float scale = (r < DC_TOKENS ? 1.f / sqrtf((float)a.dim) : 1.f) / sqrtf(warp_sum(ss) + 1e-6f);
-        for (int d = lane; d < DP; d += 32) x[d] *= scale;
+    // ---- what makes unit vectors (a warp per row), running sums of the decays --------------------------------
+    {
+        const float* rows = (warp < 4 ? q_s : k_s) + (warp & 3) * 4 * RS;  // four rows per warp, queries first
+        float ss[4] = {0.f, 0.f, 0.f, 0.f};
+        for (int d = lane; d < DP; d += 32)
+#pragma unroll
+            for (int x = 0; x < 4; ++x) ss[x] = fmaf(rows[x * RS + d], rows[x * RS + d], ss[x]);
+        // the four sums at once: after two steps a quarter of the warp is left with each
+        const bool up = lane & 16, right = lane & 8;
+        const float s0 = (up ? ss[2] : ss[0]) + __shfl_xor_sync(0xffffffffu, up ? ss[0] : ss[2], 16);
+        const float s1 = (up ? ss[3] : ss[1]) + __shfl_xor_sync(0xffffffffu, up ? ss[1] : ss[3], 16);
+        float sum = (right ? s1 : s0) + __shfl_xor_sync(0xffffffffu, right ? s0 : s1, 8);
+#pragma unroll
+        for (int o = 4; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+        if (!(lane & 7)) scale_s[warp * 4 + lane / 8] = rsqrtf(sum + 1e-6f) * (warp < 4 ? rsqrtf((float)a.dim) : 1.f);
     }
     for (int d = tid; d < DP; d += DC_THREADS) {
         float sum = 0.f;
@@ -153,46 +192,50 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_prep_kernel(DeltaChunk
         for (int t = 0; t < DC_TOKENS; ++t) { sum += g_s[t * RS + d]; g_s[t * RS + d] = sum; }
     }
     __syncthreads();
-    // ---- A and B: 4 x 4 blocks of (i, j) below the diagonal, sixteen lanes share the channels of a block ------
-    for (int unit = warp; unit < 5; unit += DC_THREADS / 32) {
-        const int block = unit * 2 + (lane >> 4), sub = lane & 15;
+    uint32_t* mats = reinterpret_cast<uint32_t*>(record);
+    auto operands = [&](int t) { dc_operands(q_s, k_s, g_s, RS, DP, t, scale_s[DC_TOKENS + t], scale_s[t], mats, lane); };
+    if (warp >= 5) {  // the warps that have no pairs take the operands
+        for (int t = warp - 5; t < DC_TOKENS; t += 3) operands(t);
+    } else {
+        // ---- A and B: 4 x 4 blocks of (i, j) below the diagonal, sixteen lanes share the channels of a block ------
+        const int block = warp * 2 + (lane >> 4), sub = lane & 15;
         const int bi = block < 1 ? 0 : block < 3 ? 1 : block < 6 ? 2 : 3, bj = block - bi * (bi + 1) / 2;
         float acc[32];  // A then B of the 16 pairs
 #pragma unroll
         for (int x = 0; x < 32; ++x) acc[x] = 0.f;
-        for (int d = sub * 2; d < DP; d += 32) {
-            float2 gi[4], ki[4], qi[4], gj[4], kj[4];
+        for (int d = sub; d < DP; d += 16) {
+            float gi[4], ki[4], qi[4], gj[4], kj[4];
 #pragma unroll
             for (int x = 0; x < 4; ++x) {
-                gi[x] = *reinterpret_cast<const float2*>(g_s + (bi * 4 + x) * RS + d);
-                ki[x] = *reinterpret_cast<const float2*>(k_s + (bi * 4 + x) * RS + d);
-                qi[x] = *reinterpret_cast<const float2*>(q_s + (bi * 4 + x) * RS + d);
-                gj[x] = *reinterpret_cast<const float2*>(g_s + (bj * 4 + x) * RS + d);
-                kj[x] = *reinterpret_cast<const float2*>(k_s + (bj * 4 + x) * RS + d);
+                gi[x] = g_s[(bi * 4 + x) * RS + d];
+                ki[x] = k_s[(bi * 4 + x) * RS + d];
+                qi[x] = q_s[(bi * 4 + x) * RS + d];
+                gj[x] = g_s[(bj * 4 + x) * RS + d];
+                kj[x] = k_s[(bj * 4 + x) * RS + d];
             }
             if (bi != bj) {  // exp(G_i - G_j) in two factors around the end of the earlier block, both at most one
-                const float2 mid = gj[3];
 #pragma unroll
                 for (int x = 0; x < 4; ++x) {
-                    const float e0 = dc_exp2(gi[x].x - mid.x), e1 = dc_exp2(gi[x].y - mid.y), f0 = dc_exp2(mid.x - gj[x].x), f1 = dc_exp2(mid.y - gj[x].y);
-                    ki[x].x *= e0; ki[x].y *= e1; qi[x].x *= e0; qi[x].y *= e1;
-                    kj[x].x *= f0; kj[x].y *= f1;
+                    const float e = dc_exp2(gi[x] - gj[3]);
+                    ki[x] *= e;
+                    qi[x] *= e;
+                    kj[x] *= dc_exp2(gj[3] - gj[x]);
                 }
 #pragma unroll
                 for (int x = 0; x < 4; ++x)
 #pragma unroll
                     for (int y = 0; y < 4; ++y) {
-                        acc[x * 4 + y] = fmaf(ki[x].x, kj[y].x, fmaf(ki[x].y, kj[y].y, acc[x * 4 + y]));
-                        acc[16 + x * 4 + y] = fmaf(qi[x].x, kj[y].x, fmaf(qi[x].y, kj[y].y, acc[16 + x * 4 + y]));
+                        acc[x * 4 + y] = fmaf(ki[x], kj[y], acc[x * 4 + y]);
+                        acc[16 + x * 4 + y] = fmaf(qi[x], kj[y], acc[16 + x * 4 + y]);
                     }
             } else {
 #pragma unroll
                 for (int x = 0; x < 4; ++x)
 #pragma unroll
                     for (int y = 0; y <= x; ++y) {
-                        const float e0 = x == y ? kj[y].x : kj[y].x * dc_exp2(gi[x].x - gj[y].x), e1 = x == y ? kj[y].y : kj[y].y * dc_exp2(gi[x].y - gj[y].y);
-                        acc[x * 4 + y] = fmaf(ki[x].x, e0, fmaf(ki[x].y, e1, acc[x * 4 + y]));
-                        acc[16 + x * 4 + y] = fmaf(qi[x].x, e0, fmaf(qi[x].y, e1, acc[16 + x * 4 + y]));
+                        const float e = x == y ? kj[y] : kj[y] * dc_exp2(gi[x] - gj[y]);
+                        acc[x * 4 + y] = fmaf(ki[x], e, acc[x * 4 + y]);
+                        acc[16 + x * 4 + y] = fmaf(qi[x], e, acc[16 + x * 4 + y]);
                     }
             }
         }
@@ -204,7 +247,8 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_prep_kernel(DeltaChunk
 #pragma unroll
         for (int x = 0; x < 2; ++x) {
             const int at = sub * 2 + x, i = bi * 4 + (at & 15) / 4, j = bj * 4 + (at & 3);
-            (at < 16 ? A_s : B_s)[i][j] = j < i || (at >= 16 && j == i) ? acc[x] : 0.f;
+            if (at < 16) A_s[i][j] = j < i ? acc[x] * scale_s[DC_TOKENS + i] * scale_s[DC_TOKENS + j] : 0.f;
+            else B_s[i][j] = j <= i ? acc[x] * scale_s[i] * scale_s[DC_TOKENS + j] : 0.f;
         }
     }
     for (int i = tid; i < DC_TOKENS * DC_TOKENS; i += DC_THREADS)  // blocks above the diagonal
@@ -230,43 +274,35 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_prep_kernel(DeltaChunk
             lb[(2 * DC_TOKENS + i / DC_TOKENS) * DC_LB + i % DC_TOKENS] = hi;
             lb[(3 * DC_TOKENS + i / DC_TOKENS) * DC_LB + i % DC_TOKENS] = __float2bfloat16_rn(x - __bfloat162float(hi));
         }
+    } else if (warp == 2) {
+        float* gamma = reinterpret_cast<float*>(record + dc_mats_bytes(DP) + 4 * DC_TOKENS * DC_LB * 2);
+        for (int d = lane; d < DP; d += 32) gamma[d] = dc_exp2(g_s[(DC_TOKENS - 1) * RS + d]);
     }
-    // ---- the operands that meet the state --------------------------------------------------------------------
-    uint32_t* mats = reinterpret_cast<uint32_t*>(record);
-    const int words = (DP + 8) / 2;
-    for (int i = tid; i < DC_TOKENS * DP / 2; i += DC_THREADS) {
-        const int t = i / (DP / 2), d = i % (DP / 2) * 2;
-        const float2 g = *reinterpret_cast<const float2*>(g_s + t * RS + d), end = *reinterpret_cast<const float2*>(g_s + (DC_TOKENS - 1) * RS + d);
-        const float2 k = *reinterpret_cast<const float2*>(k_s + t * RS + d), q = *reinterpret_cast<const float2*>(q_s + t * RS + d);
-        const float e0 = dc_exp2(g.x), e1 = dc_exp2(g.y), f0 = dc_exp2(end.x - g.x), f1 = dc_exp2(end.y - g.y);
-        const float2 x[3] = {{k.x * e0, k.y * e1}, {q.x * e0, q.y * e1}, {k.x * f0, k.y * f1}};
-#pragma unroll
-        for (int m = 0; m < 3; ++m) dc_split(x[m].x, x[m].y, mats[((2 * m) * DC_TOKENS + t) * words + d / 2], mats[((2 * m + 1) * DC_TOKENS + t) * words + d / 2]);
-    }
-    float* gamma = reinterpret_cast<float*>(record + dc_mats_bytes(DP) + 4 * DC_TOKENS * DC_LB * 2);
-    for (int d = tid; d < DP; d += DC_THREADS) gamma[d] = dc_exp2(g_s[(DC_TOKENS - 1) * RS + d]);
 }
 
 // ---------------------------------------------------------------------------------------------------
-#define DC_STAGES 4
+#define DC_STAGES 3
 
 __device__ __forceinline__ void dc_bulk_load(void* smem_dst, const void* src, uint32_t bytes, uint64_t* bar) {
     asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
                  ::"r"(smem_u32(smem_dst)), "l"(src), "r"(bytes), "r"(smem_u32(bar)) : "memory");
 }
 
-// grid (groups of `warps` blocks of 16 value channels, H), 32 * warps threads.  KS: key channels / 16.
+// grid (groups of `blocks` blocks of 16 value channels, H), 64 * blocks threads: two warps share a block, each with half of the key channels
+// (the tensor pipe of one scheduler is what a single warp would wait for).  KS: key channels / 32, the 16-channel steps of a warp.
 template <int KS>
-__global__ void __launch_bounds__(128) delta_chunk_scan_kernel(DeltaChunkArgs p) {
-    constexpr int DP = KS * 16, RS = DP + 8;
+__global__ void __launch_bounds__(256) delta_chunk_scan_kernel(DeltaChunkArgs p) {
+    constexpr int DP = KS * 32, RS = DP + 8;
     const DeltaArgs& a = p.d;
     extern __shared__ __align__(128) unsigned char smem_raw[];
     __shared__ __align__(8) uint64_t full_bar[DC_STAGES];
+    __shared__ float4 swap_s[4][2][3][32];  // [block][half]: what a warp's half of the key channels adds to the products
     const int h = blockIdx.y, kvh = h / (a.H / a.G), chunks = (p.count + DC_TOKENS - 1) / DC_TOKENS;
-    const int blocks = (a.vdim + 15) / 16, block0 = blockIdx.x * p.warps, here = min(p.warps, blocks - block0);
-    const int head_bytes = dc_head_bytes(DP), value_bytes = here * dc_value_block(), stage_bytes = head_bytes + p.warps * dc_value_block();
+    const int blocks = (a.vdim + 15) / 16, block0 = blockIdx.x * p.blocks, here = min(p.blocks, blocks - block0);
+    const int head_bytes = dc_head_bytes(DP), value_bytes = here * dc_value_block(), stage_bytes = head_bytes + p.blocks * dc_value_block();
     const int64_t record_bytes = dc_record_bytes(DP, a.vdim);
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3, mr = lane & 7, mi = lane >> 3;
+    const int lane = threadIdx.x & 31, block = threadIdx.x >> 6, half = (threadIdx.x >> 5) & 1;
+    const int g = lane >> 2, t4 = lane & 3, mr = lane & 7, mi = lane >> 3;
     if (threadIdx.x == 0) {
         for (int s = 0; s < DC_STAGES; ++s) mbar_init(full_bar + s, 1);
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
@@ -283,11 +319,11 @@ __global__ void __launch_bounds__(128) delta_chunk_scan_kernel(DeltaChunkArgs p)
     };
     if (threadIdx.x == 0)
         for (int i = 0; i < min(DC_STAGES, chunks); ++i) load(i);
-    const bool mine = warp < here;
-    const int c0 = (block0 + warp) * 16, seq = delta_lane(a, 0), start = a.row_pos[0] + p.row0;
-    float* state = a.state + ((int64_t)seq * a.H + h) * a.vdim * DP;
+    const bool mine = block < here;
+    const int c0 = (block0 + block) * 16, k0 = half * KS * 16, seq = delta_lane(a, 0), start = a.row_pos[0] + p.row0;
+    float* state = a.state + ((int64_t)seq * a.H + h) * a.vdim * DP + k0;
     const bool writes = delta_writes(a, 0);
-    // accumulators of the transposed state: value channels c0 + g, + 8; key channels 8 j + 2 t4, + 1
+    // accumulators of the transposed state: value channels c0 + g, + 8; key channels k0 + 8 j + 2 t4, + 1
     float s[2 * KS][4];
 #pragma unroll
     for (int j = 0; j < 2 * KS; ++j)
@@ -306,17 +342,17 @@ __global__ void __launch_bounds__(128) delta_chunk_scan_kernel(DeltaChunkArgs p)
             ok = false;  // meaningless from here on, but every barrier is still met
         }
         const unsigned char* base = smem_raw + stage * stage_bytes;
-        const bf16* mats = reinterpret_cast<const bf16*>(base);
+        const bf16* mats = reinterpret_cast<const bf16*>(base) + k0;
         const bf16* lb = reinterpret_cast<const bf16*>(base + dc_mats_bytes(DP));
-        const float* gamma = reinterpret_cast<const float*>(base + dc_mats_bytes(DP) + 4 * DC_TOKENS * DC_LB * 2);
-        const float* v_s = reinterpret_cast<const float*>(base + head_bytes + warp * dc_value_block());
+        const float* gamma = reinterpret_cast<const float*>(base + dc_mats_bytes(DP) + 4 * DC_TOKENS * DC_LB * 2) + k0;
+        const float* v_s = reinterpret_cast<const float*>(base + head_bytes + block * dc_value_block());
         if (mine) {
-            // ---- (e^G k) S and (e^G q) S, transposed: value channels x tokens ------------------------------
-            float w[2][4], wl[2][4], r[2][4], rl[2][4];
+            // ---- (e^G k) S and (e^G q) S, transposed: value channels x tokens, over this warp's key channels --------
+            float w[2][4], wl[2][4], wm[2][4], r[2][4], rl[2][4], rm[2][4];
 #pragma unroll
             for (int n = 0; n < 2; ++n)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) w[n][e] = wl[n][e] = r[n][e] = rl[n][e] = 0.f;
+                for (int e = 0; e < 4; ++e) w[n][e] = wl[n][e] = wm[n][e] = r[n][e] = rl[n][e] = rm[n][e] = 0.f;
             const bf16* at = mats + (mr + 8 * (mi >> 1)) * RS + 8 * (mi & 1);
 #pragma unroll
             for (int kk = 0; kk < KS; ++kk) {
@@ -332,38 +368,54 @@ __global__ void __launch_bounds__(128) delta_chunk_scan_kernel(DeltaChunkArgs p)
 #pragma unroll
                 for (int n = 0; n < 2; ++n) {
                     mma_bf16_16816(w[n], hi, kh[2 * n], kh[2 * n + 1]);
-                    mma_bf16_16816(r[n], hi, qh[2 * n], qh[2 * n + 1]);
                     mma_bf16_16816(wl[n], lo, kh[2 * n], kh[2 * n + 1]);
+                    mma_bf16_16816(wm[n], hi, kl[2 * n], kl[2 * n + 1]);
+                }
+#pragma unroll
+                for (int n = 0; n < 2; ++n) {
+                    mma_bf16_16816(r[n], hi, qh[2 * n], qh[2 * n + 1]);
                     mma_bf16_16816(rl[n], lo, qh[2 * n], qh[2 * n + 1]);
-                    mma_bf16_16816(wl[n], hi, kl[2 * n], kl[2 * n + 1]);
-                    mma_bf16_16816(rl[n], hi, ql[2 * n], ql[2 * n + 1]);
+                    mma_bf16_16816(rm[n], hi, ql[2 * n], ql[2 * n + 1]);
                 }
             }
+            // ---- the two halves meet: both warps go on with all of w, each with the read-out of eight tokens ---------
+#pragma unroll
+            for (int n = 0; n < 2; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) { w[n][e] += wl[n][e] + wm[n][e]; r[n][e] += rl[n][e] + rm[n][e]; }
+            const int other = half ^ 1;
+            swap_s[block][half][0][lane] = make_float4(w[0][0], w[0][1], w[0][2], w[0][3]);
+            swap_s[block][half][1][lane] = make_float4(w[1][0], w[1][1], w[1][2], w[1][3]);
+            swap_s[block][half][2][lane] = half ? make_float4(r[0][0], r[0][1], r[0][2], r[0][3]) : make_float4(r[1][0], r[1][1], r[1][2], r[1][3]);
+            asm volatile("bar.sync %0, 64;" ::"r"(block + 1) : "memory");
+            const float4 w0 = swap_s[block][other][0][lane], w1 = swap_s[block][other][1][lane], r0 = swap_s[block][other][2][lane];
+            w[0][0] += w0.x; w[0][1] += w0.y; w[0][2] += w0.z; w[0][3] += w0.w;
+            w[1][0] += w1.x; w[1][1] += w1.y; w[1][2] += w1.z; w[1][3] += w1.w;
+            float out[4] = {(half ? r[1][0] : r[0][0]) + r0.x, (half ? r[1][1] : r[0][1]) + r0.y, (half ? r[1][2] : r[0][2]) + r0.z, (half ? r[1][3] : r[0][3]) + r0.w};
             // ---- U = L (V - ..) -----------------------------------------------------------------------------
             uint32_t xh[4], xl[4];
 #pragma unroll
             for (int n = 0; n < 2; ++n)
 #pragma unroll
-                for (int e = 0; e < 2; ++e) {
-                    const float x0 = v_s[(n * 8 + 2 * t4) * DC_VB + g + 8 * e] - (w[n][2 * e] + wl[n][2 * e]);
-                    const float x1 = v_s[(n * 8 + 2 * t4 + 1) * DC_VB + g + 8 * e] - (w[n][2 * e + 1] + wl[n][2 * e + 1]);
-                    dc_split(x0, x1, xh[2 * n + e], xl[2 * n + e]);
-                }
-            uint32_t lh[4], ll[4], bh[4], bl[4];
-            const bf16* lat = lb + (mr + 8 * (mi >> 1)) * DC_LB + 8 * (mi & 1);
-            ldmatrix_x4(lh, lat);
-            ldmatrix_x4(ll, lat + DC_TOKENS * DC_LB);
-            ldmatrix_x4(bh, lat + 2 * DC_TOKENS * DC_LB);
-            ldmatrix_x4(bl, lat + 3 * DC_TOKENS * DC_LB);
+                for (int e = 0; e < 2; ++e)
+                    dc_split(v_s[(n * 8 + 2 * t4) * DC_VB + g + 8 * e] - w[n][2 * e], v_s[(n * 8 + 2 * t4 + 1) * DC_VB + g + 8 * e] - w[n][2 * e + 1], xh[2 * n + e],
+                             xl[2 * n + e]);
+            uint32_t lh[4], ll[4], bh[2], bl[2];
+            const bf16* at_l = lb + (mr + 8 * (mi >> 1)) * DC_LB + 8 * (mi & 1);
+            const bf16* at_b = lb + (2 * DC_TOKENS + half * 8 + mr) * DC_LB + 8 * (mi & 1);
+            ldmatrix_x4(lh, at_l);
+            ldmatrix_x4(ll, at_l + DC_TOKENS * DC_LB);
+            ldmatrix_x2(bh, at_b);
+            ldmatrix_x2(bl, at_b + DC_TOKENS * DC_LB);
             uint32_t uh[4], ul[4];
 #pragma unroll
             for (int n = 0; n < 2; ++n) {
-                float u[4] = {0.f, 0.f, 0.f, 0.f}, ulow[4] = {0.f, 0.f, 0.f, 0.f};
+                float u[4] = {0.f, 0.f, 0.f, 0.f}, u1[4] = {0.f, 0.f, 0.f, 0.f}, u2[4] = {0.f, 0.f, 0.f, 0.f};
                 mma_bf16_16816(u, xh, lh[2 * n], lh[2 * n + 1]);
-                mma_bf16_16816(ulow, xl, lh[2 * n], lh[2 * n + 1]);
-                mma_bf16_16816(ulow, xh, ll[2 * n], ll[2 * n + 1]);
-                dc_split(u[0] + ulow[0], u[1] + ulow[1], uh[2 * n], ul[2 * n]);
-                dc_split(u[2] + ulow[2], u[3] + ulow[3], uh[2 * n + 1], ul[2 * n + 1]);
+                mma_bf16_16816(u1, xl, lh[2 * n], lh[2 * n + 1]);
+                mma_bf16_16816(u2, xh, ll[2 * n], ll[2 * n + 1]);
+                dc_split(u[0] + (u1[0] + u2[0]), u[1] + (u1[1] + u2[1]), uh[2 * n], ul[2 * n]);
+                dc_split(u[2] + (u1[2] + u2[2]), u[3] + (u1[3] + u2[3]), uh[2 * n + 1], ul[2 * n + 1]);
             }
             // ---- state: decay, then the chunk's writes -------------------------------------------------------
             const bf16* ke = mats + 4 * DC_TOKENS * RS + (mr + 8 * (mi & 1)) * RS + 8 * (mi >> 1);
@@ -376,26 +428,26 @@ __global__ void __launch_bounds__(128) delta_chunk_scan_kernel(DeltaChunkArgs p)
                 for (int x = 0; x < 2; ++x) {
                     const float2 f = *reinterpret_cast<const float2*>(gamma + (j + x) * 8 + 2 * t4);
                     s[j + x][0] *= f.x; s[j + x][1] *= f.y; s[j + x][2] *= f.x; s[j + x][3] *= f.y;
-                    mma_bf16_16816(s[j + x], uh, eh[2 * x], eh[2 * x + 1]);
-                    mma_bf16_16816(s[j + x], ul, eh[2 * x], eh[2 * x + 1]);
-                    mma_bf16_16816(s[j + x], uh, el[2 * x], el[2 * x + 1]);
                 }
+#pragma unroll
+                for (int x = 0; x < 2; ++x) mma_bf16_16816(s[j + x], uh, eh[2 * x], eh[2 * x + 1]);
+#pragma unroll
+                for (int x = 0; x < 2; ++x) mma_bf16_16816(s[j + x], ul, eh[2 * x], eh[2 * x + 1]);
+#pragma unroll
+                for (int x = 0; x < 2; ++x) mma_bf16_16816(s[j + x], uh, el[2 * x], el[2 * x + 1]);
             }
-            // ---- read-out ------------------------------------------------------------------------------------
+            // ---- read-out of this warp's eight tokens ----------------------------------------------------------
+            mma_bf16_16816(out, uh, bh[0], bh[1]);
+            mma_bf16_16816(out, ul, bh[0], bh[1]);
+            mma_bf16_16816(out, uh, bl[0], bl[1]);
 #pragma unroll
-            for (int n = 0; n < 2; ++n) {
-                mma_bf16_16816(r[n], uh, bh[2 * n], bh[2 * n + 1]);
-                mma_bf16_16816(rl[n], ul, bh[2 * n], bh[2 * n + 1]);
-                mma_bf16_16816(rl[n], uh, bl[2 * n], bl[2 * n + 1]);
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int t = i * DC_TOKENS + n * 8 + 2 * t4 + (e & 1), c = c0 + g + 8 * (e >> 1);
-                    if (t < p.count && c < a.vdim) a.o[((int64_t)(p.row0 + t) * a.H + h) * a.vdim + c] = r[n][e] + rl[n][e];
-                }
+            for (int e = 0; e < 4; ++e) {
+                const int t = i * DC_TOKENS + half * 8 + 2 * t4 + (e & 1), c = c0 + g + 8 * (e >> 1);
+                if (t < p.count && c < a.vdim) a.o[((int64_t)(p.row0 + t) * a.H + h) * a.vdim + c] = out[e];
             }
         }
         if (i + 1 < chunks) {
-            __syncthreads();  // every warp has read the stage
+            __syncthreads();  // every warp has read the stage, and its partner's sums
             if (threadIdx.x == 0 && i + DC_STAGES < chunks) load(i + DC_STAGES);
         }
     }
@@ -430,44 +482,98 @@ static int launch_chunk_scan(const DeltaChunkArgs& p, cudaStream_t st) {
     static DeviceOnce once;
     const int dev = once.pending();
     if (dev != DeviceOnce::SET) {
-        const cudaError_t e = cudaFuncSetAttribute(delta_chunk_scan_kernel<KS>, cudaFuncAttributeMaxDynamicSharedMemorySize, DC_STAGES * (dc_head_bytes(KS * 16) + 4 * dc_value_block()));
+        const cudaError_t e = cudaFuncSetAttribute(delta_chunk_scan_kernel<KS>, cudaFuncAttributeMaxDynamicSharedMemorySize, DC_STAGES * (dc_head_bytes(KS * 32) + 4 * dc_value_block()));
         if (e != cudaSuccess) return (int)e;
         once.mark(dev);
     }
-    const size_t smem = (size_t)DC_STAGES * (dc_head_bytes(KS * 16) + p.warps * dc_value_block());
-    GLMB_LAUNCH(delta_chunk_scan_kernel<KS>, dim3(ceil_div(ceil_div(p.d.vdim, 16), p.warps), p.d.H), 32 * p.warps, smem, st, p);
+    const size_t smem = (size_t)DC_STAGES * (dc_head_bytes(KS * 32) + p.blocks * dc_value_block());
+    GLMB_LAUNCH(delta_chunk_scan_kernel<KS>, dim3(ceil_div(ceil_div(p.d.vdim, 16), p.blocks), p.d.H), 64 * p.blocks, smem, st, p);
     return (int)cudaGetLastError();
 }
 
+// The scan of a segment and the preparation of the next run side by side: a second stream per device, two halves of the records in turn.
+struct DeltaStreams {
+    cudaStream_t scan = nullptr;
+    cudaEvent_t prepared = nullptr, scanned[2] = {nullptr, nullptr};
+    bool ready = false;
+};
+static cudaError_t delta_streams(DeltaStreams** out) {
+    static std::mutex mutex;
+    static DeltaStreams per_device[DeviceOnce::MAX_DEVICES];
+    int dev = 0;
+    cudaError_t e = cudaGetDevice(&dev);
+    if (e != cudaSuccess) return e;
+    if (dev < 0 || dev >= DeviceOnce::MAX_DEVICES) return cudaErrorInvalidDevice;
+    std::lock_guard<std::mutex> lock(mutex);
+    DeltaStreams& s = per_device[dev];
+    if (!s.ready) {
+        int low = 0, high = 0;
+        cudaDeviceGetStreamPriorityRange(&low, &high);
+        if ((e = cudaStreamCreateWithPriority(&s.scan, cudaStreamNonBlocking, high)) != cudaSuccess) return e;
+        for (cudaEvent_t* event : {&s.prepared, &s.scanned[0], &s.scanned[1]})
+            if ((e = cudaEventCreateWithFlags(event, cudaEventDisableTiming)) != cudaSuccess) return e;
+        s.ready = true;
+    }
+    *out = &s;
+    return cudaSuccess;
+}
+
+static int launch_scan_of(const DeltaChunkArgs& p, cudaStream_t st) {
+    switch (p.d.dimp / 32) {
+        case 1: return launch_chunk_scan<1>(p, st);
+        case 2: return launch_chunk_scan<2>(p, st);
+        case 3: return launch_chunk_scan<3>(p, st);
+        default: return launch_chunk_scan<4>(p, st);
+    }
+}
+
 // bf16, consecutive rows of one sequence: projection rows -> o, state and convolution history of the lane.  `records` holds at least H records
-// and is used for as many chunks at a time as fit.
+// and is used for as many chunks at a time as fit (half of it, in turn, when the step does not fit at once).
 GLMB_API int glmb_delta_chunk(const DeltaArgs* args, void* records, int64_t bytes, void* stream) {
     DeltaChunkArgs p;
     p.d = *args;
     const DeltaArgs& a = p.d;
     const int record = glmb_delta_chunk_record(a.dim, a.vdim, a.taps);
     if (!delta_sizes_ok(a) || a.decode || !record || a.dimp > 128 || (a.proj_stride & 7) || a.off_b < 2 * a.G * a.dim + a.H * a.vdim || a.H > 65535) return 1;
-    const int64_t chunks = bytes / ((int64_t)record * a.H);
+    const int64_t per_chunk = (int64_t)record * a.H, chunks = bytes / per_chunk, needed = ceil_div(a.rows, DC_TOKENS);
     if (chunks < 1 || (reinterpret_cast<uintptr_t>(records) & 15)) return 2;
     cudaStream_t st = (cudaStream_t)stream;
-    p.records = reinterpret_cast<unsigned char*>(records);
+    unsigned char* base = reinterpret_cast<unsigned char*>(records);
     const int blocks = ceil_div(a.vdim, 16);
-    p.warps = blocks * a.H <= 148 ? 1 : blocks * a.H <= 2 * 148 ? 2 : 4;
-    const int per_segment = (int)(chunks < ceil_div(a.rows, DC_TOKENS) ? chunks : ceil_div(a.rows, DC_TOKENS)) * DC_TOKENS;
+    p.blocks = blocks * a.H <= 148 ? 1 : blocks * a.H <= 2 * 148 ? 2 : 4;
     const size_t prep_smem = (size_t)3 * DC_TOKENS * (a.dimp + 4) * 4;
-    for (p.row0 = 0; p.row0 < a.rows; p.row0 += per_segment) {
-        p.count = min(per_segment, a.rows - p.row0);
-        p.last = p.row0 + p.count == a.rows;
+    auto prepare = [&] {
         GLMB_LAUNCH(delta_chunk_prep_kernel, dim3(ceil_div(p.count, DC_TOKENS), a.H), DC_THREADS, prep_smem, st, p);
-        int code = (int)cudaGetLastError();
-        if (code) return code;
-        switch (a.dimp / 32) {
-            case 1: code = launch_chunk_scan<2>(p, st); break;
-            case 2: code = launch_chunk_scan<4>(p, st); break;
-            case 3: code = launch_chunk_scan<6>(p, st); break;
-            default: code = launch_chunk_scan<8>(p, st);
+        return (int)cudaGetLastError();
+    };
+    const bool halves = needed > DC_OVERLAP_CHUNKS && chunks >= 2;  // worth two streams
+    const int64_t at_once = halves ? (needed + 1) / 2 < chunks / 2 ? (needed + 1) / 2 : chunks / 2 : chunks;
+    const int segment = (int)(at_once < needed ? at_once : needed) * DC_TOKENS;
+    if (!halves) {
+        p.records = base;
+        for (p.row0 = 0; p.row0 < a.rows; p.row0 += segment) {
+            p.count = min(segment, a.rows - p.row0);
+            p.last = p.row0 + p.count == a.rows;
+            int code = prepare();
+            if (!code) code = launch_scan_of(p, st);
+            if (code) return code;
         }
-        if (code) return code;
+        return 0;
     }
-    return 0;
+    DeltaStreams* side = nullptr;
+    cudaError_t e = delta_streams(&side);
+    if (e != cudaSuccess) return (int)e;
+    int i = 0;
+    for (p.row0 = 0; p.row0 < a.rows; p.row0 += segment, ++i) {
+        p.count = min(segment, a.rows - p.row0);
+        p.last = p.row0 + p.count == a.rows;
+        p.records = base + (i & 1) * at_once * per_chunk;
+        if (i >= 2 && (e = cudaStreamWaitEvent(st, side->scanned[i & 1], 0)) != cudaSuccess) return (int)e;
+        int code = prepare();
+        if (code) return code;
+        if ((e = cudaEventRecord(side->prepared, st)) != cudaSuccess || (e = cudaStreamWaitEvent(side->scan, side->prepared, 0)) != cudaSuccess) return (int)e;
+        if ((code = launch_scan_of(p, side->scan))) return code;
+        if ((e = cudaEventRecord(side->scanned[i & 1], side->scan)) != cudaSuccess) return (int)e;
+    }
+    return (int)cudaStreamWaitEvent(st, side->scanned[(i - 1) & 1], 0);
 }

@@ -199,23 +199,20 @@ __global__ void __launch_bounds__(DR_THREADS) delta_out_kernel(DeltaArgs a) {
     const float* o = a.o + unit * a.vdim;
     const T* gate = reinterpret_cast<const T*>(a.gate) + (int64_t)row * a.gate_stride + h * a.vdim;
     T* out = reinterpret_cast<T*>(a.out) + (int64_t)row * a.out_stride + h * a.vdim;
-    if (!(a.vdim & 7) && a.vdim <= 256) {  // eight channels per lane, everything asked for at once
-        const int c = lane * 8;
-        float x[8], z[8], w[8], ss = 0.f;
-#pragma unroll
-        for (int e = 0; e < 8; ++e) x[e] = 0.f;
+    if (!(a.vdim & 3) && a.vdim <= 128 && !(a.gate_stride & 3) && !(a.out_stride & 3)) {  // four channels per lane, everything asked for at once
+        const int c = lane * 4;
+        float x[4] = {0.f, 0.f, 0.f, 0.f}, z[4], w[4];
         if (c < a.vdim) {
-            load8(o + c, x);
-            load8(gate + c, z);
-            load8(a.norm + c, w);
+            load4(o + c, x);
+            load4(gate + c, z);
+            load4(a.norm + c, w);
         }
-#pragma unroll
-        for (int e = 0; e < 8; ++e) ss = fmaf(x[e], x[e], ss);
-        const float denom = sqrtf(warp_sum(ss) / (float)a.vdim + a.eps);
+        const float ss = warp_sum(x[0] * x[0] + x[1] * x[1] + x[2] * x[2] + x[3] * x[3]);
+        const float inv = 1.f / sqrtf(ss / (float)a.vdim + a.eps);
         if (c >= a.vdim) return;
 #pragma unroll
-        for (int e = 0; e < 8; ++e) x[e] = x[e] / denom * w[e] * sigmoidf_precise(z[e]);
-        store8(out + c, x);
+        for (int e = 0; e < 4; ++e) x[e] = x[e] * inv * w[e] * sigmoidf_precise(z[e]);
+        store4(out + c, x);
         return;
     }
     float ss = 0.f;

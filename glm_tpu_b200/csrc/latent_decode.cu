@@ -22,8 +22,8 @@ namespace cg = cooperative_groups;
 #define LD_THREADS (LD_WARPS * 32)
 #define LD_BOX (LD_KEYS * 128)
 #define LD_PSTRIDE 72
-#define LD_CLUSTER 8
-#define LD_CLUSTERS 16  // clusters the grid aims at: two per graphics processing cluster
+#define LD_CLUSTER 4
+#define LD_CLUSTERS 32  // clusters the grid aims at: all of them resident at once (of eight CTAs only fifteen were)
 #define LD_LOG2E 1.4426950408889634f
 
 static inline int ld_boxes(int W) { return (W + 63) / 64; }
@@ -280,7 +280,7 @@ __global__ void __launch_bounds__(LD_THREADS, 1) latent_decode_kernel(const __gr
 // ---------------------------------------------------------------------------------------------------
 #define LM_WARPS 8
 #define LM_COLS 32
-#define LM_PARTS 16
+#define LM_PARTS 32
 
 // grid (pieces of LM_COLS value channels, H); up to R rows.
 template <int R>
@@ -377,7 +377,7 @@ static int launch_latent_decode(const LatentArgs& a, int cluster, cudaStream_t s
 }
 
 // Attention and value projection of 1..8 rows, bf16, lat <= 512, lat + pe <= 640 (both multiples of 16): qa, cache -> out.
-// part_o / part_ml hold max(rows, LD_CLUSTERS) states per head: [max(rows, 16), H, lat] and [.., 2] fp32.
+// part_o / part_ml hold max(rows, LD_CLUSTERS) states per head: [max(rows, 32), H, lat] and [.., 2] fp32.
 GLMB_API int glmb_latent_decode(const LatentArgs* args, void* stream) {
     LatentArgs a = *args;
     if (!latent_ok(a) || a.rows > GLMB_MAX_ROWS || a.lat > 512 || a.lat + a.pe > 640 || (a.lat & 15) || (a.pe & 15) || !a.part_o || !a.part_ml) return 1;

@@ -101,8 +101,8 @@ def workspace_elements(g, cache: HybridCacheConfig, rows: int, *, prefill: bool,
             few = min(rows, ABSORB_ROWS) if prefill else rows
             need(t, "qa", few * m.heads * (lat + pe))
             need(t, "o_lat", few * m.heads * m.kv_rank)
-            need(f, "part_o", max(few, 16) * m.heads * lat)
-            need(f, "part_ml", max(few, 16) * m.heads * 2)
+            need(f, "part_o", max(few, 32) * m.heads * lat)
+            need(f, "part_ml", max(few, 32) * m.heads * 2)
             if prefill and rows > ABSORB_ROWS:
                 heads = expand_heads(m, cache.context_capacity, cache.element_bytes)
                 need(t, "keys", cache.context_capacity * heads * pad16(m.dim + m.rot_dim))

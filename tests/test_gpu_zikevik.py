@@ -315,7 +315,7 @@ def test_latent_decode_attention(native_lib, shape):
     if rows > 2:
         active[2] = 0
     keep = [torch.tensor(positions, dtype=torch.int32, device=DEV), torch.arange(rows, dtype=torch.int32, device=DEV), torch.tensor(active, dtype=torch.int32, device=DEV)]
-    qa_d, gate_d, sink_d, part_o, part_ml = qa.to(BF16).to(DEV), gate.to(DEV), sink.to(DEV), f(max(rows, 16) * H * lat), f(max(rows, 16) * H * 2)
+    qa_d, gate_d, sink_d, part_o, part_ml = qa.to(BF16).to(DEV), gate.to(DEV), sink.to(DEV), f(max(rows, 32) * H * lat), f(max(rows, 32) * H * 2)
     uv_d = torch.nn.functional.pad(uv, (0, lat - rank)).contiguous().to(DEV)
     a = native.LatentArgs()
     a.proj, a.proj_stride, a.off_gate = gate_d.data_ptr(), H, 0
