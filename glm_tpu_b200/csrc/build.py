@@ -24,7 +24,7 @@ NVCC = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
 # sources each model family needs when the complete library has not been built
 COMPONENTS = {
     "namizen": ("parallel_block", "qkv_conv", "chunk_attention", "chunk_attention_tcgen05", "gemm_f32", "swiglu_rows", "gemv", "gemm_tcgen05", "misc", "peer_registry"),
-    "zikevik": ("parallel_block", "delta_rule", "delta_chunk", "latent", "latent_decode", "chunk_attention", "chunk_attention_tcgen05", "moe_rows", "route_sort", "gemm_f32", "swiglu_rows",
+    "zikevik": ("parallel_block", "delta_rule", "delta_chunk", "delta_step", "latent", "latent_decode", "chunk_attention", "chunk_attention_tcgen05", "moe_rows", "route_sort", "gemm_f32", "swiglu_rows",
                 "gemv", "gemm_tcgen05", "misc", "peer_registry"),
 }
 FLAGS = [

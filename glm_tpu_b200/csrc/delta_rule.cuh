@@ -9,6 +9,7 @@ struct DeltaArgs {
     const float* conv_w; int taps;               // [taps, C], C = 2 G dim + H vdim
     void* conv_state;                            // [lanes, taps, C]: slot = position mod taps
     const float* a; int64_t a_stride;            // [rows, H dim]: the decay's projection, before bias and softplus
+    const void *a2, *g2; int off_a, off_g, ra, rg;  // delta_step: second halves of the low-rank projections [H dim, ra], [H vdim, rg], inputs in proj
     const float *a_rate, *dt_bias;               // [H] (positive), [H dim]
     const int *row_pos, *row_lane, *row_active;  // row_active may be NULL
     float *q, *k, *v, *lg, *beta;                // [rows, G, dimp], same, [rows, H, vdim], [rows, H, dimp] (log of the decay), [rows, H]

@@ -31,7 +31,7 @@ from glm_tpu_b200.parallel.peer import PeerGroup
 from glm_tpu_b200.runner.lane_state import RING, LaneRegisters
 
 EXPAND_BYTES = 1 << 30  # keys and values of as many heads at a time as fit here
-RECORD_BYTES = 64 << 20  # what the chunked recurrence keeps between its two kernels stays in the L2
+RECORD_BYTES = 128 << 20  # what the chunked recurrence keeps between its two kernels
 ABSORB_ROWS = native.MAX_ROWS  # steps of up to this many rows attend over the cache rows as they are
 MAX_EXPERTS, MAX_TOP = 256, 32  # limits of the route sort and the router kernel
 
@@ -206,20 +206,25 @@ class ZikevikModel:
         h = ws.h[:rows]
         proj = ws.view("proj", rows, t.proj.shape[0])
         self._mm(h, t.proj, proj)
-        decay, gate = ws.view("a", rows, t.a2.shape[0]), ws.view("gate", rows, t.g2.shape[0])
-        self._mm(proj[:, t.off_a : t.off_a + t.a2.shape[1]], t.a2, decay)
-        self._mm(proj[:, t.off_g : t.off_g + t.g2.shape[1]], t.g2, gate)
         out = ws.view("mixed", rows, t.out.shape[1])
         a = native.DeltaArgs()
         self._rows(a, rows, row_pos, row_lane, row_active)
         a.proj, a.proj_stride, a.off_b = proj.data_ptr(), proj.stride(0), t.off_b
         a.conv_w, a.taps, a.conv_state = t.conv.data_ptr(), m.conv, state.conv[layer].data_ptr()
-        a.a, a.a_stride, a.a_rate, a.dt_bias = decay.data_ptr(), decay.stride(0), t.a_rate.data_ptr(), t.dt_bias.data_ptr()
+        a.a_rate, a.dt_bias, a.norm = t.a_rate.data_ptr(), t.dt_bias.data_ptr(), t.norm.data_ptr()
         a.q, a.k, a.v, a.lg, a.beta, a.o = (ws.flat[n].data_ptr() for n in ("dq", "dk", "dv", "lg", "beta", "do"))
         a.state = state.state[layer].data_ptr()
-        a.gate, a.gate_stride, a.norm = gate.data_ptr(), gate.stride(0), t.norm.data_ptr()
         a.out, a.out_stride = out.data_ptr(), out.stride(0)
         a.H, a.G, a.dim, a.dimp, a.vdim, a.decode, a.eps = m.heads, m.kv_heads, m.dim, pad_to(m.dim, 32), m.vdim, int(decode), self.g.norm_eps
+        ra, rg = t.a2.shape[1], t.g2.shape[1]
+        if decode and not (self.is_f32 or self.plain_kernels) and native.delta_step_takes(m.vdim, ra + rg):
+            a.a2, a.g2, a.off_a, a.off_g, a.ra, a.rg = t.a2.data_ptr(), t.g2.data_ptr(), t.off_a, t.off_g, ra, rg
+            native.delta_step(a)
+            return out
+        decay, gate = ws.view("a", rows, t.a2.shape[0]), ws.view("gate", rows, t.g2.shape[0])
+        self._mm(proj[:, t.off_a : t.off_a + ra], t.a2, decay)
+        self._mm(proj[:, t.off_g : t.off_g + rg], t.g2, gate)
+        a.a, a.a_stride, a.gate, a.gate_stride = decay.data_ptr(), decay.stride(0), gate.data_ptr(), gate.stride(0)
         if not decode and "records" in ws.flat and delta_record_bytes(m) and not self.plain_kernels:
             native.delta_chunk(a, ws.flat["records"])
         else:

@@ -120,6 +120,7 @@ class DeltaArgs(C.Structure):
         ("conv_w", C.c_void_p), ("taps", C.c_int),
         ("conv_state", C.c_void_p),
         ("a", C.c_void_p), ("a_stride", C.c_int64),
+        ("a2", C.c_void_p), ("g2", C.c_void_p), ("off_a", C.c_int), ("off_g", C.c_int), ("ra", C.c_int), ("rg", C.c_int),
         ("a_rate", C.c_void_p), ("dt_bias", C.c_void_p),
         ("row_pos", C.c_void_p), ("row_lane", C.c_void_p), ("row_active", C.c_void_p),
         ("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("lg", C.c_void_p), ("beta", C.c_void_p),
@@ -593,6 +594,15 @@ def delta_chunk(args: DeltaArgs, records) -> None:
 def delta_scan(args: DeltaArgs) -> None:
     """The recurrence, token by token."""
     _check(lib().glmb_delta_scan(C.byref(args), _stream()), "delta_scan")
+
+
+def delta_step_takes(vdim: int, ranks: int) -> bool:
+    return vdim <= 1024 and ranks <= 4096
+
+
+def delta_step(args: DeltaArgs) -> None:
+    """bf16 decode: everything between a delta-rule layer's two projections in one launch."""
+    _check(lib().glmb_delta_step(C.byref(args), _stream()), "delta_step")
 
 
 def delta_out(args: DeltaArgs, is_f32: bool) -> None:

@@ -77,7 +77,7 @@ def test_norm_weights_around_zero_and_scaled_embedding(native_lib, dtype):
     assert int(status) == 0 and not out[:, width:].any()
 
 
-def delta_case(m, rows, seed, heads_zero=()):
+def delta_case(m, rows, seed):
     """Projection rows and everything else a delta-rule mixer's kernels read, on the CPU in fp64 (bf16 values where the engine keeps bf16)."""
     gen = torch.Generator().manual_seed(seed)
     r = lambda *s: torch.randn(s, generator=gen).double()  # noqa: E731
@@ -138,6 +138,18 @@ class DeltaHarness:
         a.gate, a.gate_stride, a.norm, a.out, a.out_stride = p(keep["gate"]), keep["gate"].stride(0), p(keep["norm"]), p(out), out.stride(0)
         a.H, a.G, a.dim, a.dimp, a.vdim, a.rows, a.decode = m.heads, m.kv_heads, m.dim, self.dimp, m.vdim, rows, int(decode)
         a.lanes, a.capacity, a.eps, a.status = self.lanes, self.capacity, self.eps, p(self.status)
+        if fused:  # the low-rank halves: ranks as wide as the products, whose second table is the identity on this head's rows
+            ra, rg = -(-m.heads * m.dim // 8) * 8, -(-m.v_width // 8) * 8
+            wide = torch.zeros(rows, proj.shape[1] + ra + rg, dtype=T, device=DEV)
+            wide[:, : proj.shape[1]] = proj
+            wide[:, proj.shape[1] : proj.shape[1] + m.heads * m.dim], wide[:, proj.shape[1] + ra : proj.shape[1] + ra + m.v_width] = keep["a"].to(T), keep["gate"]
+            a2, g2 = torch.zeros(m.heads * m.dim, ra, dtype=T, device=DEV), torch.zeros(m.v_width, rg, dtype=T, device=DEV)
+            a2.fill_diagonal_(1.0), g2.fill_diagonal_(1.0)
+            a.proj, a.proj_stride, a.off_a, a.off_g, a.ra, a.rg, a.a2, a.g2 = p(wide), wide.stride(0), proj.shape[1], proj.shape[1] + ra, ra, rg, p(a2), p(g2)
+            native.delta_step(a)
+            torch.cuda.synchronize()
+            assert int(self.status) == 0 and (out[:, m.v_width :] == 2.0).all()
+            return out[:, : m.v_width], None
         if chunked:
             native.delta_chunk(a, self.records)
         else:
@@ -178,34 +190,28 @@ def test_delta_rule_in_portions(native_lib, shape, kernel):
 
 
 @pytest.mark.parametrize("shape", DELTA_SHAPES)
-@pytest.mark.parametrize("kernel", ["f32", "bf16"])
+@pytest.mark.parametrize("kernel", ["f32", "bf16", "fused"])
 def test_delta_rule_decoding_in_unequal_lanes(native_lib, shape, kernel):
     """One row per lane at unequal positions, an inactive lane whose state stays as it is, and a lane that starts over."""
     m = delta(*shape)
     dtype = F32 if kernel == "f32" else BF16
     cases = [delta_case(m, 40, seed=10 + i) for i in range(3)]
+    for c in cases:
+        c |= {key: cases[0][key] for key in ("conv", "a_log", "bias", "norm")}
+        c["a"] = c["a"].to(BF16).double()  # what a bf16 product with the identity gives back
     wants = [delta_expected(m, c, 1e-3) for c in cases]
     hx = DeltaHarness(native_lib, m, dtype, lanes=3)
     hx.run(cases[0], slice(0, 5), range(5), [2] * 5, decode=False)
-    frozen = None
     for step in range(12):
         at = [5 + step, step if step < 6 else step - 6, 0 if step < 8 else step - 8]  # lane 1 starts over after six tokens
         active = [1, 1, int(step >= 8)]
         rows = {key: torch.stack([cases[i][key][at[i]] for i in range(3)]) if key in ("x", "b", "a", "gate") else cases[0][key] for key in cases[0]}
-        for key in ("conv", "a_log", "bias", "norm"):
-            for i in range(1, 3):
-                cases[i][key] = cases[0][key]
-        if step == 0:
-            wants = [delta_expected(m, c, 1e-3) for c in cases]
-            hx = DeltaHarness(native_lib, m, dtype, lanes=3)
-            hx.run(cases[0], slice(0, 5), range(5), [2] * 5, decode=False)
-            frozen = hx.state[0].clone()
-        out, o = hx.run(rows, slice(0, 3), at, [2, 1, 0], decode=True, active=active)
+        out, _ = hx.run(rows, slice(0, 3), at, [2, 1, 0], decode=True, fused=kernel == "fused", active=active)
         for i in range(3):
             if active[i]:
                 close(out[i], wants[i][0][at[i]], 1e-3 if dtype is F32 else 0.03)
         if step < 8:
-            assert torch.isnan(hx.state[0]).all() and torch.isnan(frozen).all()
+            assert torch.isnan(hx.state[0]).all() and torch.isnan(hx.ring[0].float()).all()
 
 
 def latent_case(m, total, seed, sharp=2.0):
