@@ -48,7 +48,7 @@ __device__ __forceinline__ void dt_prefetch(const void* p, int64_t bytes) {
 
 // grid (CTAs of a cluster, H, rows)
 template <int DQ>
-__global__ void __launch_bounds__(DT_THREADS) delta_step_kernel(DeltaArgs a) {
+__global__ void __launch_bounds__(DT_THREADS, DQ <= 4 ? 4 : 2) delta_step_kernel(DeltaArgs a) {
     constexpr int DP = DQ * 32;
     asm volatile("griddepcontrol.launch_dependents;");
     cg::cluster_group cluster = cg::this_cluster();
@@ -197,7 +197,8 @@ GLMB_API int glmb_delta_step(const DeltaArgs* args, void* stream) {
     const DeltaArgs a = *args;
     if (!delta_sizes_ok(a) || !a.decode || a.taps < 1 || !a.a2 || !a.g2 || a.ra < 8 || a.rg < 8 || (a.ra & 7) || (a.rg & 7) || a.ra + a.rg > 4096 || a.vdim > DT_VALUES * DT_CLUSTER) return 1;
     if ((reinterpret_cast<uintptr_t>(a.a2) | reinterpret_cast<uintptr_t>(a.g2)) & 15) return 1;
-    const int cluster = a.vdim >= 64 ? 4 : a.vdim >= 32 ? 2 : 1;
+    int cluster = a.vdim >= 64 ? 4 : a.vdim >= 32 ? 2 : 1;
+    while (cluster > 1 && (int64_t)cluster * a.H * a.rows > 4 * 148 && a.vdim * 2 <= cluster * DT_VALUES) cluster /= 2;  // all CTAs resident at once
     cudaStream_t st = (cudaStream_t)stream;
     switch (a.dimp / 32) {
         case 1: return launch_step<1>(a, cluster, st);

@@ -47,10 +47,38 @@ __global__ void __launch_bounds__(LR_THREADS) latent_rows_kernel(LatentArgs a) {
         dst = reinterpret_cast<T*>(a.cache) + ((int64_t)lane * a.capacity + pos) * (a.lat + a.pe);
     }
     float ss = 0.f;
-    for (int c = threadIdx.x; c < n; c += LR_THREADS) { const float x = to_f32(src[c]); ss = fmaf(x, x, ss); }
-    const float denom = sqrtf(lr_block_sum(ss, scratch) / (float)n + a.eps);
-    if (!ok) return;
-    for (int c = threadIdx.x; c < cols; c += LR_THREADS) from_f32(c < n ? to_f32(src[c]) / denom * w[c] : 0.f, dst[c]);
+    if (!(n & 7) && n == cols && n <= LR_THREADS * 16) {  // whole vectors, all of them asked for before the first is used
+        float x[2][8];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const int c = (threadIdx.x + i * LR_THREADS) * 8;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) x[i][e] = 0.f;
+            if (c < n) load8(src + c, x[i]);
+        }
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+            for (int e = 0; e < 8; ++e) ss = fmaf(x[i][e], x[i][e], ss);
+        const float denom = sqrtf(lr_block_sum(ss, scratch) / (float)n + a.eps);
+        if (!ok) return;
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const int c = (threadIdx.x + i * LR_THREADS) * 8;
+            if (c < n) {
+                float y[8];
+                load8(w + c, y);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) y[e] *= x[i][e] / denom;
+                store8(dst + c, y);
+            }
+        }
+    } else {
+        for (int c = threadIdx.x; c < n; c += LR_THREADS) { const float x = to_f32(src[c]); ss = fmaf(x, x, ss); }
+        const float denom = sqrtf(lr_block_sum(ss, scratch) / (float)n + a.eps);
+        if (!ok) return;
+        for (int c = threadIdx.x; c < cols; c += LR_THREADS) from_f32(c < n ? to_f32(src[c]) / denom * w[c] : 0.f, dst[c]);
+    }
     if (is_q) return;
     const T* pe = src + a.kv_rank;
     const int half = a.rot_dim / 2;
@@ -67,19 +95,33 @@ __global__ void __launch_bounds__(LR_THREADS) latent_rows_kernel(LatentArgs a) {
     }
 }
 
-// A thread per pair, grid (pieces of H rot / 2 pairs, rows).
-template <typename T>
+// A thread per VEC pairs, grid (pieces of H rot / (2 VEC) threads, rows).
+template <typename T, int VEC>
 __global__ void __launch_bounds__(256) latent_query_kernel(LatentArgs a) {
     GLMB_PDL_PROLOGUE();
-    const int half = a.rot_dim / 2, i = blockIdx.x * 256 + threadIdx.x, row = blockIdx.y;
-    if (i >= a.H * half) return;
+    const int half = a.rot_dim / 2, per = half / VEC, i = blockIdx.x * 256 + threadIdx.x, row = blockIdx.y;
+    if (i >= a.H * per) return;
     bool ok;
-    const int pos = latent_pos(a, row, ok);
-    T* q = reinterpret_cast<T*>(a.q) + ((int64_t)row * a.H + i / half) * a.dimp + a.dim + i % half * 2;
-    const float2 cs = a.rot[(int64_t)pos * half + i % half];
-    const float u = to_f32(q[0]), v = to_f32(q[1]);
-    from_f32(u * cs.x - v * cs.y, q[0]);
-    from_f32(v * cs.x + u * cs.y, q[1]);
+    const int pos = latent_pos(a, row, ok), p = i % per * VEC;
+    T* q = reinterpret_cast<T*>(a.q) + ((int64_t)row * a.H + i / per) * a.dimp + a.dim + p * 2;
+    const float2* cs = a.rot + (int64_t)pos * half + p;
+    if constexpr (VEC == 4) {
+        float x[8];
+        load8(q, x);
+        const float4 t0 = *reinterpret_cast<const float4*>(cs), t1 = *reinterpret_cast<const float4*>(cs + 2);
+        const float cosine[4] = {t0.x, t0.z, t1.x, t1.z}, sine[4] = {t0.y, t0.w, t1.y, t1.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const float u = x[2 * e], v = x[2 * e + 1];
+            x[2 * e] = u * cosine[e] - v * sine[e];
+            x[2 * e + 1] = v * cosine[e] + u * sine[e];
+        }
+        store8(q, x);
+    } else {
+        const float u = to_f32(q[0]), v = to_f32(q[1]);
+        from_f32(u * cs->x - v * cs->y, q[0]);
+        from_f32(v * cs->x + u * cs->y, q[1]);
+    }
 }
 
 // grid (pieces of 256 latent columns, H, blocks of LA_ROWS rows): a lane owns eight columns, the warps share the unrotated dimensions.
@@ -200,7 +242,17 @@ GLMB_API int glmb_latent_rows(const LatentArgs* args, int is_f32, void* stream) 
 GLMB_API int glmb_latent_query(const LatentArgs* args, int is_f32, void* stream) {
     const LatentArgs a = *args;
     if (!latent_ok(a)) return 1;
-    LATENT_LAUNCH(latent_query_kernel, dim3(ceil_div(a.H * (a.rot_dim / 2), 256), a.rows), 256, 0);
+    const int vec = (a.dim & 7) || (a.rot_dim & 7) ? 1 : 4;
+    const dim3 grid(ceil_div(a.H * (a.rot_dim / 2 / vec), 256), a.rows);
+    cudaStream_t st = (cudaStream_t)stream;
+    if (is_f32) {
+        if (vec == 4) GLMB_LAUNCH((latent_query_kernel<float, 4>), grid, 256, 0, st, a);
+        else GLMB_LAUNCH((latent_query_kernel<float, 1>), grid, 256, 0, st, a);
+    } else {
+        if (vec == 4) GLMB_LAUNCH((latent_query_kernel<bf16, 4>), grid, 256, 0, st, a);
+        else GLMB_LAUNCH((latent_query_kernel<bf16, 1>), grid, 256, 0, st, a);
+    }
+    return (int)cudaGetLastError();
 }
 template <typename T, int R>
 static int launch_absorb(const LatentArgs& a, cudaStream_t st) {

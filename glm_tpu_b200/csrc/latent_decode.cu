@@ -282,18 +282,22 @@ __global__ void __launch_bounds__(LD_THREADS, 1) latent_decode_kernel(const __gr
 #define LM_COLS 32
 #define LM_PARTS 32
 
-// grid (pieces of LM_COLS value channels, H); up to R rows.
+// grid (pieces of LM_COLS value channels, H); up to R rows.  In the projection eight lanes share a value channel, a warp has four.
 template <int R>
 __global__ void __launch_bounds__(LM_WARPS * 32) latent_merge_value_kernel(LatentArgs a) {
     asm volatile("griddepcontrol.launch_dependents;");
     const int h = blockIdx.y, c0 = blockIdx.x * LM_COLS, cols = min(LM_COLS, a.vdim - c0);
-    const bf16* w = reinterpret_cast<const bf16*>(a.uv) + ((int64_t)h * a.vdim + c0) * a.lat;
-    if (threadIdx.x == 0)
-        asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(w), "r"((uint32_t)(cols * a.lat * 2)) : "memory");
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, sub = lane & 7, c = warp * 4 + (lane >> 3);
+    const bf16* w = reinterpret_cast<const bf16*>(a.uv) + ((int64_t)h * a.vdim + c0 + min(c, cols - 1)) * a.lat;
+    uint4 wv[8];  // this lane's weights: they do not depend on the kernel before
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        wv[i] = make_uint4(0, 0, 0, 0);
+        if (sub * 8 + i * 64 < a.lat) wv[i] = *reinterpret_cast<const uint4*>(w + sub * 8 + i * 64);
+    }
     asm volatile("griddepcontrol.wait;" ::: "memory");
-    extern __shared__ __align__(16) float o_s[];  // [R][lat]
+    extern __shared__ __align__(16) float o_s[];  // [2][R][lat]
     __shared__ float w_s[R][LM_PARTS];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (warp < a.rows) {  // a warp per row: weights of its parts, divided by the total
         const float sink2 = a.sink ? a.sink[h] * LD_LOG2E : -INFINITY;
         float2 ml = make_float2(-INFINITY, 0.f);
@@ -301,45 +305,50 @@ __global__ void __launch_bounds__(LM_WARPS * 32) latent_merge_value_kernel(Laten
         const float top = warp_max(fmaxf(ml.x, sink2));
         const float f = ml.x == -INFINITY ? 0.f : exp2f(ml.x - top);
         const float total = warp_sum(ml.y * f) + (a.sink ? exp2f(sink2 - top) : 0.f);
-        if (lane < a.parts) w_s[warp][lane] = total > 0.f ? f / total : 0.f;
+        w_s[warp][lane] = total > 0.f ? f / total : 0.f;
     }
     __syncthreads();
-    for (int i = threadIdx.x * 4; i < a.rows * a.lat; i += LM_WARPS * 32 * 4) {
-        const int r = i / a.lat, c = i % a.lat;
-        const float* src = a.part_o + ((int64_t)r * a.H + h) * a.parts * a.lat + c;
+    const int half = threadIdx.x >> 7, quads = a.rows * a.lat / 4, parts = (a.parts + 1) / 2;  // two halves of the parts side by side
+    for (int i = threadIdx.x & 127; i < quads; i += 128) {
+        const int r = i * 4 / a.lat, at = i * 4 % a.lat;
+        const float* src = a.part_o + (((int64_t)r * a.H + h) * a.parts + half * parts) * a.lat + at;
+        const int n = min(parts, a.parts - half * parts);
         float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 8
-        for (int p = 0; p < a.parts; ++p) {
+        for (int p = 0; p < n; ++p) {
             const float4 x = *reinterpret_cast<const float4*>(src + (int64_t)p * a.lat);
-            const float f = w_s[r][p];
+            const float f = w_s[r][half * parts + p];
             v.x = fmaf(x.x, f, v.x); v.y = fmaf(x.y, f, v.y); v.z = fmaf(x.z, f, v.z); v.w = fmaf(x.w, f, v.w);
         }
-        *reinterpret_cast<float4*>(o_s + i) = v;
+        *reinterpret_cast<float4*>(o_s + half * a.rows * a.lat + i * 4) = v;
     }
     __syncthreads();
-    for (int c = warp; c < cols; c += LM_WARPS) {
-        float acc[R];
+    for (int i = threadIdx.x; i < quads; i += LM_WARPS * 32) {
+        const float4 x = reinterpret_cast<const float4*>(o_s)[i], y = reinterpret_cast<const float4*>(o_s)[quads + i];
+        reinterpret_cast<float4*>(o_s)[i] = make_float4(x.x + y.x, x.y + y.y, x.z + y.z, x.w + y.w);
+    }
+    __syncthreads();
 #pragma unroll
-        for (int r = 0; r < R; ++r) acc[r] = 0.f;
-        for (int l = lane * 8; l < a.lat; l += 256) {
-            float x[8];
-            load8(w + (int64_t)c * a.lat + l, x);
+    for (int r = 0; r < R; ++r) {
+        if (r >= a.rows) break;
+        float sum = 0.f;
 #pragma unroll
-            for (int r = 0; r < R; ++r)
-                if (r < a.rows) {
-                    float y[8];
-                    load8(o_s + r * a.lat + l, y);
+        for (int i = 0; i < 8; ++i) {
+            const int l = sub * 8 + i * 64;
+            if (l < a.lat) {
+                float x[8];
+                load8(o_s + r * a.lat + l, x);
+                const uint32_t u[4] = {wv[i].x, wv[i].y, wv[i].z, wv[i].w};
 #pragma unroll
-                    for (int e = 0; e < 8; ++e) acc[r] = fmaf(x[e], y[e], acc[r]);
-                }
-        }
-#pragma unroll
-        for (int r = 0; r < R; ++r) {
-            const float y = warp_sum(acc[r]);
-            if (lane == 0 && r < a.rows) {
-                const float z = __bfloat162float(reinterpret_cast<const bf16*>(a.proj)[(int64_t)r * a.proj_stride + a.off_gate + h]);
-                reinterpret_cast<bf16*>(a.out)[(int64_t)r * a.out_stride + h * a.vdim + c0 + c] = __float2bfloat16_rn(y * sigmoidf_precise(z));
+                for (int e = 0; e < 4; ++e) sum = fmaf(bf16_hi(u[e]), x[2 * e + 1], fmaf(bf16_lo(u[e]), x[2 * e], sum));
             }
+        }
+        sum += __shfl_xor_sync(0xffffffffu, sum, 1);
+        sum += __shfl_xor_sync(0xffffffffu, sum, 2);
+        sum += __shfl_xor_sync(0xffffffffu, sum, 4);
+        if (sub == 0 && c < cols) {
+            const float z = __bfloat162float(reinterpret_cast<const bf16*>(a.proj)[(int64_t)r * a.proj_stride + a.off_gate + h]);
+            reinterpret_cast<bf16*>(a.out)[(int64_t)r * a.out_stride + h * a.vdim + c0 + c] = __float2bfloat16_rn(sum * sigmoidf_precise(z));
         }
     }
 }
@@ -390,7 +399,7 @@ GLMB_API int glmb_latent_decode(const LatentArgs* args, void* stream) {
     const int code = a.H <= 16 ? launch_latent_decode<1>(a, cluster, (cudaStream_t)stream) : launch_latent_decode<2>(a, cluster, (cudaStream_t)stream);
     if (code) return code;
     const dim3 grid(ceil_div(a.vdim, LM_COLS), a.H);
-#define CALL(R) GLMB_LAUNCH(latent_merge_value_kernel<R>, grid, LM_WARPS * 32, (size_t)a.rows * a.lat * 4, (cudaStream_t)stream, a)
+#define CALL(R) GLMB_LAUNCH(latent_merge_value_kernel<R>, grid, LM_WARPS * 32, (size_t)2 * a.rows * a.lat * 4, (cudaStream_t)stream, a)
     if (a.rows == 1) CALL(1);
     else if (a.rows <= 4) CALL(4);
     else CALL(8);
