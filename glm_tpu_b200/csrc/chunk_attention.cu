@@ -37,7 +37,7 @@ __device__ __forceinline__ int ca_lane(const ChunkAttnArgs& a, int row) {
 __device__ __forceinline__ int ca_pos(const ChunkAttnArgs& a, int row) {
     const int pos = a.row_pos[row];
     if (pos >= 0 && pos < a.capacity) return pos;
-    if (threadIdx.x == 0) raise_status(a.status, GLMB_STATUS_BAD_INDEX);
+    if (threadIdx.x == 0 && (!a.row_active || a.row_active[row])) raise_status(a.status, GLMB_STATUS_BAD_INDEX);  // a frozen lane may be full
     return min(max(pos, 0), a.capacity - 1);
 }
 // bf16 value and bf16 remainder of two weights, packed as mma operands

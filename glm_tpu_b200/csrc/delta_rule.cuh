@@ -30,12 +30,11 @@ __device__ __forceinline__ int delta_lane(const DeltaArgs& a, int row) {
     return min(max(lane, 0), a.lanes - 1);
 }
 __device__ __forceinline__ bool delta_writes(const DeltaArgs& a, int row) {  // an inactive row, or one at no position, leaves the lane as it is
+    if (a.row_active && a.row_active[row] == 0) return false;
     const int pos = a.row_pos[row];
-    if (pos < 0 || pos >= a.capacity) {
-        if (threadIdx.x == 0) raise_status(a.status, GLMB_STATUS_BAD_INDEX);
-        return false;
-    }
-    return !a.row_active || a.row_active[row] != 0;
+    if (pos >= 0 && pos < a.capacity) return true;
+    if (threadIdx.x == 0) raise_status(a.status, GLMB_STATUS_BAD_INDEX);
+    return false;
 }
 // log(1 + e^z) = max(z, 0) + log(1 + e), e = e^-|z| in (0, 1]; log(1 + e) = 2 artanh(e / (2 + e)) by its power series, whose argument is at most
 // 1/3: the first term left out is below 2^-27 of the sum, and small results keep their relative accuracy.

@@ -28,7 +28,7 @@ struct LatentArgs {
 __device__ __forceinline__ int latent_pos(const LatentArgs& a, int row, bool& ok) {
     const int pos = a.row_pos[row];
     ok = pos >= 0 && pos < a.capacity;
-    if (!ok && threadIdx.x == 0) raise_status(a.status, GLMB_STATUS_BAD_INDEX);
+    if (!ok && threadIdx.x == 0 && (!a.row_active || a.row_active[row])) raise_status(a.status, GLMB_STATUS_BAD_INDEX);  // a frozen lane may be full
     return min(max(pos, 0), a.capacity - 1);
 }
 

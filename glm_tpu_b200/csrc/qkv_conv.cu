@@ -156,7 +156,7 @@ __global__ void __launch_bounds__(QC_THREADS) qkv_conv_kernel(QkvConvArgs a) {
         int pos = a.row_pos[row];
         const bool bad = pos < 0 || pos >= a.capacity;
         if (bad) {
-            if (c == 0) raise_status(a.status, GLMB_STATUS_BAD_INDEX);
+            if (c == 0 && active) raise_status(a.status, GLMB_STATUS_BAD_INDEX);  // a frozen lane may be full
             pos = min(max(pos, 0), a.capacity - 1);
         }
         const float* y = y_s + r * hd;

@@ -454,6 +454,18 @@ def test_a_failed_position_is_reported_and_refused(native_lib):
         runner.close()
 
 
+def test_a_lane_filled_to_the_last_position_does_not_disturb_the_others(native_lib):
+    g = geometries()["tiny"]
+    ck = sharp_checkpoint(g, 11)
+    full, other = tokens_for(g, 64, 1), tokens_for(g, 12, 2)
+    runner = runner_for(g, ck, F32, capacity=64, lanes=2)
+    try:
+        check(feed(runner, 0, full, [50] + list(range(51, 64))), expected(g, ck, full), F32)
+        check(feed(runner, 1, other, [5] + list(range(6, 12))), expected(g, ck, other), F32)
+    finally:
+        runner.close()
+
+
 # ------------------------------------------------------------------------------------------------ the engine's own entry points
 def near_greedy(g, ck, prompt, tokens, slack):
     """Every generated token is the plain model's best, or within ``slack`` (of the logits' spread) of it."""
