@@ -75,7 +75,8 @@ def parameters(g) -> int:
         return total
     from glm_tpu_b200.models.glm_moe_dsa.weights import projection_shapes
 
-    return sum(a * b for i in range(g.num_layers) for a, b in projection_shapes(g, i).values()) + g.vocab_size * g.hidden_size
+    shapes = [shape for i in range(g.num_layers) for shape in projection_shapes(g, i).values()]
+    return sum((g.routed_top_k if len(shape) == 3 else 1) * shape[-2] * shape[-1] for shape in shapes) + g.vocab_size * g.hidden_size
 
 
 def make_runner(family: str, size: dict, lanes: int, prefill_chunk: int, graphs: bool = True):

@@ -188,37 +188,49 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(DeltaArgs a) {
 }
 
 // ---------------------------------------------------------------------------------------------------
-// A warp per (row, head): out = o / rms(o) * norm * sigmoid(gate).
-template <typename T>
+// out = o / rms(o) * norm * sigmoid(gate) per (row, head).  VEC: heads up to 128 wide in whole vectors, a warp takes DR_UNITS of them, four channels
+// per lane, everything asked for at once; otherwise a warp per (row, head), any size.
+#define DR_UNITS 4
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(DR_THREADS) delta_out_kernel(DeltaArgs a) {
     GLMB_PDL_PROLOGUE();
     const int lane = threadIdx.x & 31;
-    const int64_t unit = (int64_t)blockIdx.x * DR_WARPS + (threadIdx.x >> 5);
-    if (unit >= (int64_t)a.rows * a.H) return;
-    const int row = (int)(unit / a.H), h = (int)(unit % a.H);
-    const float* o = a.o + unit * a.vdim;
-    const T* gate = reinterpret_cast<const T*>(a.gate) + (int64_t)row * a.gate_stride + h * a.vdim;
-    T* out = reinterpret_cast<T*>(a.out) + (int64_t)row * a.out_stride + h * a.vdim;
-    if (!(a.vdim & 3) && a.vdim <= 128 && !(a.gate_stride & 3) && !(a.out_stride & 3)) {  // four channels per lane, everything asked for at once
+    const int64_t units = (int64_t)a.rows * a.H, warp = (int64_t)blockIdx.x * DR_WARPS + (threadIdx.x >> 5);
+    if constexpr (VEC) {
         const int c = lane * 4;
-        float x[4] = {0.f, 0.f, 0.f, 0.f}, z[4], w[4];
-        if (c < a.vdim) {
-            load4(o + c, x);
-            load4(gate + c, z);
-            load4(a.norm + c, w);
-        }
-        const float ss = warp_sum(x[0] * x[0] + x[1] * x[1] + x[2] * x[2] + x[3] * x[3]);
-        const float inv = 1.f / sqrtf(ss / (float)a.vdim + a.eps);
-        if (c >= a.vdim) return;
+        const bool in = c < a.vdim;
+        float x[DR_UNITS][4], z[DR_UNITS][4], w[4] = {0.f, 0.f, 0.f, 0.f};
+        if (in) load4(a.norm + c, w);
 #pragma unroll
-        for (int e = 0; e < 4; ++e) x[e] = x[e] * inv * w[e] * sigmoidf_precise(z[e]);
-        store4(out + c, x);
-        return;
+        for (int i = 0; i < DR_UNITS; ++i) {
+            const int64_t unit = warp * DR_UNITS + i;
+#pragma unroll
+            for (int e = 0; e < 4; ++e) x[i][e] = z[i][e] = 0.f;
+            if (in && unit < units) {
+                load4(a.o + unit * a.vdim + c, x[i]);
+                load4(reinterpret_cast<const T*>(a.gate) + unit / a.H * a.gate_stride + unit % a.H * a.vdim + c, z[i]);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < DR_UNITS; ++i) {
+            const int64_t unit = warp * DR_UNITS + i;
+            const float ss = warp_sum(x[i][0] * x[i][0] + x[i][1] * x[i][1] + x[i][2] * x[i][2] + x[i][3] * x[i][3]);
+            const float inv = 1.f / sqrtf(ss / (float)a.vdim + a.eps);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) x[i][e] = x[i][e] * inv * w[e] * sigmoidf_precise(z[i][e]);
+            if (in && unit < units) store4(reinterpret_cast<T*>(a.out) + unit / a.H * a.out_stride + unit % a.H * a.vdim + c, x[i]);
+        }
+    } else {
+        if (warp >= units) return;
+        const int row = (int)(warp / a.H), h = (int)(warp % a.H);
+        const float* o = a.o + warp * a.vdim;
+        const T* gate = reinterpret_cast<const T*>(a.gate) + (int64_t)row * a.gate_stride + h * a.vdim;
+        T* out = reinterpret_cast<T*>(a.out) + (int64_t)row * a.out_stride + h * a.vdim;
+        float ss = 0.f;
+        for (int c = lane; c < a.vdim; c += 32) ss = fmaf(o[c], o[c], ss);
+        const float denom = sqrtf(warp_sum(ss) / (float)a.vdim + a.eps);
+        for (int c = lane; c < a.vdim; c += 32) from_f32(o[c] / denom * a.norm[c] * sigmoidf_precise(to_f32(gate[c])), out[c]);
     }
-    float ss = 0.f;
-    for (int c = lane; c < a.vdim; c += 32) ss = fmaf(o[c], o[c], ss);
-    const float denom = sqrtf(warp_sum(ss) / (float)a.vdim + a.eps);
-    for (int c = lane; c < a.vdim; c += 32) from_f32(o[c] / denom * a.norm[c] * sigmoidf_precise(to_f32(gate[c])), out[c]);
 }
 
 // ===================================================================================================
@@ -267,8 +279,16 @@ GLMB_API int glmb_delta_scan(const DeltaArgs* args, void* stream) {
 GLMB_API int glmb_delta_out(const DeltaArgs* args, int is_f32, void* stream) {
     const DeltaArgs a = *args;
     if (!delta_sizes_ok(a)) return 1;
-    const int grid = (int)(((int64_t)a.rows * a.H + DR_WARPS - 1) / DR_WARPS);
-    if (is_f32) GLMB_LAUNCH(delta_out_kernel<float>, grid, DR_THREADS, 0, (cudaStream_t)stream, a);
-    else GLMB_LAUNCH(delta_out_kernel<bf16>, grid, DR_THREADS, 0, (cudaStream_t)stream, a);
+    const bool vec = !(a.vdim & 3) && a.vdim <= 128 && !(a.gate_stride & 3) && !(a.out_stride & 3);
+    const int64_t per_block = DR_WARPS * (vec ? DR_UNITS : 1);
+    const int grid = (int)(((int64_t)a.rows * a.H + per_block - 1) / per_block);
+    cudaStream_t st = (cudaStream_t)stream;
+    if (is_f32) {
+        if (vec) GLMB_LAUNCH((delta_out_kernel<float, true>), grid, DR_THREADS, 0, st, a);
+        else GLMB_LAUNCH((delta_out_kernel<float, false>), grid, DR_THREADS, 0, st, a);
+    } else {
+        if (vec) GLMB_LAUNCH((delta_out_kernel<bf16, true>), grid, DR_THREADS, 0, st, a);
+        else GLMB_LAUNCH((delta_out_kernel<bf16, false>), grid, DR_THREADS, 0, st, a);
+    }
     return (int)cudaGetLastError();
 }
