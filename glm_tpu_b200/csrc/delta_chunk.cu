@@ -57,7 +57,7 @@ __device__ __forceinline__ void dc_split(float x, float y, uint32_t& hi, uint32_
 
 // One step of a sum over 16 lanes that leaves every lane with a sixteenth of the values: N values become N / 2.
 template <int N>
-__device__ __forceinline__ void dc_fold(float (&v)[32], int lane, int offset) {
+__device__ __forceinline__ void dc_fold(float (&v)[16], int lane, int offset) {
     const bool upper = lane & offset;
 #pragma unroll
     for (int i = 0; i < N / 2; ++i) {
@@ -92,7 +92,7 @@ __device__ __forceinline__ void dc_operands(const float* q_s, const float* k_s, 
 }
 
 // grid (chunks, H)
-__global__ void __launch_bounds__(DC_THREADS, 3) delta_chunk_prep_kernel(DeltaChunkArgs p) {
+__global__ void __launch_bounds__(DC_THREADS, 4) delta_chunk_prep_kernel(DeltaChunkArgs p) {
     GLMB_PDL_PROLOGUE();
     const DeltaArgs& a = p.d;
     extern __shared__ __align__(16) float smem_f[];
@@ -110,48 +110,44 @@ __global__ void __launch_bounds__(DC_THREADS, 3) delta_chunk_prep_kernel(DeltaCh
     const int start = a.row_pos[0], seq = delta_lane(a, 0);
     const bf16* state = reinterpret_cast<const bf16*>(a.conv_state) + (int64_t)seq * a.taps * C;
 
-    // ---- convolution: a thread takes eight channels of four tokens -----------------------------------------
-    const int kvec = a.dim / 8, vecs = 2 * kvec + a.vdim / 8;
+    // ---- convolution: a thread takes four channels of four tokens ------------------------------------------
+    const int kvec = a.dim / 4, vecs = 2 * kvec + a.vdim / 4;
     for (int i = tid; i < vecs * 4; i += DC_THREADS) {
         const int strip = i / vecs, vec = i - strip * vecs, first = strip * 4;
-        const int kind = vec < kvec ? 0 : vec < 2 * kvec ? 1 : 2, c = (kind == 0 ? vec : kind == 1 ? vec - kvec : vec - 2 * kvec) * 8;
+        const int kind = vec < kvec ? 0 : vec < 2 * kvec ? 1 : 2, c = (kind == 0 ? vec : kind == 1 ? vec - kvec : vec - 2 * kvec) * 4;
         const int chan = (kind == 0 ? kvh * a.dim : kind == 1 ? (a.G + kvh) * a.dim : 2 * a.G * a.dim + h * a.vdim) + c;
-        uint4 u[4 + DC_TAPS - 1];
+        uint2 u[4 + DC_TAPS - 1];
 #pragma unroll
         for (int j = 0; j < 4 + DC_TAPS - 1; ++j) {
             const int row = t0 + first + j - (DC_TAPS - 1);  // row of the step; before it: the lane's ring of projected rows
-            u[j] = make_uint4(0, 0, 0, 0);
-            if (row >= 0 && row < t0 + n) u[j] = *reinterpret_cast<const uint4*>(proj + (int64_t)row * a.proj_stride + chan);
-            else if (row < 0 && row >= -keep && start + row >= 0) u[j] = *reinterpret_cast<const uint4*>(state + (int64_t)((start + row) % a.taps) * C + chan);
+            u[j] = make_uint2(0, 0);
+            if (row >= 0 && row < t0 + n) u[j] = *reinterpret_cast<const uint2*>(proj + (int64_t)row * a.proj_stride + chan);
+            else if (row < 0 && row >= -keep && start + row >= 0) u[j] = *reinterpret_cast<const uint2*>(state + (int64_t)((start + row) % a.taps) * C + chan);
         }
-        float y[4][8];
+        float y[4][4];
 #pragma unroll
         for (int t = 0; t < 4; ++t)
 #pragma unroll
-            for (int e = 0; e < 8; ++e) y[t][e] = 0.f;
+            for (int e = 0; e < 4; ++e) y[t][e] = 0.f;
 #pragma unroll
         for (int j = 0; j < DC_TAPS; ++j) {
             const int tap = j - (DC_TAPS - a.taps);  // fewer taps: the oldest ones are not there
             if (tap < 0) continue;
-            float w[8];
-            load8(a.conv_w + (int64_t)tap * C + chan, w);
+            const float4 w = *reinterpret_cast<const float4*>(a.conv_w + (int64_t)tap * C + chan);
 #pragma unroll
             for (int t = 0; t < 4; ++t) {
-                const uint32_t x[4] = {u[t + j].x, u[t + j].y, u[t + j].z, u[t + j].w};
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    y[t][2 * e] = fmaf(w[2 * e], bf16_lo(x[e]), y[t][2 * e]);
-                    y[t][2 * e + 1] = fmaf(w[2 * e + 1], bf16_hi(x[e]), y[t][2 * e + 1]);
-                }
+                y[t][0] = fmaf(w.x, bf16_lo(u[t + j].x), y[t][0]);
+                y[t][1] = fmaf(w.y, bf16_hi(u[t + j].x), y[t][1]);
+                y[t][2] = fmaf(w.z, bf16_lo(u[t + j].y), y[t][2]);
+                y[t][3] = fmaf(w.w, bf16_hi(u[t + j].y), y[t][3]);
             }
         }
+        float* dst = kind == 2 ? v_out + ((int64_t)(c / 16) * DC_TOKENS + first) * DC_VB + c % 16 : (kind == 0 ? q_s : k_s) + first * RS + c;
+        const int stride = kind == 2 ? DC_VB : RS;
 #pragma unroll
-        for (int t = 0; t < 4; ++t) {
-#pragma unroll
-            for (int e = 0; e < 8; ++e) y[t][e] = first + t < n ? dc_silu(y[t][e]) : 0.f;
-            if (kind == 2) store8(v_out + ((int64_t)(c / 16) * DC_TOKENS + first + t) * DC_VB + c % 16, y[t]);
-            else store8((kind == 0 ? q_s : k_s) + (first + t) * RS + c, y[t]);
-        }
+        for (int t = 0; t < 4; ++t)
+            *reinterpret_cast<float4*>(dst + t * stride) = first + t < n ? make_float4(dc_silu(y[t][0]), dc_silu(y[t][1]), dc_silu(y[t][2]), dc_silu(y[t][3]))
+                                                                         : make_float4(0.f, 0.f, 0.f, 0.f);
     }
     if (a.dim < DP)  // padding of the key channels
         for (int r = warp; r < 2 * DC_TOKENS; r += DC_THREADS / 32)
@@ -197,58 +193,48 @@ __global__ void __launch_bounds__(DC_THREADS, 3) delta_chunk_prep_kernel(DeltaCh
     if (warp >= 5) {  // the warps that have no pairs take the operands
         for (int t = warp - 5; t < DC_TOKENS; t += 3) operands(t);
     } else {
-        // ---- A and B: 4 x 4 blocks of (i, j) below the diagonal, sixteen lanes share the channels of a block ------
-        const int block = warp * 2 + (lane >> 4), sub = lane & 15;
-        const int bi = block < 1 ? 0 : block < 3 ? 1 : block < 6 ? 2 : 3, bj = block - bi * (bi + 1) / 2;
-        float acc[32];  // A then B of the 16 pairs
+        // ---- A and B: 4 x 4 blocks of (i, j) below the diagonal, one after the other two per warp; half of the warp makes A, half B -------
+        const int sub = lane & 15;
+        const float* x_s = lane < 16 ? k_s : q_s;
+        for (int block = warp * 2; block < warp * 2 + 2; ++block) {
+            const int bi = block < 1 ? 0 : block < 3 ? 1 : block < 6 ? 2 : 3, bj = block - bi * (bi + 1) / 2;
+            float acc[16];
 #pragma unroll
-        for (int x = 0; x < 32; ++x) acc[x] = 0.f;
-        for (int d = sub; d < DP; d += 16) {
-            float gi[4], ki[4], qi[4], gj[4], kj[4];
-#pragma unroll
-            for (int x = 0; x < 4; ++x) {
-                gi[x] = g_s[(bi * 4 + x) * RS + d];
-                ki[x] = k_s[(bi * 4 + x) * RS + d];
-                qi[x] = q_s[(bi * 4 + x) * RS + d];
-                gj[x] = g_s[(bj * 4 + x) * RS + d];
-                kj[x] = k_s[(bj * 4 + x) * RS + d];
-            }
-            if (bi != bj) {  // exp(G_i - G_j) in two factors around the end of the earlier block, both at most one
+            for (int x = 0; x < 16; ++x) acc[x] = 0.f;
+            for (int d = sub; d < DP; d += 16) {
+                float gi[4], xi[4], gj[4], kj[4];
 #pragma unroll
                 for (int x = 0; x < 4; ++x) {
-                    const float e = dc_exp2(gi[x] - gj[3]);
-                    ki[x] *= e;
-                    qi[x] *= e;
-                    kj[x] *= dc_exp2(gj[3] - gj[x]);
+                    gi[x] = g_s[(bi * 4 + x) * RS + d];
+                    xi[x] = x_s[(bi * 4 + x) * RS + d];
+                    gj[x] = g_s[(bj * 4 + x) * RS + d];
+                    kj[x] = k_s[(bj * 4 + x) * RS + d];
                 }
+                if (bi != bj) {  // exp(G_i - G_j) in two factors around the end of the earlier block, both at most one
 #pragma unroll
-                for (int x = 0; x < 4; ++x)
-#pragma unroll
-                    for (int y = 0; y < 4; ++y) {
-                        acc[x * 4 + y] = fmaf(ki[x], kj[y], acc[x * 4 + y]);
-                        acc[16 + x * 4 + y] = fmaf(qi[x], kj[y], acc[16 + x * 4 + y]);
+                    for (int x = 0; x < 4; ++x) {
+                        xi[x] *= dc_exp2(gi[x] - gj[3]);
+                        kj[x] *= dc_exp2(gj[3] - gj[x]);
                     }
-            } else {
 #pragma unroll
-                for (int x = 0; x < 4; ++x)
+                    for (int x = 0; x < 4; ++x)
 #pragma unroll
-                    for (int y = 0; y <= x; ++y) {
-                        const float e = x == y ? kj[y] : kj[y] * dc_exp2(gi[x] - gj[y]);
-                        acc[x * 4 + y] = fmaf(ki[x], e, acc[x * 4 + y]);
-                        acc[16 + x * 4 + y] = fmaf(qi[x], e, acc[16 + x * 4 + y]);
-                    }
+                        for (int y = 0; y < 4; ++y) acc[x * 4 + y] = fmaf(xi[x], kj[y], acc[x * 4 + y]);
+                } else {
+#pragma unroll
+                    for (int x = 0; x < 4; ++x)
+#pragma unroll
+                        for (int y = 0; y <= x; ++y) acc[x * 4 + y] = fmaf(xi[x], x == y ? kj[y] : kj[y] * dc_exp2(gi[x] - gj[y]), acc[x * 4 + y]);
+                }
             }
-        }
-        dc_fold<32>(acc, lane, 8);
-        dc_fold<16>(acc, lane, 4);
-        dc_fold<8>(acc, lane, 2);
-        dc_fold<4>(acc, lane, 1);
-        // lane bits from the highest choose the half at every step: this lane holds values 2 sub, 2 sub + 1
-#pragma unroll
-        for (int x = 0; x < 2; ++x) {
-            const int at = sub * 2 + x, i = bi * 4 + (at & 15) / 4, j = bj * 4 + (at & 3);
-            if (at < 16) A_s[i][j] = j < i ? acc[x] * scale_s[DC_TOKENS + i] * scale_s[DC_TOKENS + j] : 0.f;
-            else B_s[i][j] = j <= i ? acc[x] * scale_s[i] * scale_s[DC_TOKENS + j] : 0.f;
+            dc_fold<16>(acc, lane, 8);
+            dc_fold<8>(acc, lane, 4);
+            dc_fold<4>(acc, lane, 2);
+            dc_fold<2>(acc, lane, 1);
+            // lane bits from the highest choose the half at every step: this lane holds value `sub`
+            const int i = bi * 4 + sub / 4, j = bj * 4 + (sub & 3);
+            if (lane < 16) A_s[i][j] = j < i ? acc[0] * scale_s[DC_TOKENS + i] * scale_s[DC_TOKENS + j] : 0.f;
+            else B_s[i][j] = j <= i ? acc[0] * scale_s[i] * scale_s[DC_TOKENS + j] : 0.f;
         }
     }
     for (int i = tid; i < DC_TOKENS * DC_TOKENS; i += DC_THREADS)  // blocks above the diagonal

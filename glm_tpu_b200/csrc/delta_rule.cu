@@ -188,42 +188,49 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(DeltaArgs a) {
 }
 
 // ---------------------------------------------------------------------------------------------------
-// out = o / rms(o) * norm * sigmoid(gate) per (row, head).  VEC: heads up to 128 wide in whole vectors, a warp takes DR_UNITS of them, four channels
-// per lane, everything asked for at once; otherwise a warp per (row, head), any size.
-#define DR_UNITS 4
+// out = o / rms(o) * norm * sigmoid(gate) per (row, head).  VEC: heads up to 128 wide in whole vectors, sixteen lanes per head with eight channels
+// each, DR_UNITS heads per half of a warp, everything asked for at once; otherwise a warp per (row, head), any size.
+#define DR_UNITS 2
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(DR_THREADS) delta_out_kernel(DeltaArgs a) {
     GLMB_PDL_PROLOGUE();
     const int lane = threadIdx.x & 31;
-    const int64_t units = (int64_t)a.rows * a.H, warp = (int64_t)blockIdx.x * DR_WARPS + (threadIdx.x >> 5);
+    const uint32_t units = (uint32_t)a.rows * a.H, warp = blockIdx.x * DR_WARPS + (threadIdx.x >> 5);
     if constexpr (VEC) {
-        const int c = lane * 4;
+        const int c = (lane & 15) * 8;
         const bool in = c < a.vdim;
-        float x[DR_UNITS][4], z[DR_UNITS][4], w[4] = {0.f, 0.f, 0.f, 0.f};
-        if (in) load4(a.norm + c, w);
+        float x[DR_UNITS][8], z[DR_UNITS][8], w[8];
+        uint32_t row[DR_UNITS], at[DR_UNITS];
 #pragma unroll
         for (int i = 0; i < DR_UNITS; ++i) {
-            const int64_t unit = warp * DR_UNITS + i;
+            const uint32_t unit = (warp * DR_UNITS + i) * 2 + (lane >> 4);
+            row[i] = unit / (uint32_t)a.H;
+            at[i] = (unit - row[i] * a.H) * a.vdim + c;
 #pragma unroll
-            for (int e = 0; e < 4; ++e) x[i][e] = z[i][e] = 0.f;
+            for (int e = 0; e < 8; ++e) x[i][e] = z[i][e] = 0.f;
             if (in && unit < units) {
-                load4(a.o + unit * a.vdim + c, x[i]);
-                load4(reinterpret_cast<const T*>(a.gate) + unit / a.H * a.gate_stride + unit % a.H * a.vdim + c, z[i]);
+                load8(a.o + (int64_t)unit * a.vdim + c, x[i]);
+                load8(reinterpret_cast<const T*>(a.gate) + (int64_t)row[i] * a.gate_stride + at[i], z[i]);
             }
         }
+        if (in) load8(a.norm + c, w);
 #pragma unroll
         for (int i = 0; i < DR_UNITS; ++i) {
-            const int64_t unit = warp * DR_UNITS + i;
-            const float ss = warp_sum(x[i][0] * x[i][0] + x[i][1] * x[i][1] + x[i][2] * x[i][2] + x[i][3] * x[i][3]);
-            const float inv = 1.f / sqrtf(ss / (float)a.vdim + a.eps);
+            float ss = 0.f;
 #pragma unroll
-            for (int e = 0; e < 4; ++e) x[i][e] = x[i][e] * inv * w[e] * sigmoidf_precise(z[i][e]);
-            if (in && unit < units) store4(reinterpret_cast<T*>(a.out) + unit / a.H * a.out_stride + unit % a.H * a.vdim + c, x[i]);
+            for (int e = 0; e < 8; ++e) ss = fmaf(x[i][e], x[i][e], ss);
+#pragma unroll
+            for (int o = 8; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+            const float inv = 1.f / sqrtf(ss / (float)a.vdim + a.eps);
+            if (!in || (warp * DR_UNITS + i) * 2 + (lane >> 4) >= units) continue;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) x[i][e] = x[i][e] * inv * w[e] * (sizeof(T) == 4 ? sigmoidf_precise(z[i][e]) : __fdividef(1.f, 1.f + __expf(-z[i][e])));
+            store8(reinterpret_cast<T*>(a.out) + (int64_t)row[i] * a.out_stride + at[i], x[i]);
         }
     } else {
         if (warp >= units) return;
         const int row = (int)(warp / a.H), h = (int)(warp % a.H);
-        const float* o = a.o + warp * a.vdim;
+        const float* o = a.o + (int64_t)warp * a.vdim;
         const T* gate = reinterpret_cast<const T*>(a.gate) + (int64_t)row * a.gate_stride + h * a.vdim;
         T* out = reinterpret_cast<T*>(a.out) + (int64_t)row * a.out_stride + h * a.vdim;
         float ss = 0.f;
@@ -278,9 +285,9 @@ GLMB_API int glmb_delta_scan(const DeltaArgs* args, void* stream) {
 
 GLMB_API int glmb_delta_out(const DeltaArgs* args, int is_f32, void* stream) {
     const DeltaArgs a = *args;
-    if (!delta_sizes_ok(a)) return 1;
-    const bool vec = !(a.vdim & 3) && a.vdim <= 128 && !(a.gate_stride & 3) && !(a.out_stride & 3);
-    const int64_t per_block = DR_WARPS * (vec ? DR_UNITS : 1);
+    if (!delta_sizes_ok(a) || (int64_t)a.rows * a.H >= (int64_t)1 << 31) return 1;
+    const bool vec = !(a.vdim & 7) && a.vdim <= 128 && !(a.gate_stride & 7) && !(a.out_stride & 7);
+    const int64_t per_block = DR_WARPS * (vec ? 2 * DR_UNITS : 1);
     const int grid = (int)(((int64_t)a.rows * a.H + per_block - 1) / per_block);
     cudaStream_t st = (cudaStream_t)stream;
     if (is_f32) {
