@@ -296,38 +296,54 @@ __global__ void __launch_bounds__(LM_WARPS * 32) latent_merge_value_kernel(Laten
         if (sub * 8 + i * 64 < a.lat) wv[i] = *reinterpret_cast<const uint4*>(w + sub * 8 + i * 64);
     }
     asm volatile("griddepcontrol.wait;" ::: "memory");
-    extern __shared__ __align__(16) float o_s[];  // [2][R][lat]
-    __shared__ float w_s[R][LM_PARTS];
+    extern __shared__ __align__(16) float o_s[];  // [SPLIT][rows][lat]
+    __shared__ float w_s[R][LM_PARTS], gate_s[R];
+    // every partial state a thread adds up is asked for before the weights are known
+    constexpr int SPLIT = R == 1 ? 2 : 1, PAIRS = R == 1 ? 1 : R / 2, MOST = R == 8 ? 8 : 16;
+    const int quads = a.rows * a.lat / 4, first = R == 1 ? (threadIdx.x >> 7) * MOST : 0, thread = R == 1 ? threadIdx.x & 127 : threadIdx.x;
+    float4 x[PAIRS][MOST];
+#pragma unroll
+    for (int k = 0; k < PAIRS; ++k) {
+        const int i = thread + k * LM_WARPS * 32, r = i * 4 / a.lat, at = i * 4 % a.lat;
+        const float* src = a.part_o + (((int64_t)r * a.H + h) * a.parts + first) * a.lat + at;
+#pragma unroll
+        for (int p = 0; p < MOST; ++p) {
+            x[k][p] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (i < quads && first + p < a.parts) x[k][p] = *reinterpret_cast<const float4*>(src + (int64_t)p * a.lat);
+        }
+    }
     if (warp < a.rows) {  // a warp per row: weights of its parts, divided by the total
         const float sink2 = a.sink ? a.sink[h] * LD_LOG2E : -INFINITY;
         float2 ml = make_float2(-INFINITY, 0.f);
         if (lane < a.parts) ml = *reinterpret_cast<const float2*>(a.part_ml + (((int64_t)warp * a.H + h) * a.parts + lane) * 2);
+        if (lane == 31) gate_s[warp] = sigmoidf_precise(__bfloat162float(reinterpret_cast<const bf16*>(a.proj)[(int64_t)warp * a.proj_stride + a.off_gate + h]));
         const float top = warp_max(fmaxf(ml.x, sink2));
         const float f = ml.x == -INFINITY ? 0.f : exp2f(ml.x - top);
         const float total = warp_sum(ml.y * f) + (a.sink ? exp2f(sink2 - top) : 0.f);
         w_s[warp][lane] = total > 0.f ? f / total : 0.f;
     }
     __syncthreads();
-    const int half = threadIdx.x >> 7, quads = a.rows * a.lat / 4, parts = (a.parts + 1) / 2;  // two halves of the parts side by side
-    for (int i = threadIdx.x & 127; i < quads; i += 128) {
-        const int r = i * 4 / a.lat, at = i * 4 % a.lat;
-        const float* src = a.part_o + (((int64_t)r * a.H + h) * a.parts + half * parts) * a.lat + at;
-        const int n = min(parts, a.parts - half * parts);
+#pragma unroll
+    for (int k = 0; k < PAIRS; ++k) {
+        const int i = thread + k * LM_WARPS * 32;
+        if (i >= quads) continue;
+        const float* f = w_s[i * 4 / a.lat] + first;
         float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 8
-        for (int p = 0; p < n; ++p) {
-            const float4 x = *reinterpret_cast<const float4*>(src + (int64_t)p * a.lat);
-            const float f = w_s[r][half * parts + p];
-            v.x = fmaf(x.x, f, v.x); v.y = fmaf(x.y, f, v.y); v.z = fmaf(x.z, f, v.z); v.w = fmaf(x.w, f, v.w);
+#pragma unroll
+        for (int p = 0; p < MOST; ++p) {
+            v.x = fmaf(x[k][p].x, f[p], v.x); v.y = fmaf(x[k][p].y, f[p], v.y);
+            v.z = fmaf(x[k][p].z, f[p], v.z); v.w = fmaf(x[k][p].w, f[p], v.w);
         }
-        *reinterpret_cast<float4*>(o_s + half * a.rows * a.lat + i * 4) = v;
+        reinterpret_cast<float4*>(o_s)[(R == 1 ? (threadIdx.x >> 7) * quads : 0) + i] = v;
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < quads; i += LM_WARPS * 32) {
-        const float4 x = reinterpret_cast<const float4*>(o_s)[i], y = reinterpret_cast<const float4*>(o_s)[quads + i];
-        reinterpret_cast<float4*>(o_s)[i] = make_float4(x.x + y.x, x.y + y.y, x.z + y.z, x.w + y.w);
+    if constexpr (SPLIT == 2) {
+        if ((int)threadIdx.x < quads) {
+            const float4 u = reinterpret_cast<const float4*>(o_s)[threadIdx.x], v = reinterpret_cast<const float4*>(o_s)[quads + threadIdx.x];
+            reinterpret_cast<float4*>(o_s)[threadIdx.x] = make_float4(u.x + v.x, u.y + v.y, u.z + v.z, u.w + v.w);
+        }
+        __syncthreads();
     }
-    __syncthreads();
 #pragma unroll
     for (int r = 0; r < R; ++r) {
         if (r >= a.rows) break;
@@ -347,8 +363,7 @@ __global__ void __launch_bounds__(LM_WARPS * 32) latent_merge_value_kernel(Laten
         sum += __shfl_xor_sync(0xffffffffu, sum, 2);
         sum += __shfl_xor_sync(0xffffffffu, sum, 4);
         if (sub == 0 && c < cols) {
-            const float z = __bfloat162float(reinterpret_cast<const bf16*>(a.proj)[(int64_t)r * a.proj_stride + a.off_gate + h]);
-            reinterpret_cast<bf16*>(a.out)[(int64_t)r * a.out_stride + h * a.vdim + c0 + c] = __float2bfloat16_rn(sum * sigmoidf_precise(z));
+            reinterpret_cast<bf16*>(a.out)[(int64_t)r * a.out_stride + h * a.vdim + c0 + c] = __float2bfloat16_rn(sum * gate_s[r]);
         }
     }
 }
@@ -395,6 +410,8 @@ GLMB_API int glmb_latent_decode(const LatentArgs* args, void* stream) {
     while (cluster < LD_CLUSTER && cluster * 2 <= tiles) cluster *= 2;
     a.parts = LD_CLUSTERS / blocks;
     if (a.parts > tiles / cluster) a.parts = tiles / cluster;
+    const int most = a.rows == 1 ? LM_PARTS : a.rows <= 4 ? 16 : 8;  // what the merge takes
+    if (a.parts > most) a.parts = most;
     if (a.parts < 1) a.parts = 1;
     const int code = a.H <= 16 ? launch_latent_decode<1>(a, cluster, (cudaStream_t)stream) : launch_latent_decode<2>(a, cluster, (cudaStream_t)stream);
     if (code) return code;

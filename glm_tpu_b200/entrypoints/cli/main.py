@@ -30,7 +30,9 @@ def _info(args) -> int:
         "engine": "glm_tpu_b200",
         "model": "GlmMoeDsaForCausalLM (GLM-5.3), FP8 e4m3 routed experts with 128x128 block scales, bf16 elsewhere",
         "other_models": {"Namizen": "small parallel-block decoder with chunked attention; bf16 (32-bit for checks), one GPU, any directory "
-                                    "with its config.json and safetensors"},
+                                    "with its config.json and safetensors",
+                         "Zikevik": "small decoder of gated-delta-rule and latent-attention layers with dense or routed feed-forwards; bf16 (32-bit "
+                                    "for checks), one GPU, any directory with its config.json and safetensors"},
         "hardware": "one box of 1, 2, 4 or 8 NVIDIA B200 (sm_100a) with NVLink peer access",
         "modes": ["one-shot answer", "sequential queue (<= 10)", "four concurrent chats (32k)", "resident session",
                   "loopback chat UI", "OpenAI-compatible /v1 (chat completions, models, tools, SSE)"],
@@ -115,7 +117,7 @@ def build_parser() -> argparse.ArgumentParser:
     ask.add_argument("--max-new-tokens", type=int)
     ask.add_argument("--wall-seconds", type=int, default=86400)
     ask.add_argument("--prepare-only", action="store_true")
-    ask.add_argument("--model", help="random:<tiny|small|glm53|namizen-tiny>[:layers], a packed checkpoint, or a Namizen directory (default: the site's)")
+    ask.add_argument("--model", help="random:<tiny|small|glm53|namizen-tiny|zikevik-tiny>[:layers], a packed checkpoint, or a Namizen or Zikevik directory (default: the site's)")
     ask.add_argument("--backend", choices=("gpu", "oracle"), default="gpu")
     ask.add_argument("--gpus", type=int)
     ask.add_argument("--site", type=Path)

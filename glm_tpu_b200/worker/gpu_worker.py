@@ -41,7 +41,7 @@ def parse_args(argv=None):
     ap.add_argument("--request", help="prepared request or batch (JSON file); optional with --keep-loaded")
     ap.add_argument("--request-sha256", help="expected request_sha256 of --request")
     ap.add_argument("--keep-loaded", action="store_true")
-    ap.add_argument("--model", default="random:tiny", help="random:<tiny|small|glm53|namizen-tiny>[:layers], a packed checkpoint directory, or a directory with config.json and safetensors")
+    ap.add_argument("--model", default="random:tiny", help="random:<tiny|small|glm53|namizen-tiny|zikevik-tiny>[:layers], a packed checkpoint directory, or a directory with config.json and safetensors")
     ap.add_argument("--backend", default="gpu", choices=["gpu", "oracle"], help="'oracle' runs the CPU contract reference")
     ap.add_argument("--context", type=int, default=0, help="context capacity (0: the request's)")
     ap.add_argument("--lanes", type=int, default=1)
